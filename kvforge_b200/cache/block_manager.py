@@ -12,6 +12,8 @@ Added: cache *groups*.  Layers that keep the same thing per token form a group w
 and tables of its own.  A ``full`` group keeps every key.  A ``window`` group keeps the last
 ``window`` keys: ``append_slots`` gives pages back once every position in them lies before
 ``write_start - window + 1`` (no later query can see them); the table entry becomes ``-1``.
+A ``chunk`` group's queries see the keys of their own chunk of ``window`` positions (counted from
+position 0): a page comes back once every position in it lies before the chunk of ``write_start``.
 A window group may also keep the first ``keep_first`` positions of every request for good
 (queries see them at any distance): the pages that hold them are never given back.
 """
@@ -33,15 +35,15 @@ RELEASED = -1
 
 @dataclass(frozen=True)
 class GroupSpec:
-    kind: str = "full"  # "full" or "window"
-    window: int | None = None
+    kind: str = "full"  # "full", "window" or "chunk"
+    window: int | None = None  # keys of a window, positions of a chunk
     keep_first: int = 0  # window groups: the first positions of a request stay visible, so their pages stay
 
     def __post_init__(self) -> None:
-        if self.kind not in ("full", "window"):
-            raise ValueError(f"cache group kind {self.kind!r} is not 'full' or 'window'")
-        if self.kind == "window" and (self.window is None or self.window <= 0):
-            raise ValueError("a window group needs a positive window")
+        if self.kind not in ("full", "window", "chunk"):
+            raise ValueError(f"cache group kind {self.kind!r} is not 'full', 'window' or 'chunk'")
+        if self.kind != "full" and (self.window is None or self.window <= 0):
+            raise ValueError(f"a {self.kind} group needs a positive {self.kind}")
         if self.keep_first < 0 or (self.keep_first and self.kind != "window"):
             raise ValueError("keep_first is a count of positions of a window group")
 
@@ -146,20 +148,22 @@ class BlockManager:
     # ------------------------------------------------------------------ sizing
     def _first_live_block(self, pool: _Pool, write_start: int) -> int:
         """First page a query at ``write_start`` or later can still see."""
-        if pool.spec.kind != "window":
+        if pool.spec.kind == "full":
             return 0
+        if pool.spec.kind == "chunk":
+            return (write_start - write_start % pool.spec.window) // self.block_size
         return max(0, write_start - pool.spec.window + 1) // self.block_size
 
     def _kept_blocks(self, pool: _Pool) -> int:
-        """Pages at the start of a request that a window group never gives back."""
-        return self.blocks_needed(pool.spec.keep_first) if pool.spec.kind == "window" else 0
+        """Pages at the start of a request that are never given back though the group gives pages back."""
+        return self.blocks_needed(pool.spec.keep_first)
 
     def _demand(self, pool: _Pool, seq_id: str | None, total_tokens: int, write_start: int) -> tuple[int, int]:
         """(pages to take, pages that come back first) for holding ``total_tokens`` tokens
         when writing starts at ``write_start``."""
         table = pool.tables.get(seq_id, []) if seq_id is not None else []
         want = self.blocks_needed(total_tokens)
-        if pool.spec.kind != "window":
+        if pool.spec.kind == "full":
             return max(0, want - len(table)), 0  # a full group never gives pages back: no holes in its table
         first = self._first_live_block(pool, write_start)
         kept = min(self._kept_blocks(pool), first)
@@ -173,7 +177,7 @@ class BlockManager:
         step, run in an otherwise empty pool (leaving the watermark free)?"""
         for pool in self._pools:
             need = self.blocks_needed(num_tokens)
-            if pool.spec.kind == "window":
+            if pool.spec.kind != "full":
                 need = min(need, self.blocks_needed(pool.spec.window - 1 + max_portion) + 1 + self._kept_blocks(pool))
             if need > pool.num_blocks - self.watermark_blocks:
                 return False
@@ -182,7 +186,7 @@ class BlockManager:
     # ------------------------------------------------------------------ admission
     def can_allocate(self, num_tokens: int, num_scheduled: int | None = None) -> bool:
         """Room for a new request of ``num_tokens`` known tokens, keeping the watermark free
-        (block_manager.py:165-170).  A window group only needs the first portion
+        (block_manager.py:165-170).  A window or chunk group only needs the first portion
         (``num_scheduled`` tokens) at once."""
         for pool in self._pools:
             n = num_tokens if pool.spec.kind == "full" else min(num_tokens, num_scheduled or num_tokens)
@@ -217,8 +221,8 @@ class BlockManager:
         return True
 
     def append_slots(self, seq_id: str, total_tokens: int, write_start: int) -> list[tuple[int, int]]:
-        """Pages for positions up to ``total_tokens`` (block_manager.py:209-236); window groups
-        first give back the pages no query from ``write_start`` on can see.  Returns the
+        """Pages for positions up to ``total_tokens`` (block_manager.py:209-236); window and chunk
+        groups first give back the pages no query from ``write_start`` on can see.  Returns the
         copies to make before the step: always none (nothing is shared)."""
         if seq_id not in self._num_tokens:
             raise KeyError(f"sequence {seq_id} has no tables")
@@ -227,7 +231,7 @@ class BlockManager:
         want = self.blocks_needed(total_tokens)
         for pool in self._pools:
             table = pool.tables[seq_id]
-            if pool.spec.kind != "window":
+            if pool.spec.kind == "full":
                 while len(table) < want:
                     table.append(pool.pop())
                 continue

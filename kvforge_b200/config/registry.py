@@ -83,6 +83,11 @@ def _ensure_builtin() -> None:
 
     if SONALIX not in ARCHITECTURES:
         register_architecture(SONALIX, SonalixConfig.from_dict, sonalix_spec)
+    from ..models.ritizen import ritizen_spec
+    from .ritizen_config import ARCHITECTURE as RITIZEN, RitizenConfig
+
+    if RITIZEN not in ARCHITECTURES:
+        register_architecture(RITIZEN, RitizenConfig.from_dict, ritizen_spec)
 
 
 _LLAMA3_32 = RopeScaling(factor=32.0, low_freq_factor=1.0, high_freq_factor=4.0, original_max_position_embeddings=8192)
@@ -135,3 +140,7 @@ PRESETS.update(GUKIRAX_PRESETS)
 from .sonalix_config import SONALIX_PRESETS  # noqa: E402
 
 PRESETS.update(SONALIX_PRESETS)
+
+from .ritizen_config import RITIZEN_PRESETS  # noqa: E402
+
+PRESETS.update(RITIZEN_PRESETS)

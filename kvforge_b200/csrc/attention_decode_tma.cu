@@ -199,9 +199,9 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   const bool seq_live = (p.single_only ? q_len == 1 : q_len > 0) && ctx > 0;  // the same for all ranges of a sequence: for a whole cluster
   const bool live = seq_live && range_lo < ctx && aligned;
   const int kv_hi = min(ctx, range_lo + split_size);
-  const int first_seen = max(range_lo, p.window > 0 ? ctx - p.window : 0);  // first key this range may show
+  const int first_seen = max(range_lo, first_key(ctx - 1, p.window));  // first key this range may show
   const int kv_lo = (first_seen / UNIT) * UNIT;
-  const bool empty = kv_lo >= kv_hi;  // wholly before the window
+  const bool empty = kv_lo >= kv_hi;  // wholly before the keys in sight
   const int n_units = (live && !empty) ? (kv_hi - kv_lo + UNIT - 1) / UNIT : 0;
   const int n_mine = n_units > warp ? (n_units - warp + NWARPS - 1) / NWARPS : 0;
   const int* bt = p.block_tables + (size_t)b * p.bt_stride;

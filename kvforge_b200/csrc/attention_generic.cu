@@ -7,7 +7,8 @@
 // ctx_b keys in its pages after this step's writes and q_b = qsl[b+1]-qsl[b] queries;
 // query i sits at position p = ctx_b - q_b + i and sees key j iff j <= p (and
 // j > p - window when window > 0, or j < keep_first: the first keys of a sequence may stay
-// visible at any distance).  S = scale * (q . k) in float, plus, when a table is given, a learned
+// visible at any distance).  window < 0 stands for chunks of -window positions counted from position 0:
+// query i then sees key j iff j <= p and both lie in the same chunk (csrc/common.cuh first_key).  S = scale * (q . k) in float, plus, when a table is given, a learned
 // bias by distance: bias[head][min(p - j, far)], `bias` float [nh][far + 1] (a head's values for
 // neighbouring keys lie side by side); softmax in float, O = P V in float, one rounding to T.
 // With softcap c > 0 the scaled score becomes c * tanh(S / c) (before any bias).  With `sinks` (float [nh])
@@ -102,9 +103,9 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attn_generic_kernel(const At
     kv_lo = blockIdx.x * p.split_size;
     if (kv_lo >= ctx) return;  // a range past the context: the merge never reads it
     kv_hi = min(ctx, kv_lo + p.split_size);
-    if (p.window > 0) win_lo = ((max(0, ctx - p.window)) / TK) * TK;
-    if (p.window > 0 && kv_hi <= win_lo && kv_lo >= p.keep_first) {
-      // a range that lies wholly before the window is empty, and says so to the merge
+    win_lo = (first_key(ctx - 1, p.window) / TK) * TK;
+    if (p.window != 0 && kv_hi <= win_lo && kv_lo >= p.keep_first) {
+      // a range that lies wholly before the keys in sight is empty, and says so to the merge
       for (int r = threadIdx.x; r < p.gh; r += blockDim.x) {
         const int head = kvh * g + chunk * p.gh + r;
         if (head < (kvh + 1) * g) {
@@ -121,7 +122,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attn_generic_kernel(const At
     const int p_first = ctx - q_len + q0;
     const int p_last = ctx - q_len + min(q0 + p.tq, q_len) - 1;
     kv_lo = 0;
-    if (p.window > 0) win_lo = (max(0, p_first - p.window + 1) / TK) * TK;
+    win_lo = (first_key(p_first, p.window) / TK) * TK;
     kv_hi = p_last + 1;
   }
   const int n_tok = SPLIT ? 1 : min(p.tq, q_len - q0);
@@ -139,13 +140,14 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attn_generic_kernel(const At
 
   // per-row state; row of (warp, slot i) is r = i * WARPS + warp
   float m[RPW], l[RPW], acc[RPW][DPL];
-  int pos[RPW], hd[RPW];
+  int pos[RPW], lo[RPW], hd[RPW];
 #pragma unroll
   for (int i = 0; i < RPW; ++i) {
     const int r = i * WARPS + warp;
     const int tok = r / p.gh, hh = chunk * p.gh + (r - tok * p.gh);
     const bool valid = (tok < n_tok) && (hh < g);
     pos[i] = valid ? (ctx - q_len + q0 + tok) : -1;  // -1: sees nothing
+    lo[i] = first_key(pos[i], p.window);
     hd[i] = kvh * g + hh;
     m[i] = -INFINITY;
     l[i] = 0.f;
@@ -161,7 +163,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attn_generic_kernel(const At
 
   for (int t0 = kv_lo; t0 < kv_hi; t0 += TK) {
     // tiles between the kept first keys and the window hold nothing any query of this CTA sees
-    if (p.window > 0 && t0 >= p.keep_first && t0 + TK <= win_lo) {
+    if (t0 >= p.keep_first && t0 + TK <= win_lo) {
       t0 = win_lo - TK;
       continue;
     }
@@ -209,7 +211,7 @@ __global__ void __launch_bounds__(WARPS * 32) paged_attn_generic_kernel(const At
 #pragma unroll
     for (int i = 0; i < RPW; ++i) {
       bool vis = (kp <= pos[i]) && (kp < kv_hi);
-      if (p.window > 0) vis = vis && (kp > pos[i] - p.window || kp < p.keep_first);
+      vis = vis && (kp >= lo[i] || kp < p.keep_first);
       if (SPLIT) vis = vis && (kp >= kv_lo);
       float sc = -INFINITY;
       if (vis) {

@@ -1,7 +1,7 @@
 // Paged grouped-query attention for bfloat16 on the tensor cores (mma.sync m16n8k16), head
 // sizes 64 and 128.  Same contract as attention_generic.cu: sequence b has ctx_b keys after
 // this step's writes and q_b queries; query i sits at p = ctx_b - q_b + i and sees key j
-// iff j <= p (and j > p - window when window > 0); softmax in float, one rounding.  The tile
+// iff j <= p (and j > p - window when window > 0; in the same chunk of -window positions when window < 0); softmax in float, one rounding.  The tile
 // Both forms also take, under a window, first keys that stay visible at any distance (j < keep_first)
 // and a bias on the scaled scores by distance and head: bias[head][min(p - j, far)] (float [nh][far + 1]);
 // a soft cap c on the scaled scores (c * tanh(S / c), before any bias); and a sink a head, a learned number whose
@@ -334,7 +334,7 @@ __global__ void __launch_bounds__(NWARPS * 32) attn_mma_tile_kernel(const MmaPar
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int p_first = ctx - q_len + q0;
   const int kv_hi = p_first + n_tok;  // one past the last position any row sees
-  const int kv_lo = p.window > 0 ? (max(0, p_first - p.window + 1) / BN) * BN : 0;
+  const int kv_lo = (first_key(p_first, p.window) / BN) * BN;
   const int* bt = p.block_tables + (size_t)b * p.bt_stride;
 
   TileLoader<D> loader;
@@ -347,7 +347,7 @@ __global__ void __launch_bounds__(NWARPS * 32) attn_mma_tile_kernel(const MmaPar
     const int r = warp * 16 + (lane >> 2) + 8 * h;
     const int tok = r / g;
     pos[h] = tok < n_tok ? p_first + tok : -1;  // -1: a row past the tile's tokens sees nothing
-    lo[h] = p.window > 0 ? pos[h] - p.window + 1 : 0;
+    lo[h] = first_key(pos[h], p.window);
     head[h] = kvh * g + (r - tok * g);
   }
   // tiles that hold kept first keys and lie wholly before the window's first tile are walked first
@@ -368,7 +368,7 @@ __global__ void __launch_bounds__(NWARPS * 32) attn_mma_tile_kernel(const MmaPar
   // and starts at or after the last row's window
   const int warp_tok0 = (warp * 16) / g, warp_tok1 = min(n_tok - 1, (warp * 16 + 15) / g);
   const int all_hi = p_first + warp_tok0;  // keys <= this are seen by every valid row of the warp
-  const int all_lo = p.window > 0 ? p_first + warp_tok1 - p.window + 1 : 0;
+  const int all_lo = first_key(p_first + warp_tok1, p.window);
   const bool rows_full = (warp * 16 + 15) / g < n_tok;  // no row of the warp lies past the tile's tokens
   loader.load(p, bt, kvh, ctx, tile_key0(0), smem, smem + TILE_BYTES);
   cp_async_commit();
@@ -442,7 +442,7 @@ __global__ void __launch_bounds__(NWARPS * 32) attn_mma_split_kernel(const MmaPa
   const bool live = q_len > 0 && ctx > 0 && kv_lo < ctx;
   const int kv_hi = min(ctx, kv_lo + p.split_size);
   const int key_lo = kv_lo;
-  if (p.window > 0) kv_lo = max(kv_lo, (max(0, ctx - p.window) / BN) * BN);
+  if (live) kv_lo = max(kv_lo, (first_key(ctx - 1, p.window) / BN) * BN);
   // tiles of the range that hold kept first keys and lie before the window's first tile are walked first
   const int keep = p.window > 0 ? p.keep_first : 0;
   const int keep_hi = min(min(kv_hi, kv_lo), ((keep + BN - 1) / BN) * BN);
@@ -489,7 +489,7 @@ __global__ void __launch_bounds__(NWARPS * 32) attn_mma_split_kernel(const MmaPa
   }
   // every row sees the keys of this range that lie inside the window; keys at or past
   // kv_hi were zero-filled and are masked
-  const int first_seen = max(key_lo, p.window > 0 ? ctx - p.window : 0);
+  const int first_seen = max(key_lo, first_key(ctx - 1, p.window));
   const int lo[2] = {first_seen, first_seen};
   const int hi[2] = {kv_hi - 1, kv_hi - 1};
   const int qpos[2] = {ctx - 1, ctx - 1};

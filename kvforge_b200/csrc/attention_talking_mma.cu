@@ -529,3 +529,8 @@ KVF_API int kvf_talking_attention_mma_bf16(
     return pl.mt == 1 ? launch_mma<64, 64, 1, false>(p, grid, pl.smem, st) : launch_mma<64, 64, 2, false>(p, grid, pl.smem, st);
   return launch_mma<128, 32, 1, false>(p, grid, pl.smem, st);
 }
+
+KVF_API int kvf_talking_set_pdl(int enabled) {
+  g_pdl_enabled = enabled ? 1 : 0;
+  return 0;
+}

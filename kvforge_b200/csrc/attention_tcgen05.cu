@@ -335,7 +335,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
   const int n_tok = live ? min(tq, q_len - q0) : 0;
   const int p_first = ctx - q_len + q0;
   const int kv_hi = p_first + n_tok;
-  const int kv_lo = p.window > 0 ? (max(0, p_first - p.window + 1) / BN) * BN : 0;
+  const int kv_lo = live ? (first_key(p_first, p.window) / BN) * BN : 0;
   const int n_tiles = live ? (kv_hi - kv_lo + BN - 1) / BN : 0;
 
   if (threadIdx.x == 0) {
@@ -560,7 +560,7 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
     const int tok = r / g, hh = r - tok * g;
     const bool valid = tok < n_tok;
     const int pos = valid ? p_first + tok : -1;
-    const int lo = p.window > 0 ? pos - p.window + 1 : 0;
+    const int lo = first_key(pos, p.window);
     const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;
     const uint32_t my_s = tmem_s + lane_addr + (uint32_t)(grp * BN), my_o = tmem_o + lane_addr + (uint32_t)(grp * D);
     const uint32_t s_bar = s_full0 + 8 * grp, p_bar = p_full0 + 8 * grp, pv_bar = pv_done0 + 8 * grp;

@@ -94,6 +94,15 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
   return r;
 }
 
+// The first key that a query at position `pos` sees (it sees no key after itself): span > 0: the last `span` keys, itself
+// included (a sliding window); span < 0: the keys of its own chunk of -span positions, chunks counted from position 0;
+// span == 0: every key.  It never falls as `pos` grows.
+__device__ __forceinline__ int first_key(int pos, int span) {
+  if (span == 0 || pos < 0) return 0;
+  if (span < 0) return pos - pos % (-span);
+  return pos - span + 1 > 0 ? pos - span + 1 : 0;
+}
+
 // 8 bfloat16 values (one 16-byte load) to floats.
 __device__ __forceinline__ void bf16x8_to_float(const uint4& u, float* f) {
   const __nv_bfloat162* p = reinterpret_cast<const __nv_bfloat162*>(&u);

@@ -1,7 +1,7 @@
 // What a layer needs around its matrix products when every sublayer's result is gated, normed and only then
 // added to the residual stream, and when queries and keys are rotated and then normed per head:
 //
-//   norm_step    : resid += norm_post(y * sigmoid(z + b)) ; out = norm_next(resid)   (one pass over a row)
+//   norm_step    : resid += norm_post((y + y_bias) * sigmoid(z + b)) ; out = norm_next(resid)   (one pass over a row)
 //   qk_prepare   : rotation of split pairs, per-head RMS norm without a weight, keys and values to the cache
 //   unary_act    : xIELU, squared ReLU or tanh-GELU on the rows of an inner activation
 //
@@ -20,6 +20,7 @@ struct NormStepParams {
   const float* y_parts;    // ... or float slices [nsplit][*, W] that are summed in slice order, or null
   long long y_stride, split_stride;
   int nsplit;
+  const float* y_bias;     // [W] joins the pending result first, or null
   const void* z;           // gate logits in the storage type [*, z_stride] (the gate is sigmoid(z + z_bias)), or null
   long long z_stride;
   const float* z_bias;     // [W] or null
@@ -74,6 +75,7 @@ __global__ void __launch_bounds__(256) norm_step_kernel(const NormStepParams p) 
       if (y) a = to_float<T>(y[i]);
       if (yp)
         for (int s = 0; s < p.nsplit; ++s) a += yp[(size_t)s * p.split_stride + i];
+      if (p.y_bias) a += p.y_bias[i];
       if (z) {
         const float g = to_float<T>(z[i]) + (p.z_bias ? p.z_bias[i] : 0.f);
         a *= 1.f / (1.f + expf(-g));
@@ -207,6 +209,16 @@ __global__ void __launch_bounds__(256) norm_step_vec_kernel(const NormStepParams
     }
   }
   if (pending) {
+    if (p.y_bias) {
+#pragma unroll
+      for (int it = 0; it < NIT; ++it) {
+        if (!live[it]) continue;
+        float t[4];
+        Vec4<float>::load(p.y_bias + (it * 256 + threadIdx.x) * 4, t);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) a[it][e] += t[e];
+      }
+    }
     if (z) {
 #pragma unroll
       for (int it = 0; it < NIT; ++it)
@@ -242,7 +254,7 @@ template <typename T>
 bool norm_step_vec_ok(const NormStepParams& p) {
   auto al = [](const void* q, size_t n) { return q == nullptr || ((uintptr_t)q % n) == 0; };
   constexpr size_t TB = 4 * sizeof(T);
-  return p.W % 4 == 0 && p.W <= 4 * 256 * 4 && al(p.resid, 16) && al(p.y_parts, 16) && al(p.z_bias, 16) && al(p.post_w, 16) &&
+  return p.W % 4 == 0 && p.W <= 4 * 256 * 4 && al(p.resid, 16) && al(p.y_parts, 16) && al(p.z_bias, 16) && al(p.y_bias, 16) && al(p.post_w, 16) &&
          al(p.next_w, 16) && al(p.y, TB) && al(p.z, TB) && al(p.out, TB) && p.y_stride % 4 == 0 && p.z_stride % 4 == 0 &&
          p.out_stride % 4 == 0 && p.split_stride % 4 == 0;
 }
@@ -328,7 +340,7 @@ __global__ void __launch_bounds__(128) qk_prepare_kernel(T* __restrict__ x, long
 }
 
 // ---------------------------------------------------------------- activations of one input
-// kind 0: xIELU with the two numbers (p, q) of `ab`: z > 0: softplus(p) z^2 + z/2; z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2
+// of x + bias (bias [cols] or null).  kind 0: xIELU with the two numbers (p, q) of `ab`: z > 0: softplus(p) z^2 + z/2; z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2
 // kind 1: relu(z)^2     kind 2: 0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))
 __device__ __forceinline__ float softplus_f(float x) { return x > 20.f ? x : log1pf(expf(x)); }
 
@@ -344,7 +356,7 @@ __device__ __forceinline__ float unary_act(float z, int kind, float ap, float aq
 template <typename T>
 __global__ void __launch_bounds__(256) unary_act_kernel(const T* __restrict__ in, long long in_stride, T* __restrict__ out,
                                                          long long out_stride, long long rows, int cols, int kind,
-                                                         const float* __restrict__ ab) {
+                                                         const float* __restrict__ ab, const float* __restrict__ bias) {
   pdl_launch();
   pdl_wait();
   float ap = 0.f, aq = 0.f;
@@ -356,7 +368,7 @@ __global__ void __launch_bounds__(256) unary_act_kernel(const T* __restrict__ in
   for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (long long)gridDim.x * blockDim.x) {
     const long long r = idx / cols;
     const int c = (int)(idx - r * cols);
-    out[r * out_stride + c] = from_float<T>(unary_act(to_float<T>(in[r * in_stride + c]), kind, ap, aq));
+    out[r * out_stride + c] = from_float<T>(unary_act(to_float<T>(in[r * in_stride + c]) + (bias ? bias[c] : 0.f), kind, ap, aq));
   }
 }
 
@@ -376,14 +388,14 @@ KVF_API int kvf_gated_set_pdl(int enabled) {
 #define KVF_GATED_API(SUF, T)                                                                                          \
   KVF_API int kvf_norm_step_##SUF(float* resid, const int* rows, const void* y, const float* y_parts, long long y_stride, \
                                   long long split_stride, int nsplit, const void* z, long long z_stride,              \
-                                  const float* z_bias, const float* post_w, const float* next_w, void* out,           \
+                                  const float* z_bias, const float* y_bias, const float* post_w, const float* next_w, void* out, \
                                   long long out_stride, int n_rows, int W, int centred, int store_normed, float eps,  \
                                   cudaStream_t st) {                                                                  \
     if (n_rows <= 0) return 0;                                                                                        \
     if (W <= 0 || (y && y_parts) || (store_normed && rows)) return (int)cudaErrorInvalidValue;                        \
     NormStepParams p;                                                                                                 \
     p.resid = resid; p.rows = rows; p.y = y; p.y_parts = y_parts; p.y_stride = y_stride; p.split_stride = split_stride; \
-    p.nsplit = nsplit; p.z = z; p.z_stride = z_stride; p.z_bias = z_bias; p.post_w = post_w; p.next_w = next_w;       \
+    p.nsplit = nsplit; p.z = z; p.z_stride = z_stride; p.z_bias = z_bias; p.y_bias = y_bias; p.post_w = post_w; p.next_w = next_w;       \
     p.out = out; p.out_stride = out_stride; p.W = W; p.centred = centred; p.store_normed = store_normed; p.eps = eps; \
     if (norm_step_vec_ok<T>(p)) {                                                                                     \
       if (W <= 1024) return launch(norm_step_vec_kernel<T, 1>, dim3(n_rows), dim3(256), 0, st, p);                    \
@@ -412,11 +424,11 @@ KVF_API int kvf_gated_set_pdl(int enabled) {
                   nkv, d, dv, block_size, num_slots, err);                                                            \
   }                                                                                                                   \
   KVF_API int kvf_unary_act_##SUF(const void* in, long long in_stride, void* out, long long out_stride, long long rows, \
-                                  int cols, int kind, const float* ab, cudaStream_t st) {                             \
+                                  int cols, int kind, const float* ab, const float* bias, cudaStream_t st) {          \
     if (rows <= 0 || cols <= 0) return 0;                                                                             \
     if (kind < 0 || kind > 2 || (kind == 0 && !ab)) return (int)cudaErrorInvalidValue;                                \
     return launch(unary_act_kernel<T>, dim3(grid_for(rows * cols)), dim3(256), 0, st, (const T*)in, in_stride, (T*)out, \
-                  out_stride, rows, cols, kind, ab);                                                                  \
+                  out_stride, rows, cols, kind, ab, bias);                                                                  \
   }
 
 KVF_GATED_API(f32, float)

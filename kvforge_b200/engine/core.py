@@ -93,7 +93,7 @@ class EngineCore:
             self.num_blocks = max(1, max_num_seqs * -(-self.max_model_len // cache.block_size))
         else:
             self.num_blocks = cache.resolve_num_blocks(per_block)
-        groups = [GroupSpec(g.need.kind, g.need.window, g.need.keep_first if g.need.kind == "window" else 0) for g in self.model.groups] or [GroupSpec()]
+        groups = [GroupSpec(g.need.kind, g.need.window, g.need.keep_first) for g in self.model.groups] or [GroupSpec()]
         self.block_manager = BlockManager(self.num_blocks, cache.block_size, cache.watermark, groups)
         self.state_slots = StateSlotPool(max_num_seqs)
         self.pool = KVPool(self.model, self.num_blocks, cache.block_size, max_num_seqs, self.dtype, self.device)

@@ -73,6 +73,8 @@ class Runtime:
                 what.append("a cache slot outside the pool")
             if flag & 4:
                 what.append("a bounded wait inside a kernel ran out")
+            if flag & 16:
+                what.append("a position beyond the model's table of positions")
             raise RuntimeError("device-side check failed: " + ", ".join(what or [f"flag {flag}"]))
 
 

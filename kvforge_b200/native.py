@@ -36,6 +36,8 @@ LIBRARIES: dict[str, tuple[list[str], list[str]]] = {
     # one entry point that allocates nothing (csrc/kvforge_noalloc.h); a library of its own, so
     # that only a process that asks for it holds its built-in scratch array
     "noalloc": (["attention_decode_noalloc.cu"], []),
+    # the short causal convolution of mixers with a running state
+    "conv": (["causal_conv.cu"], []),
     # what mixers with a running state, several residual streams and the general rotary form need; a
     # library of its own, so that a model without them never compiles it
     "mixers": (["sequence_mix_f32.cu", "sequence_mix_bf16.cu", "streams.cu"], []),
@@ -43,10 +45,14 @@ LIBRARIES: dict[str, tuple[list[str], list[str]]] = {
     # library of its own for the same reason
     "routed": (["head_ops.cu", "experts.cu"], []),
     # layers whose sublayer results are gated and normed before they join the residual stream, heads that are
-    # rotated and then normed, attention whose heads talk before the softmax; a library of its own for the same reason
-    "gated": (["gated_ops.cu", "attention_talking_f32.cu", "attention_talking_bf16.cu", "attention_talking_mma.cu"], []),
-    # a recurrent mixer with a fixed decay a head and a norm without statistics; a library of its own for the same reason
-    "decay": (["retention.cu", "tanh_norm.cu"], []),
+    # rotated and then normed; attention whose heads talk before the softmax; libraries of their own for the same reason
+    "gated": (["gated_ops.cu"], []),
+    "talking": (["attention_talking_f32.cu", "attention_talking_bf16.cu", "attention_talking_mma.cu"], []),
+    # recurrent mixers with one decay a head or a token and head, the norm and gate after them, a norm without statistics;
+    # a library of its own for the same reason
+    "decay": (["retention.cu", "state_space.cu", "tanh_norm.cu"], []),
+    # attention whose queries and keys are normed as one vector and whose result is gated, learned positions
+    "joint": (["joint_ops.cu"], []),
 }
 
 _loaded: dict[str, ctypes.CDLL] = {}

@@ -39,8 +39,10 @@ _SIGNATURES = {
     "kvf_sample_f32": "pliippppppp",
     "kvf_argmax_f32": "pliipipp",
     "kvf_scale_softcap_f32": "plffp",
+    # library "conv"
+    "kvf_causal_conv_{s}": "pippplppiiiiipiip",
+    "kvf_conv_set_pdl": "i",
     # library "mixers"
-    "kvf_causal_conv_{s}": "pipplppiiiiipiip",
     "kvf_gated_delta_{s}": "pppipipippiplpippiiiiiffiippppilp",
     "kvf_gated_head_norm_{s}": "pipipfiliipip",
     "kvf_hc_step_{s}": "pppilppppppiiifp",
@@ -64,18 +66,26 @@ _SIGNATURES = {
     "kvf_gemm_grouped_tcgen05_bf16": "pppiiiiiiipppipfffp",
     "kvf_routed_set_pdl": "i",
     # library "gated"
-    "kvf_norm_step_{s}": "pppplliplppppliiiifp",
+    "kvf_norm_step_{s}": "pppplliplpppppliiiifp",
     "kvf_qk_prepare_{s}": "pliiippiifpppiiiiiilpp",
-    "kvf_unary_act_{s}": "plplliipp",
+    "kvf_unary_act_{s}": "plplliippp",
     "kvf_talking_attention_{s}": "pppppppppiiiiiiiiiifiiiippp",
     "kvf_talking_attention_mma_bf16": "pppppppppiiiiiiiiiifiiiippp",
     "kvf_talking_mma_ok": "iiiiii",
+    "kvf_talking_set_pdl": "i",
     "kvf_gated_set_pdl": "i",
     # library "decay"
-    "kvf_retention_{s}": "pliiippiifpplplppiliiipppip",
+    "kvf_retention_{s}": "pliiippiifipplplppiliiipppip",
     "kvf_retention_gate_{s}": "plplfiliiplp",
     "kvf_tanh_norm_{s}": "pppilfppppplip",
     "kvf_decay_set_pdl": "i",
+    "kvf_state_space_{s}": "plplppplplppiliiiippppip",
+    "kvf_wide_norm_gate_{s}": "plpplipliipffliiplp",
+    # library "joint"
+    "kvf_joint_norm_cache_{s}": "plpilipppiifpppiiiiiilpp",
+    "kvf_output_gate_{s}": "plplifpliiip",
+    "kvf_add_position_rows_{s}": "pppiiipp",
+    "kvf_joint_set_pdl": "i",
 }
 _CTYPES = {"p": ctypes.c_void_p, "i": ctypes.c_int, "l": ctypes.c_longlong, "f": ctypes.c_float}
 
@@ -155,7 +165,10 @@ def set_pdl(enabled: bool) -> None:
 
 
 # every shared library has a flag of its own; it follows the core's once the library is loaded
-_PDL_SETTERS = {"mixers": "kvf_mixers_set_pdl", "routed": "kvf_routed_set_pdl", "gated": "kvf_gated_set_pdl", "decay": "kvf_decay_set_pdl"}
+_PDL_SETTERS = {
+    "conv": "kvf_conv_set_pdl", "mixers": "kvf_mixers_set_pdl", "routed": "kvf_routed_set_pdl", "gated": "kvf_gated_set_pdl",
+    "talking": "kvf_talking_set_pdl", "decay": "kvf_decay_set_pdl", "joint": "kvf_joint_set_pdl",
+}  # fmt: skip
 _library_pdl: dict[str, bool] = {}
 
 
@@ -554,9 +567,11 @@ def paged_attention(
     bias: DistanceBias | None = None,
     softcap: float = 0.0,
     sinks: torch.Tensor | None = None,
+    chunk: int = 0,
 ) -> None:
     """Paged GQA attention of a flat batch (the contract is at the top of
-    ``csrc/attention_generic.cu``).
+    ``csrc/attention_generic.cu``).  ``window`` (0: none): a query sees the last ``window`` keys.  ``chunk`` (0: none; not
+    with a window): a query sees the keys of its own chunk of ``chunk`` positions, counted from position 0.
 
     ``dv``: size of a value head when it differs from ``d`` (``vcache`` is then
     ``[num_blocks, nkv, block_size, dv]`` and ``out`` ``[N, nh*dv]``); only the FP32-pipe kernel
@@ -584,14 +599,19 @@ def paged_attention(
     context, over all pairs, are at most this many (``attention_wave_target``).
     """
     s = _suffix(q.dtype)
+    _rows2d(q, None, "q")
     capped = float(softcap) > 0.0 or sinks is not None
+    if chunk:
+        if window or keep_first or chunk < 0:
+            raise ValueError("paged_attention: chunk is a positive number of positions, without a window and kept first keys")
+        window = -int(chunk)  # what the kernels call a span below zero
     if float(softcap) < 0.0:
         raise ValueError("paged_attention: softcap must be positive (0: none)")
     special = vcache is kcache or keep_first > 0 or bias is not None or d > 256 or (dv or d) > 256 or capped
     # kept first keys and a bias alone, on heads of 64 or 128 in bfloat16 with many queries: the tile form of the mma.sync kernel
     biased_mma = (
         special and vcache is not kcache and (dv or d) == d and kernel == "auto"
-        and mma_attention_supported(q.dtype, nh, nkv, d, scratch is not None) and (q_stride or q.shape[-1]) % 2 == 0 and out.shape[-1] % 2 == 0
+        and mma_attention_supported(q.dtype, nh, nkv, d, scratch is not None) and (q_stride or q.stride(0)) % 2 == 0 and out.shape[-1] % 2 == 0
         and (scratch is None or len(scratch) > 2)
     )  # fmt: skip
     if special and not biased_mma:
@@ -599,7 +619,6 @@ def paged_attention(
             raise ValueError("only the FP32-pipe attention kernel takes kept first keys, a distance bias, capped scores, sinks, values inside keys or heads wider than 256")
         kernel = "generic"
     check_head_dim(d, MAX_KEY_DIM if special and not biased_mma else 256)
-    _need(q, None, "q")
     _need(out, q.dtype, "out")
     _need(kcache, q.dtype, "kcache")
     _need(vcache, q.dtype, "vcache")
@@ -639,7 +658,7 @@ def paged_attention(
         kernel = "generic"
     block_size = kcache.shape[2]
     if q_stride is None:
-        q_stride = q.shape[-1]
+        q_stride = q.stride(0)
     bt_stride = block_tables.shape[-1] if block_tables.dim() == 2 else block_tables.numel() // max(1, num_seqs)
     split, max_splits, grid_splits, pa, pm, tickets = 0, 0, 0, None, None, None
     if scratch is not None:
@@ -1099,6 +1118,7 @@ def splitmix64(z: int) -> int:
 # ------------------------------------------------------------------ mixers with a running state (library "mixers")
 
 MIXERS_LIB = "mixers"
+CONV_LIB = "conv"
 
 
 def _rows2d(t: torch.Tensor, dtype: torch.dtype | None, what: str) -> None:
@@ -1119,12 +1139,12 @@ def _state_view(state: torch.Tensor, width: int, what: str) -> tuple[int, int]:
 
 def causal_conv(
     x: torch.Tensor, weight: torch.Tensor, state: torch.Tensor, qsl: torch.Tensor, state_slots: torch.Tensor,
-    num_seqs: int, out: torch.Tensor, activation: str | None = None, max_query_len: int = 0,
+    num_seqs: int, out: torch.Tensor, activation: str | None = None, max_query_len: int = 0, bias: torch.Tensor | None = None,
 ) -> None:  # fmt: skip
     """Short causal convolution over time per channel of a flat batch, and the state moved on.
 
     ``x [N, C]`` (rows may be a slice of a wider buffer), ``weight`` float ``[C, taps]`` whose last
-    column multiplies the current token, ``state`` float ``[slots, (taps-1)*C]``: the last
+    column multiplies the current token, ``bias`` float ``[C]`` or ``None``, ``state`` float ``[slots, (taps-1)*C]``: the last
     ``taps-1`` inputs of each sequence, oldest first, zeros before its start.  ``out [N, C]`` gets
     the sums (``activation``: ``None`` or ``"silu"``); afterwards the state holds this step's last
     inputs.  Sequences without rows and slots below zero are left alone.  ``max_query_len`` (0 =
@@ -1137,6 +1157,10 @@ def causal_conv(
     taps = weight.shape[1]
     if tuple(weight.shape) != (c, taps) or tuple(out.shape) != (n, c):
         raise ValueError("causal_conv: shapes do not agree")
+    if bias is not None:
+        _need(bias, torch.float32, "conv bias")
+        if bias.numel() != c:
+            raise ValueError("causal_conv: one bias per channel")
     if activation not in (None, "silu"):
         raise ValueError("causal_conv: activation must be None or 'silu'")
     sptr, sstride = (0, 0) if taps == 1 else _state_view(state, (taps - 1) * c, "conv state")
@@ -1144,8 +1168,8 @@ def causal_conv(
     _need(state_slots, torch.int32, "state_slots")
     name = f"kvf_causal_conv_{s}"
     _check(
-        _fn(name, MIXERS_LIB)(
-            _ptr(x), x.stride(0), _ptr(weight), sptr, sstride, _ptr(qsl), _ptr(state_slots), n, num_seqs, c, taps,
+        _fn(name, CONV_LIB)(
+            _ptr(x), x.stride(0), _ptr(weight), _ptr(bias), sptr, sstride, _ptr(qsl), _ptr(state_slots), n, num_seqs, c, taps,
             1 if activation == "silu" else 0, _ptr(out), out.stride(0), int(max_query_len), _stream(),
         ),
         name,
@@ -1681,21 +1705,30 @@ def moe_experts(
     )  # fmt: skip
 
 
-# ------------------------------------------------------------------ library "gated"
+# ------------------------------------------------------------------ libraries "gated" and "talking"
 # gated and normed sublayer results, rotation followed by a head norm, attention whose heads talk
 
 GATED_LIB = "gated"
+TALKING_LIB = "talking"
+
+
+@dataclass
+class Biased:
+    """A product's result (a tensor in the storage type or ``Partials``) that still lacks its bias, float ``[W]``."""
+
+    y: "torch.Tensor | Partials"
+    bias: torch.Tensor
 
 
 @dataclass
 class GatedWrite:
     """A sublayer's result that is still to be gated, normed and added to the residual stream:
-    ``resid += norm(y * sigmoid(z + z_bias)) * post_w``.  ``y``: a tensor in the storage type or the
-    ``Partials`` of a split product; ``z``: gate logits in the storage type ``[N, W]`` (a view with a row
+    ``resid += norm(y * sigmoid(z + z_bias)) * post_w``.  ``y``: a tensor in the storage type, the
+    ``Partials`` of a split product, or either as ``Biased``; ``z``: gate logits in the storage type ``[N, W]`` (a view with a row
     stride of its own is fine) or ``None`` (no gate); ``post_w``: float ``[W]`` or ``None`` (added as it is).
     The norm that consumes it decides the norm's kind and eps: the same as its own."""
 
-    y: "torch.Tensor | Partials"
+    y: "torch.Tensor | Partials | Biased"
     z: torch.Tensor | None = None
     z_bias: torch.Tensor | None = None
     post_w: torch.Tensor | None = None
@@ -1713,7 +1746,7 @@ def norm_step(
 ) -> None:
     """One pass over every row of the float residual stream ``resid [N, W]``:
 
-    * ``pending`` (``None``, ``ADDED``, a tensor, ``Partials`` or a ``GatedWrite``) is gated, normed and added
+    * ``pending`` (``None``, ``ADDED``, a tensor, ``Partials``, ``Biased`` or a ``GatedWrite``) is gated, normed and added
       (the sum is written back unless ``rows`` picks rows);
     * ``out`` (storage type, rows may be a view of a wider buffer) gets the row normed with ``next_w``
       (``None``: the row itself); with ``store_normed`` the normed row also replaces the residual row.
@@ -1736,20 +1769,24 @@ def norm_step(
         s = None
     yptr = pptr = zptr = None
     ystride = sstride = zstride = nsplit = 0
+    y_bias = None
     if gw is not None:
-        if isinstance(gw.y, Partials):
-            _need(gw.y.t, torch.float32, "partials", contiguous=False)
-            if gw.y.t.shape[-1] != w or gw.y.t.stride(1) != w or gw.y.t.stride(2) != 1:
+        y = gw.y
+        if isinstance(y, Biased):
+            y, y_bias = y.y, y.bias
+        if isinstance(y, Partials):
+            _need(y.t, torch.float32, "partials", contiguous=False)
+            if y.t.shape[-1] != w or y.t.stride(1) != w or y.t.stride(2) != 1:
                 raise ValueError("norm_step: partials must be [S, M, W] with dense rows")
-            pptr, nsplit, sstride = _ptr(gw.y.t), gw.y.nsplit, gw.y.split_stride
+            pptr, nsplit, sstride = _ptr(y.t), y.nsplit, y.split_stride
         else:
-            _need(gw.y, None, "pending result", contiguous=False)
-            if gw.y.dim() != 2 or gw.y.stride(1) != 1 or gw.y.shape[1] != w:
+            _need(y, None, "pending result", contiguous=False)
+            if y.dim() != 2 or y.stride(1) != 1 or y.shape[1] != w:
                 raise ValueError("norm_step: the pending result must be [N, W] with unit inner stride")
-            if s is not None and _suffix(gw.y.dtype) != s:
+            if s is not None and _suffix(y.dtype) != s:
                 raise TypeError("norm_step: the pending result and out must have the storage type")
-            s = _suffix(gw.y.dtype)
-            yptr, ystride = _ptr(gw.y), gw.y.stride(0)
+            s = _suffix(y.dtype)
+            yptr, ystride = _ptr(y), y.stride(0)
         if gw.z is not None:
             _need(gw.z, None, "gate logits", contiguous=False)
             if gw.z.dim() != 2 or gw.z.stride(1) != 1 or gw.z.shape[1] != w:
@@ -1758,7 +1795,7 @@ def norm_step(
                 raise TypeError("norm_step: gate logits must have the storage type")
             s = _suffix(gw.z.dtype)
             zptr, zstride = _ptr(gw.z), gw.z.stride(0)
-        for t, what in ((gw.z_bias, "gate bias"), (gw.post_w, "post-norm weight")):
+        for t, what in ((gw.z_bias, "gate bias"), (y_bias, "result bias"), (gw.post_w, "post-norm weight")):
             if t is not None:
                 _need(t, torch.float32, what)
                 if t.numel() != w:
@@ -1777,7 +1814,7 @@ def norm_step(
     _check(
         _fn(name, GATED_LIB)(
             _ptr(resid), _ptr(rows), yptr, pptr, ystride, sstride, nsplit, zptr, zstride,
-            _ptr(gw.z_bias) if gw else None, _ptr(gw.post_w) if gw else None, _ptr(next_w), optr, ostride,
+            _ptr(gw.z_bias) if gw else None, _ptr(y_bias), _ptr(gw.post_w) if gw else None, _ptr(next_w), optr, ostride,
             n_rows, w, 1 if centred else 0, 1 if store_normed else 0, float(eps), _stream(),
         ),
         name,
@@ -1821,8 +1858,8 @@ def qk_prepare(
 UNARY_ACTIVATIONS = {"xielu": 0, "relu2": 1, "gelu_tanh": 2}
 
 
-def unary_act(x: torch.Tensor, out: torch.Tensor, kind: str, ab: torch.Tensor | None = None) -> None:
-    """``out = act(x)`` row by row in float, rounded once.  ``xielu`` with the two numbers ``ab = (p, q)``:
+def unary_act(x: torch.Tensor, out: torch.Tensor, kind: str, ab: torch.Tensor | None = None, bias: torch.Tensor | None = None) -> None:
+    """``out = act(x + bias)`` (``bias`` float ``[cols]`` or ``None``) row by row in float, rounded once.  ``xielu`` with the two numbers ``ab = (p, q)``:
     ``z > 0: softplus(p) z^2 + z/2``, ``z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2``; ``relu2``:
     ``relu(z)^2``; ``gelu_tanh``: ``0.5 z (1 + tanh(sqrt(2/pi) (z + 0.044715 z^3)))``."""
     s = _suffix(x.dtype)
@@ -1834,8 +1871,12 @@ def unary_act(x: torch.Tensor, out: torch.Tensor, kind: str, ab: torch.Tensor | 
         _need(ab, torch.float32, "xielu parameters")
         if ab.numel() != 2:
             raise ValueError("unary_act: xielu takes two numbers")
+    if bias is not None:
+        _need(bias, torch.float32, "activation bias")
+        if bias.numel() != x.shape[1]:
+            raise ValueError("unary_act: one bias a column")
     name = f"kvf_unary_act_{s}"
-    _check(_fn(name, GATED_LIB)(_ptr(x), x.stride(0), _ptr(out), out.stride(0), x.shape[0], x.shape[1], UNARY_ACTIVATIONS[kind], _ptr(ab), _stream()), name)
+    _check(_fn(name, GATED_LIB)(_ptr(x), x.stride(0), _ptr(out), out.stride(0), x.shape[0], x.shape[1], UNARY_ACTIVATIONS[kind], _ptr(ab), _ptr(bias), _stream()), name)
 
 
 def scale_softcap(logits: torch.Tensor, scale: float, cap: float) -> None:
@@ -1859,7 +1900,7 @@ def talking_mma_supported(dtype: torch.dtype, nh: int, nkv: int, d: int, dv: int
         return False
     key = (nh, nkv, d, bool(decode_form), bool(talk))
     if key not in _talking_mma_known:
-        _talking_mma_known[key] = bool(_fn("kvf_talking_mma_ok", GATED_LIB)(nh, nkv, d, dv, 1 if decode_form else 0, 1 if talk else 0))
+        _talking_mma_known[key] = bool(_fn("kvf_talking_mma_ok", TALKING_LIB)(nh, nkv, d, dv, 1 if decode_form else 0, 1 if talk else 0))
     return _talking_mma_known[key]
 
 
@@ -1906,7 +1947,7 @@ def talking_attention(
     if talking_mma_supported(q.dtype, nh, nkv, d, dv, scratch is not None, talk is not None) and (scratch is None or split % TALKING_MMA_RANGE_STEP == 0):
         name = "kvf_talking_attention_mma_bf16"  # the two products on the tensor cores; mixing, softmax and sink in float
     _check(
-        _fn(name, GATED_LIB)(
+        _fn(name, TALKING_LIB)(
             _ptr(q), _ptr(out), _ptr(kcache), _ptr(vcache), _ptr(block_tables), _ptr(query_start_loc), _ptr(context_lens), _ptr(talk), _ptr(sink),
             int(num_seqs), int(max_query_len), int(q_stride or q.stride(0)), out.stride(0), block_tables.stride(0), nh, nkv, d, dv, block_size,
             float(scale), int(window), split, max_splits, grid_splits, _ptr(acc), _ptr(ml), _stream(),
@@ -1992,12 +2033,12 @@ def retention(
     x: torch.Tensor, q_off: int, k_off: int, v_off: int, positions: torch.Tensor, inv_freq: torch.Tensor | None, interleaved: bool,
     k_scale: float, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, qsl: torch.Tensor, state_slots: torch.Tensor,
     num_seqs: int, num_heads: int, dk: int, dv: int, scratch: tuple[torch.Tensor, torch.Tensor, torch.Tensor] | None = None,
-    max_query_len: int = 0,
+    max_query_len: int = 0, activation: str | None = None,
 ) -> None:  # fmt: skip
     """Retention over a flat batch, token by token per sequence, on the float state ``S [heads, dk, dv]`` of each
     sequence's slot: ``S <- decay[h] S + k v^T``, ``out = S^T q`` (float ``[N, H*dv]``).  Rows of ``x`` hold the
     projections: ``H`` query heads of ``dk`` from column ``q_off``, key heads from ``k_off``, value heads of ``dv`` from
-    ``v_off``.  The first ``2*len(inv_freq)`` dims of q and k turn with the position (split pairs ``(i, i + rot/2)``
+    ``v_off``; with ``activation="silu"`` all of them pass silu.  The first ``2*len(inv_freq)`` dims of q and k turn with the position (split pairs ``(i, i + rot/2)``
     unless ``interleaved``), then k is multiplied by ``k_scale``; all of that in float.  ``scratch``: float buffers
     ``(qn [N, H*dk], kn [N, H*dk], vn [N, H*dv])``; without it they are allocated here.  ``max_query_len`` (0 = unknown):
     the most rows a sequence of the step brings (a step of single tokens stages less).  Two launches."""
@@ -2005,6 +2046,8 @@ def retention(
     _rows2d(x, None, "x")
     n = x.shape[0]
     h = int(num_heads)
+    if activation not in (None, "silu"):
+        raise ValueError("retention: activation must be None or 'silu'")
     if not 0 < dk <= RETENTION_MAX_KEY_DIM or dv <= 0:
         raise ValueError(f"retention: key heads of 1 to {RETENTION_MAX_KEY_DIM} numbers")
     if max(q_off, k_off) + h * dk > x.shape[1] or v_off + h * dv > x.shape[1]:
@@ -2037,7 +2080,7 @@ def retention(
     _check(
         _fn(name, DECAY_LIB)(
             _ptr(x), x.stride(0), int(q_off), int(k_off), int(v_off), _ptr(positions), _ptr(inv_freq) if rot else None, rot,
-            0 if interleaved else 1, float(k_scale), _ptr(decay), sptr, sstride, _ptr(out), out.stride(0), _ptr(qsl), _ptr(state_slots),
+            0 if interleaved else 1, float(k_scale), 1 if activation == "silu" else 0, _ptr(decay), sptr, sstride, _ptr(out), out.stride(0), _ptr(qsl), _ptr(state_slots),
             int(num_seqs), n, h, int(dk), int(dv), _ptr(qn), _ptr(kn), _ptr(vn), int(max_query_len), _stream(),
         ),
         name,
@@ -2066,3 +2109,185 @@ def retention_gate(o: torch.Tensor, gate: torch.Tensor | None, eps: float, out: 
         gptr, gstride = _ptr(gate), gate.stride(0)
     name = f"kvf_retention_gate_{s}"
     _check(_fn(name, DECAY_LIB)(_ptr(o), o.stride(0), gptr, gstride, float(eps), act, n, num_heads, dv, _ptr(out), out.stride(0), _stream()), name)
+
+
+STATE_SPACE_MAX_STATE = RETENTION_MAX_KEY_DIM  # the same walk
+
+
+def state_space(
+    x: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
+    qsl: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, num_heads: int, groups: int, n_state: int, dv: int,
+    scratch: tuple[torch.Tensor, torch.Tensor, torch.Tensor, torch.Tensor] | None = None, max_query_len: int = 0,
+) -> None:  # fmt: skip
+    """A state space per head whose step size follows the token, over a flat batch, on the float state ``S [heads, n_state,
+    dv]`` of each sequence's slot: ``d = softplus(dt + dt_bias)``, ``S <- exp(-exp(a_log) d) S + B (d x)^T``, ``out = S^T C``
+    (float ``[N, H*dv]``; the term that passes ``x`` on is ``wide_norm_gate``'s).  Rows of ``x`` hold ``x [H*dv] | B
+    [groups*n_state] | C [groups*n_state]`` after their convolution; head ``h`` takes group ``h // (H / groups)``; ``dt``
+    holds rows of ``H`` logits.  ``scratch``: float buffers ``(decay [N, H], cn [N, G*n_state], bn [N, G*n_state], vn
+    [N, H*dv])``; without it they are allocated here.  ``max_query_len`` as in ``retention``.  Two launches."""
+    s = _suffix(x.dtype)
+    _rows2d(x, None, "x")
+    _rows2d(dt, x.dtype, "dt")
+    n, h, g = x.shape[0], int(num_heads), int(groups)
+    if not 0 < n_state <= STATE_SPACE_MAX_STATE or dv <= 0 or g <= 0 or h % g:
+        raise ValueError(f"state_space: states of 1 to {STATE_SPACE_MAX_STATE} numbers, heads a multiple of groups")
+    if x.shape[1] != h * dv + 2 * g * n_state or tuple(dt.shape) != (n, h):
+        raise ValueError("state_space: the columns do not fit the sizes")
+    for t, what in ((dt_bias, "dt_bias"), (a_log, "A_log")):
+        _need(t, torch.float32, what)
+        if t.numel() != h:
+            raise ValueError(f"state_space: one {what} per head")
+    _rows2d(out, torch.float32, "out")
+    if tuple(out.shape) != (n, h * dv):
+        raise ValueError("state_space: out must be float [N, H*dv]")
+    sptr, sstride = _state_view(state, h * n_state * dv, "state")
+    _need(qsl, torch.int32, "query_start_loc")
+    _need(state_slots, torch.int32, "state_slots")
+    if scratch is None:
+        mk = lambda w: torch.empty((n, w), dtype=torch.float32, device=x.device)  # noqa: E731
+        scratch = (mk(h), mk(g * n_state), mk(g * n_state), mk(h * dv))
+    for t, w, what in zip(scratch, (h, g * n_state, g * n_state, h * dv), ("decay", "cn", "bn", "vn")):
+        _need(t, torch.float32, f"scratch {what}")
+        if tuple(t.shape) != (n, w):
+            raise ValueError(f"state_space: scratch {what} must be float [{n}, {w}]")
+    decay, cn, bn, vn = scratch
+    name = f"kvf_state_space_{s}"
+    _check(
+        _fn(name, DECAY_LIB)(
+            _ptr(x), x.stride(0), _ptr(dt), dt.stride(0), _ptr(dt_bias), _ptr(a_log), sptr, sstride, _ptr(out), out.stride(0), _ptr(qsl),
+            _ptr(state_slots), int(num_seqs), n, h, g, int(n_state), int(dv), _ptr(decay), _ptr(cn), _ptr(bn), _ptr(vn), int(max_query_len),
+            _stream(),
+        ),
+        name,
+        2,
+    )  # fmt: skip
+
+
+def wide_norm_gate(
+    o: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, parts: int = 1, gate: torch.Tensor | None = None,
+    activation: str | None = None, gate_first: bool = False, skip: torch.Tensor | None = None, skip_x: torch.Tensor | None = None,
+    mult: float = 1.0,
+) -> None:  # fmt: skip
+    """What follows a recurrence: ``u = o + skip[head] * skip_x`` (``skip`` float, one number per head of equal size, or
+    ``None``), with ``gate_first`` times ``act(gate)``; every one of ``parts`` equal stretches of the row is divided by its own
+    root mean square and multiplied by ``weight`` (float, as wide as the row); without ``gate_first`` times ``act(gate)``;
+    times ``mult``; rounded once.  ``o`` float ``[N, C]``; ``gate``, ``skip_x`` and ``out`` in the storage type (column ranges of
+    wider rows are fine); ``activation``: ``"silu"``, ``"sigmoid"`` or ``None`` (no gate)."""
+    s = _suffix(out.dtype)
+    _rows2d(o, torch.float32, "o")
+    _rows2d(out, None, "out")
+    _need(weight, torch.float32, "norm weight")
+    n, c = o.shape
+    if tuple(out.shape) != (n, c) or weight.numel() != c or parts <= 0 or c % parts:
+        raise ValueError("wide_norm_gate: shapes do not agree")
+    act = {None: 0, "silu": 1, "sigmoid": 2}.get(activation, -1)
+    if act < 0:
+        raise ValueError("wide_norm_gate: activation must be 'silu', 'sigmoid' or None")
+    if act:
+        _rows2d(gate, out.dtype, "gate")
+        if tuple(gate.shape) != (n, c):
+            raise ValueError("wide_norm_gate: gate shape")
+    per_head = 1
+    if skip is not None:
+        _need(skip, torch.float32, "skip")
+        _rows2d(skip_x, out.dtype, "skip_x")
+        if tuple(skip_x.shape) != (n, c) or c % skip.numel():
+            raise ValueError("wide_norm_gate: skip shapes")
+        per_head = c // skip.numel()
+    name = f"kvf_wide_norm_gate_{s}"
+    _check(
+        _fn(name, DECAY_LIB)(
+            _ptr(o), o.stride(0), _ptr(skip), _ptr(skip_x) if skip is not None else None, skip_x.stride(0) if skip is not None else 0, per_head,
+            _ptr(gate) if act else None, gate.stride(0) if act else 0, act, 1 if gate_first else 0, _ptr(weight), float(eps), float(mult), n, c,
+            int(parts), _ptr(out), out.stride(0), _stream(),
+        ),
+        name,
+    )  # fmt: skip
+
+
+# ------------------------------------------------------------------ library "joint"
+# attention whose queries and keys are normed as one vector and whose result is gated, learned positions
+
+JOINT_LIB = "joint"
+
+
+def joint_norm_cache(
+    y: torch.Tensor, parts: Partials | None, bias: torch.Tensor | None, q_weight: torch.Tensor | None, k_weight: torch.Tensor | None,
+    q_count: int, k_count: int, eps: float, slots: torch.Tensor | None, kcache: torch.Tensor | None, vcache: torch.Tensor | None,
+    nh: int, nkv: int, dk: int, dv: int, block_size: int, err: torch.Tensor | None = None,
+) -> None:  # fmt: skip
+    """What follows the input product of an attention layer whose query rows (and key rows) are normed as one vector.
+    Rows hold ``q [nh*dk] | k [nkv*dk] | v [nkv*dv] | rest`` (``nkv == 0``: ``q | rest``): those of ``y`` (storage type), or the sum
+    of the slices ``parts`` (``y`` then receives queries and rest).  ``bias`` (float, as wide as q, k and v together, or ``None``)
+    joins first; then ``q / sqrt(sum(q^2) / q_count + eps) * q_weight`` and the same for k (``q_weight=None``: no norm); queries
+    are written to ``y``, keys and values to ``slots`` of ``kcache [blocks, nkv, block_size, dk]`` / ``vcache [..., dv]``."""
+    s = _suffix(y.dtype)
+    _rows2d(y, None, "y")
+    n = y.shape[0]
+    q_dim, k_dim, v_dim = nh * dk, nkv * dk, nkv * dv
+    width = y.shape[1]
+    if width < q_dim + k_dim + v_dim:
+        raise ValueError("joint_norm_cache: rows too short")
+    pptr, nsplit, stride = None, 0, 0
+    if parts is not None:
+        _need(parts.t, torch.float32, "partials", contiguous=False)
+        if tuple(parts.t.shape[1:]) != (n, width) or parts.t.stride(1) != width or parts.t.stride(2) != 1:
+            raise ValueError("joint_norm_cache: partials must be [S, N, width] with dense rows")
+        pptr, nsplit, stride = _ptr(parts.t), parts.nsplit, parts.split_stride
+    for t, size, what in ((bias, q_dim + k_dim + v_dim, "bias"), (q_weight, q_dim, "query norm weight"), (k_weight, k_dim, "key norm weight")):
+        if t is not None:
+            _need(t, torch.float32, what)
+            if t.numel() != size:
+                raise ValueError(f"joint_norm_cache: the {what} must have {size} entries")
+    if q_weight is not None and nkv and k_weight is None:
+        raise ValueError("joint_norm_cache: queries and keys are normed together or not at all")
+    num_slots = 0
+    if nkv:
+        _need(slots, torch.int32, "slots")
+        _need(kcache, y.dtype, "kcache")
+        _need(vcache, y.dtype, "vcache")
+        if tuple(kcache.shape[1:]) != (nkv, block_size, dk) or tuple(vcache.shape) != (*kcache.shape[:3], dv) or slots.numel() < n:
+            raise ValueError("joint_norm_cache: cache shapes must be [blocks, nkv, block_size, dk] and [..., dv]")
+        num_slots = kcache.shape[0] * block_size
+    name = f"kvf_joint_norm_cache_{s}"
+    _check(
+        _fn(name, JOINT_LIB)(
+            _ptr(y), y.stride(0), pptr, nsplit, stride, width, _ptr(bias), _ptr(q_weight), _ptr(k_weight), int(q_count), int(k_count), float(eps),
+            _ptr(slots) if nkv else None, _ptr(kcache) if nkv else None, _ptr(vcache) if nkv else None, n, nh, nkv, dk, dv, block_size, num_slots,
+            _ptr(err), _stream(),
+        ),
+        name,
+    )  # fmt: skip
+
+
+def output_gate(y: torch.Tensor, gate: torch.Tensor, out: torch.Tensor, nh: int, dv: int, mult: float = 1.0) -> None:
+    """``out = mult * y * sigmoid(gate)`` for rows of ``nh`` heads of ``dv``; ``gate``: as wide as a row (one gate a number) or
+    ``nh`` wide (one a head).  ``out`` may be ``y``; all may be column ranges of wider rows."""
+    s = _suffix(y.dtype)
+    n, c = y.shape
+    for t, what in ((y, "y"), (gate, "gate"), (out, "out")):
+        _rows2d(t, y.dtype, what)
+    if c != nh * dv or tuple(out.shape) != (n, c) or gate.shape[0] != n or gate.shape[1] not in (c, nh):
+        raise ValueError("output_gate: shapes do not agree")
+    name = f"kvf_output_gate_{s}"
+    _check(
+        _fn(name, JOINT_LIB)(
+            _ptr(y), y.stride(0), _ptr(gate), gate.stride(0), 1 if gate.shape[1] == nh and dv != 1 else 0, float(mult), _ptr(out), out.stride(0),
+            n, nh, dv, _stream(),
+        ),
+        name,
+    )  # fmt: skip
+
+
+def add_position_rows(resid: torch.Tensor, table: torch.Tensor, positions: torch.Tensor, err: torch.Tensor | None = None) -> None:
+    """``resid[n, :] += float(table[positions[n], :])``; a position beyond the table raises the device error flag (bit 4)
+    and adds nothing."""
+    s = _suffix(table.dtype)
+    _need(table, None, "position table")
+    _need(resid, torch.float32, "resid")
+    _need(positions, torch.int32, "positions")
+    n, w = resid.shape
+    if table.shape[1] != w or positions.numel() < n:
+        raise ValueError("add_position_rows: shapes do not agree")
+    name = f"kvf_add_position_rows_{s}"
+    _check(_fn(name, JOINT_LIB)(_ptr(resid), _ptr(table), _ptr(positions), n, w, table.shape[0], _ptr(err), _stream()), name)

@@ -74,7 +74,8 @@ def decode_scratch(rt, ctx, nh: int, nkv: int, d: int, dv: int, tickets: torch.T
 class PagedAttention(Mixer):
     """params: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``; optional
     ``position`` (a position-encoding ``PartSpec`` or ``None``), ``window`` (keys a query
-    sees, itself included; ``None`` = all), ``scale`` (default ``1/sqrt(head_dim)``),
+    sees, itself included; ``None`` = all), ``chunk`` (instead of a window: a query sees the keys of its own chunk of
+    so many positions, chunks counted from position 0 of the sequence), ``scale`` (default ``1/sqrt(head_dim)``),
     ``v_head_dim`` (size of a value head, default ``head_dim``) and ``conv`` (taps of a short causal
     convolution over time on every channel of q, k and v, between the projection and the rotation;
     its last ``conv - 1`` inputs are the mixer's state per request; tensors ``q_proj.conv`` ...),
@@ -107,6 +108,9 @@ class PagedAttention(Mixer):
         self.window = params.get("window")
         if self.window is not None and int(self.window) <= 0:
             raise ValueError("window must be positive")
+        self.chunk = params.get("chunk")
+        if self.chunk is not None and (int(self.chunk) <= 0 or self.window is not None):
+            raise ValueError("chunk must be positive, and does not go with a window")
         self.scale = float(params.get("scale") or 1.0 / math.sqrt(self.d))  # model.py:74
         pos = params.get("position")
         if isinstance(pos, dict):
@@ -164,6 +168,8 @@ class PagedAttention(Mixer):
 
     def cache_need(self) -> CacheNeed:
         v = None if self.dv == self.d else self.dv
+        if self.chunk is not None:
+            return CacheNeed("chunk", self.nkv, self.d, int(self.chunk), v)
         if self.window is None:
             return CacheNeed("full", self.nkv, self.d, None, v)
         return CacheNeed("window", self.nkv, self.d, int(self.window), v, keep_first=self.keep_first)
@@ -175,25 +181,15 @@ class PagedAttention(Mixer):
         super().bind(weights, rt)
         self.w_qkv = torch.cat([weights["q_proj.weight"], weights["k_proj.weight"], weights["v_proj.weight"]], dim=0).contiguous()
         self.w_o = weights["o_proj.weight"].contiguous()
-        # counters of finished key ranges per (sequence, kv head) for the decode form: zero between launches
-        self._tickets = torch.zeros(max(1, rt.max_seqs) * self.nkv, dtype=torch.int32, device=rt.device)
-        # the kernel of prompts and mixed batches takes its tiles of queries from a list made with the step
-        self._query_tile = None
         self.w_conv = None
         if self.taps:
             self.w_conv = torch.cat([weights["q_proj.conv"], weights["k_proj.conv"], weights["v_proj.conv"]], dim=0).contiguous()
         self.q_norm_w = weights.get("q_norm.weight") if self.qk_eps is not None else None
         self.k_norm_w = weights.get("k_norm.weight") if self.qk_eps is not None else None
-        self.bias = None
-        if self.bias_shape is not None:
-            self.bias = ops.DistanceBias(weights["rel"].contiguous(), distance_buckets(*self.bias_shape).to(rt.device))
-        self.sinks = weights["sink"].contiguous() if self.has_sink else None
+        bias = ops.DistanceBias(weights["rel"].contiguous(), distance_buckets(*self.bias_shape).to(rt.device)) if self.bias_shape is not None else None
+        sinks = weights["sink"].contiguous() if self.has_sink else None
         self.v_lambda = weights["vmix"].reshape(1).contiguous() if self.value_mix == "mix" else None
-        # kept first keys, a bias on the scores, capped scores and sinks are not the tcgen05 kernel's
-        plain_scores = self.bias is None and not self.keep_first and not self.softcap and self.sinks is None
-        if plain_scores and self.dv == self.d and ops.tcgen05_attention_supported(rt.dtype, self.nh, self.nkv, self.d, False):
-            self._query_tile = ops.tcgen05_query_tile(self.nh, self.nkv)
-            rt.query_tile_sizes.add(self._query_tile)
+        self._bind_attention(bias, sinks)
         if self.position_spec is not None and self.position is None:
             self.position = build_part("position", self.position_spec)
             self.position.bind({}, rt)
@@ -201,7 +197,23 @@ class PagedAttention(Mixer):
         # no table: q and k are stored and used as the projections leave them
         self.inv_freq = table if table is not None else torch.empty(0, dtype=torch.float32, device=rt.device)
         self.interleaved = bool(getattr(self.position, "pairs_interleaved", False))
-        self.general = bool(self.taps) or self.dv != self.d or self.interleaved or self.qk_eps is not None or not plain_scores or self.value_mix is not None
+        self.general = (
+            bool(self.taps) or self.dv != self.d or self.interleaved or self.qk_eps is not None or not self.plain_scores or self.value_mix is not None
+        )
+
+    def _bind_attention(self, bias=None, sinks=None) -> None:
+        """What the attention kernels themselves need, whatever comes before and after them."""
+        rt = self.rt
+        self.bias, self.sinks = bias, sinks
+        # counters of finished key ranges per (sequence, kv head) for the decode form: zero between launches
+        self._tickets = torch.zeros(max(1, rt.max_seqs) * self.nkv, dtype=torch.int32, device=rt.device)
+        # the kernel of prompts and mixed batches takes its tiles of queries from a list made with the step
+        self._query_tile = None
+        # kept first keys, a bias on the scores, capped scores and sinks are not the tcgen05 kernel's
+        self.plain_scores = self.bias is None and not self.keep_first and not self.softcap and self.sinks is None
+        if self.plain_scores and self.dv == self.d and ops.tcgen05_attention_supported(rt.dtype, self.nh, self.nkv, self.d, False):
+            self._query_tile = ops.tcgen05_query_tile(self.nh, self.nkv)
+            rt.query_tile_sizes.add(self._query_tile)
 
     def _scratch(self, ctx):
         rt = self.rt
@@ -287,7 +299,7 @@ class PagedAttention(Mixer):
         scratch, bound, split = None, None, 256
         common = dict(
             window=int(self.window or 0), q_stride=q_stride, err=self.rt.err, dv=self.dv, keep_first=self.keep_first, bias=self.bias,
-            softcap=self.softcap, sinks=self.sinks,
+            softcap=self.softcap, sinks=self.sinks, chunk=int(self.chunk or 0),
         )  # fmt: skip
         args = (q, out, cache.k, cache.v, ctx.block_tables[cache.group], ctx.query_start_loc, ctx.context_lens, ctx.num_seqs)
         shape = (self.nh, self.nkv, self.d, self.scale)

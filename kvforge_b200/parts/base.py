@@ -63,7 +63,8 @@ class WeightDecl:
 @dataclass(frozen=True)
 class CacheNeed:
     """What a mixer keeps per token.  ``kind``: ``full`` (every key), ``window`` (the last
-    ``window`` keys, and for good the first ``keep_first``) or ``none``."""
+    ``window`` keys, and for good the first ``keep_first``), ``chunk`` (the keys of the query's own chunk
+    of ``window`` positions, chunks counted from position 0) or ``none``."""
 
     kind: str
     kv_heads: int = 0
@@ -81,6 +82,12 @@ class CacheNeed:
     @property
     def group_key(self) -> tuple:
         return (self.kind, self.kv_heads, self.head_dim, self.window, self.value_dim, self.keep_first, self.v_in_k)
+
+    def serves(self, other: "CacheNeed") -> bool:
+        """Whether a mixer with the need ``other`` can read a cache kept for this one: keys and values of one shape, and
+        every key that it may see is still there."""
+        same = (self.kv_heads, self.head_dim, self.value_dim, self.v_in_k) == (other.kv_heads, other.head_dim, other.value_dim, other.v_in_k)
+        return same and (self.kind == "full" or self.group_key == other.group_key)
 
 
 @dataclass

@@ -287,3 +287,49 @@ class SandwichBlock(Block):
         finally:
             ctx.residual = keep
         return pending
+
+
+@register_block("postnorm")
+class PostNormBlock(Block):
+    """A norm on each sublayer's result only: ``x = x + norm1(mixer(x)); x = x + norm2(ffn(x))``; the sublayers read the
+    stream itself.  The norm of a result, the residual sum and the stream's copy in the storage type that the next sublayer
+    reads are one kernel (an ``ops.GatedWrite`` without a gate is what the block hands on).
+
+    params: ``norm`` (the ``PartSpec`` of both norms, one that can settle what is pending: ``layernorm``, centred or not),
+    ``mixer``, ``ffn`` (``PartSpec``; ``ffn`` may be ``None``) and the names ``norm1_name``, ``norm2_name`` (the norms' tensors),
+    ``mixer_name``, ``ffn_name`` under the layer's prefix."""
+
+    def __init__(self, params, prefix=""):
+        super().__init__(params, prefix)
+        norm = _spec(params["norm"])
+
+        def named_norm(name):
+            return build_part("norm", PartSpec(norm.kind, {**norm.params, "names": {"weight": name}}), prefix)
+
+        self.norm1 = named_norm(params.get("norm1_name", "norm1"))
+        self.mixer = build_part("mixer", _spec(params["mixer"]), _stem(prefix, params.get("mixer_name", "mix")))
+        self.ffn = self.norm2 = None
+        if params.get("ffn") is not None:
+            self.norm2 = named_norm(params.get("norm2_name", "norm2"))
+            self.ffn = build_part("ffn", _spec(params["ffn"]), _stem(prefix, params.get("ffn_name", "mlp")))
+        if not hasattr(self.norm1, "settle"):
+            raise ValueError("this arrangement needs norms that can settle what is pending")
+
+    def sub_parts(self):
+        return [p for p in (self.norm1, self.mixer, self.norm2, self.ffn) if p is not None]
+
+    def mixer_part(self):
+        return self.mixer
+
+    def forward(self, ctx, resid, delta, cache):
+        keep, ctx.residual = ctx.residual, None  # a result is normed before it joins the stream
+        try:
+            x = self.norm1.rt.buf("block.x", resid.shape[0], resid.shape[1])
+            self.norm1.settle(ctx, resid, delta, x)
+            pending = ops.GatedWrite(self.mixer.forward(ctx, x, cache), post_w=self.norm1.weight)
+            if self.ffn is not None:
+                self.norm1.settle(ctx, resid, pending, x)
+                pending = ops.GatedWrite(self.ffn.forward(ctx, x), post_w=self.norm2.weight)
+        finally:
+            ctx.residual = keep
+        return pending

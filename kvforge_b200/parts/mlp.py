@@ -62,7 +62,8 @@ class GatedMLP(FeedForward):
 
 @register_feed_forward("plain_mlp")
 class PlainMLP(FeedForward):
-    """``down(act(up(x)))`` without biases and without a gate.  params: ``hidden_size``, ``intermediate_size``,
+    """``down(act(up(x)))`` without a gate.  params: ``hidden_size``, ``intermediate_size``, optional ``bias`` (tensors ``up.b``
+    and ``down.b``; the second is handed on with the result as ``ops.Biased``),
     ``activation``: ``"xielu"`` (with the tensor ``act [2]`` = (p, q): ``z > 0: softplus(p) z^2 + z/2``,
     ``z <= 0: (1/2 + softplus(q)) (exp(z) - 1 - z) + z/2``), ``"relu2"`` (the square of relu) or ``"gelu_tanh"``.
     The activation is computed in 32-bit and rounded once.  A block may hand it further rows for its first
@@ -75,6 +76,7 @@ class PlainMLP(FeedForward):
         self.activation = params.get("activation", "relu2")
         if self.activation not in ops.UNARY_ACTIVATIONS:
             raise ValueError(f"activation {self.activation!r} is not one of {sorted(ops.UNARY_ACTIVATIONS)}")
+        self.has_bias = bool(params.get("bias", False))
         self.extra_w = None
         self.extra_out = None
 
@@ -82,6 +84,9 @@ class PlainMLP(FeedForward):
     def weight_decls(cls, params):
         h, i = int(params["hidden_size"]), int(params["intermediate_size"])
         out = {"up": WeightDecl((i, h)), "down": WeightDecl((h, i))}
+        if params.get("bias"):
+            out["up.b"] = WeightDecl((i,), kind="vector", init="zeros")
+            out["down.b"] = WeightDecl((h,), kind="vector", init="zeros")
         if params.get("activation", "relu2") == "xielu":
             out["act"] = WeightDecl((2,), kind="vector", init="small")
         return out
@@ -106,6 +111,8 @@ class PlainMLP(FeedForward):
         self._stack()
         self.w_down = weights["down"].contiguous()
         self.ab = weights["act"].contiguous() if self.activation == "xielu" else None
+        self.b_up = weights["up.b"].contiguous() if self.has_bias else None
+        self.b_down = weights["down.b"].contiguous() if self.has_bias else None
 
     def forward(self, ctx, x: torch.Tensor):
         rt = self.rt
@@ -117,5 +124,6 @@ class PlainMLP(FeedForward):
             ops.linear(x, self.w_up, u)
         self.extra_out = u[:, self.extra_off : self.extra_off + self.extra_w.shape[0]] if self.extra_w is not None else None
         act = rt.buf("pmlp.act", n, self.inter)
-        ops.unary_act(u[:, : self.inter], act, self.activation, self.ab)
-        return project(rt, "pmlp.out", act, self.w_down, ctx)
+        ops.unary_act(u[:, : self.inter], act, self.activation, self.ab, self.b_up)
+        y = project(rt, "pmlp.out", act, self.w_down, None if self.has_bias else ctx)
+        return ops.Biased(y, self.b_down) if self.has_bias else y

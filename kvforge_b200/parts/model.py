@@ -146,7 +146,7 @@ class DecoderModel:
                 src = spec.execution[call.kv_from]
                 a = self.blocks[call.layer].mixer_part().cache_need()
                 b = self.blocks[src.layer].mixer_part().cache_need()
-                if a.group_key != b.group_key:
+                if not b.serves(a):
                     raise ValueError(f"execution[{idx}] reads a cache of another shape than its mixer's")
         self.state_shapes: list[tuple[int, ...] | None] = []
         for call in spec.execution:
@@ -168,10 +168,10 @@ class DecoderModel:
         return out
 
     def _all_parts(self):
-        def walk(part):
-            yield part
+        def walk(part):  # a part made of parts comes after them: what they have bound is there for it to take
             for sub in part.sub_parts():
                 yield from walk(sub)
+            yield part
 
         yield self.embedding
         yield self.head

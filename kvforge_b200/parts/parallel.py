@@ -1,6 +1,7 @@
-"""Mixers side by side: every branch reads the same normed input; each result is RMS-normed over the
+"""Mixers side by side: every branch reads the same input.  ``parallel_mixers``: each result is RMS-normed over the
 model width with a weight of its own (a plain weight, not one-plus), and the mixer's result is the
-mean of the normed results.
+mean of the normed results.  ``summed_mixers``: the mixer's result is the sum of the branches' results, each times a
+constant.
 
 The branches are ordinary mixers.  At most one of them may keep pages of keys and values (the
 block's cache group is that branch's); their per-request states lie side by side in one row of
@@ -9,27 +10,28 @@ floats, and each branch is handed its columns.
 
 from __future__ import annotations
 
+import torch
+
 from .. import ops
 from .base import CacheNeed, Mixer, PartSpec, WeightDecl, build_part, register_mixer
+from .projection import project
 
 
 def _spec(v) -> PartSpec:
     return v if isinstance(v, PartSpec) else PartSpec(v["kind"], v.get("params", {}))
 
 
-@register_mixer("parallel_mixers")
-class ParallelMixers(Mixer):
-    """params: ``hidden_size``, ``eps``, ``branches``: a list of ``(name, PartSpec)``; branch
-    ``name`` has its tensors under ``<prefix><name>.`` and its norm weight is ``<prefix><name>.out``."""
+class _SideBySide(Mixer):
+    """params: ``hidden_size`` and ``branches``, a list whose entries begin with ``(name, PartSpec)``; branch ``name`` has its
+    tensors under ``<prefix><name>.``."""
 
     def __init__(self, params, prefix=""):
         super().__init__(params, prefix)
         self.hidden = int(params["hidden_size"])
-        self.eps = float(params["eps"])
-        self.names = [name for name, _ in params["branches"]]
+        self.names = [entry[0] for entry in params["branches"]]
         if not 0 < len(self.names) <= ops.MAX_BRANCHES:
             raise ValueError(f"between 1 and {ops.MAX_BRANCHES} branches")
-        self.branches: list[Mixer] = [build_part("mixer", _spec(spec), f"{prefix}{name}.") for name, spec in params["branches"]]
+        self.branches: list[Mixer] = [build_part("mixer", _spec(entry[1]), f"{prefix}{entry[0]}.") for entry in params["branches"]]
         paged = [b for b in self.branches if b.cache_need().kind != "none"]
         if len(paged) > 1:
             raise ValueError("only one branch of parallel mixers may keep pages of keys and values")
@@ -47,11 +49,6 @@ class ParallelMixers(Mixer):
             at += shape[0]
         self._state_floats = at
 
-    @classmethod
-    def weight_decls(cls, params):
-        h = int(params["hidden_size"])
-        return {f"{name}.out": WeightDecl((h,), kind="vector", init="ones") for name, _ in params["branches"]}
-
     def sub_parts(self):
         return list(self.branches)
 
@@ -60,6 +57,27 @@ class ParallelMixers(Mixer):
 
     def state_shape(self):
         return (self._state_floats,) if self._state_floats else None
+
+    def branch_view(self, cache, cols):
+        """What a branch is handed of the layer's cache: the pages and its own columns of the state."""
+        if cache is not None and cache.state is not None:
+            return cache.with_state(*cols) if cols else cache.with_state(0, 0)
+        return cache
+
+
+@register_mixer("parallel_mixers")
+class ParallelMixers(_SideBySide):
+    """params: ``hidden_size``, ``eps``, ``branches``: a list of ``(name, PartSpec)``; branch
+    ``name`` has its tensors under ``<prefix><name>.`` and its norm weight is ``<prefix><name>.out``."""
+
+    def __init__(self, params, prefix=""):
+        super().__init__(params, prefix)
+        self.eps = float(params["eps"])
+
+    @classmethod
+    def weight_decls(cls, params):
+        h = int(params["hidden_size"])
+        return {f"{name}.out": WeightDecl((h,), kind="vector", init="ones") for name, _ in params["branches"]}
 
     def bind(self, weights, rt):
         super().bind(weights, rt)
@@ -70,10 +88,7 @@ class ParallelMixers(Mixer):
         try:
             results = []
             for branch, cols in zip(self.branches, self._state_cols):
-                view = cache
-                if cache is not None and cache.state is not None:
-                    view = cache.with_state(*cols) if cols else cache.with_state(0, 0)
-                y = branch.forward(ctx, x, view)
+                y = branch.forward(ctx, x, self.branch_view(cache, cols))
                 t = y.t if isinstance(y, ops.Partials) else y
                 if any(t.data_ptr() == (o.t if isinstance(o, ops.Partials) else o).data_ptr() for o in results):
                     # two branches of one kind hand back the same persistent buffer: keep this one's result apart
@@ -86,3 +101,52 @@ class ParallelMixers(Mixer):
         out = self.rt.buf("parallel.out", x.shape[0], self.hidden)
         ops.branch_norm_mean(results, self.out_w, self.eps, out)
         return out
+
+
+@register_mixer("summed_mixers")
+class SummedMixers(_SideBySide):
+    """``sum_b scale_b * branch_b(x)``.  params: ``hidden_size``, ``branches``: a list of ``(name, PartSpec, scale)``.
+
+    The branches must have the open form (``take_input``, ``mix``, ``take_output``): their input matrices become one product
+    of ``x``, each branch's constant is applied in the kernel that writes what its output projection multiplies (in
+    float, before the one rounding), and the output projections side by side are one product whose sum over the inner
+    width is the sum of the branches."""
+
+    def __init__(self, params, prefix=""):
+        super().__init__(params, prefix)
+        self.scales = [float(entry[2]) for entry in params["branches"]]
+        for b in self.branches:
+            if not all(hasattr(b, name) for name in ("take_input", "mix", "take_output", "inner_width")):
+                raise ValueError(f"{b.kind} has no open form: it cannot be a branch of summed_mixers")
+
+    def bind(self, weights, rt):
+        super().bind(weights, rt)  # the branches are bound already: they hand over their matrices
+        mats = [b.take_input() for b in self.branches]
+        self.in_cols, self.out_cols, at = [], [], 0
+        for m in mats:
+            self.in_cols.append((at, at + m.shape[0]))  # a branch's matrix is a multiple of 8 rows long
+            at += m.shape[0]
+        self.w_in = torch.cat(mats, dim=0).contiguous()
+        outs, at = [], 0
+        for b in self.branches:
+            w = b.take_output()
+            pad = -w.shape[1] % 8  # every branch begins at a multiple of 8 columns
+            outs.append(torch.nn.functional.pad(w, (0, pad)) if pad else w)
+            self.out_cols.append((at, at + w.shape[1]))
+            at += w.shape[1] + pad
+        self.w_o = torch.cat(outs, dim=1).contiguous()
+        self.padded = any(hi % 8 for _, hi in self.out_cols)
+
+    def forward(self, ctx, x, cache):
+        rt, n = self.rt, x.shape[0]
+        y = rt.buf("summed.in", n, self.w_in.shape[0])
+        if ops.skinny_ok(x, self.w_in):
+            ops.gemm_skinny(x, self.w_in, y)
+        else:
+            ops.linear(x, self.w_in, y)
+        inner = rt.buf("summed.inner", n, self.w_o.shape[1])
+        if self.padded:
+            inner.zero_()  # columns between the branches meet zero weights, and must be numbers
+        for branch, cols, (lo, hi), (a, b), scale in zip(self.branches, self._state_cols, self.in_cols, self.out_cols, self.scales):
+            branch.mix(ctx, y[:, lo:hi], self.branch_view(cache, cols), inner[:, a:b], scale)
+        return project(rt, "summed.proj", inner, self.w_o, ctx)

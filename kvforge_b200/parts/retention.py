@@ -1,10 +1,12 @@
-"""Retention: linear attention with one fixed decay a head, no softmax and no denominator.
+"""Retention: linear attention with one fixed decay a head, no softmax and no denominator (with silu on the projections
+and one norm over all heads it is what is called lightning attention).
 
 Per layer ``q = W_q x``, ``k = W_k x`` (``H`` heads of ``head_dim``), ``v = W_v x`` (``H`` heads of ``v_head_dim``),
 ``g = W_g x``.  The first ``rotary_dim`` dims of every query and key head turn with the position; the keys are then
 multiplied by ``head_dim^(-1/2)``.  Per head a matrix state ``S [head_dim, v_head_dim]`` is carried from token to
 token, ``S_t = a_h S_(t-1) + k_t v_t^T``, and read out as ``o_t = S_t^T q_t``.  Every head's ``o`` is divided by its
-root mean square, the heads are multiplied by ``silu(g)`` and projected back.  The state is the mixer's state slot
+root mean square (or all heads together are normed with a weight), the heads are multiplied by ``silu(g)`` (or the
+logistic function of ``g``) and projected back.  The state is the mixer's state slot
 per request: 32-bit floats, zero for a new request; the mixer keeps no pages.
 """
 
@@ -14,6 +16,7 @@ import torch
 
 from .. import ops
 from .base import CacheNeed, Mixer, PartSpec, WeightDecl, build_part, register_mixer
+from .gated_attention import stack_rows
 from .projection import project
 
 
@@ -21,10 +24,15 @@ from .projection import project
 class Retention(Mixer):
     """params: ``hidden_size``, ``num_heads``, ``head_dim``, ``v_head_dim``, ``decay`` (a list of ``num_heads`` numbers),
     ``eps`` (of the heads' norm); optional ``position`` (a rotary ``PartSpec`` or ``None``), ``key_scale`` (default
-    ``head_dim^(-1/2)``) and ``gate`` (``"silu"``, ``"sigmoid"`` or ``None``; default ``"silu"``).
+    ``head_dim^(-1/2)``), ``gate`` (``"silu"``, ``"sigmoid"`` or ``None``; default ``"silu"``), ``activation`` (``"silu"``: q, k and v
+    pass it right after their projections) and ``norm`` (``"heads"``, the default: every head by itself, without a weight;
+    ``"joint"``: the concatenated heads together, with the tensor ``norm [H*v_head_dim]``).
 
     Tensors: ``q [H*head_dim, W]``, ``k [H*head_dim, W]``, ``v [H*v_head_dim, W]``, ``g [H*v_head_dim, W]`` (with a gate),
-    ``o [W, H*v_head_dim]``."""
+    ``o [W, H*v_head_dim]``.
+
+    With the joint norm it also has the open form that ``summed_mixers`` takes: ``take_input`` / ``take_output`` hand the input
+    and output matrices over, and ``mix`` computes what lies between the two products."""
 
     def __init__(self, params, prefix=""):
         super().__init__(params, prefix)
@@ -41,15 +49,17 @@ class Retention(Mixer):
         self.gate = p.get("gate", "silu")
         if self.gate not in ("silu", "sigmoid", None):
             raise ValueError("the gate of retention is 'silu', 'sigmoid' or None")
+        self.activation = p.get("activation")
+        if self.activation not in ("silu", None):
+            raise ValueError("the activation of retention's projections is 'silu' or None")
+        self.norm = p.get("norm", "heads")
+        if self.norm not in ("heads", "joint"):
+            raise ValueError("the norm of retention is 'heads' or 'joint'")
         pos = p.get("position")
         if isinstance(pos, dict):
             pos = PartSpec(pos["kind"], pos.get("params", {}))
         self.position_spec: PartSpec | None = pos
         self.position = None
-        self.k_off = self.nh * self.dk
-        self.v_off = 2 * self.nh * self.dk
-        self.g_off = self.v_off + self.nh * self.dv
-        self.in_dim = -(-(self.g_off + (self.nh * self.dv if self.gate else 0)) // 8) * 8
 
     @classmethod
     def weight_decls(cls, params):
@@ -57,6 +67,8 @@ class Retention(Mixer):
         out = {"q": WeightDecl((h * dk, w)), "k": WeightDecl((h * dk, w)), "v": WeightDecl((h * dv, w)), "o": WeightDecl((w, h * dv))}
         if params.get("gate", "silu") is not None:
             out["g"] = WeightDecl((h * dv, w))
+        if params.get("norm", "heads") == "joint":
+            out["norm"] = WeightDecl((h * dv,), kind="vector", init="ones")
         return out
 
     def cache_need(self) -> CacheNeed:
@@ -68,10 +80,12 @@ class Retention(Mixer):
     def bind(self, weights, rt):
         super().bind(weights, rt)
         mats = [weights["q"], weights["k"], weights["v"]] + ([weights["g"]] if self.gate else [])
-        rows = sum(t.shape[0] for t in mats)
-        if rows < self.in_dim:  # rows of zeros up to a multiple of 8: the products want aligned widths
-            mats.append(torch.zeros((self.in_dim - rows, self.hidden), dtype=mats[0].dtype, device=mats[0].device))
-        self.w_in = torch.cat(mats, dim=0).contiguous()
+        # each projection from a multiple of 8 columns of the product on
+        self.w_in, offs = stack_rows(mats)
+        self.in_dim = self.w_in.shape[0]
+        self.k_off, self.v_off = offs[1], offs[2]
+        self.g_off = offs[3] if self.gate else None
+        self.norm_w = weights["norm"].contiguous() if self.norm == "joint" else None
         self.w_o = weights["o"].contiguous()
         self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=rt.device)
         if self.position_spec is not None and self.position is None:
@@ -80,17 +94,24 @@ class Retention(Mixer):
         self.inv_freq = self.position.table() if self.position is not None else None
         self.interleaved = bool(getattr(self.position, "pairs_interleaved", False))
 
-    def forward(self, ctx, x: torch.Tensor, cache):
-        rt = self.rt
-        n = x.shape[0]
+    # ------------------------------------------------------------------ between the two products
+    inner_width = property(lambda self: self.nh * self.dv)
+
+    def take_input(self) -> torch.Tensor:
+        w, self.w_in = self.w_in, None
+        return w
+
+    def take_output(self) -> torch.Tensor:
+        w, self.w_o = self.w_o, None
+        return w
+
+    def mix(self, ctx, y: torch.Tensor, cache, out: torch.Tensor, mult: float = 1.0) -> None:
+        """``y [N, in_dim]``: the input product's rows; ``out [N, inner_width]`` gets ``mult`` times what the output
+        projection multiplies."""
+        rt, n = self.rt, y.shape[0]
         if cache is None or cache.state is None:
             raise RuntimeError("retention needs its state slots")
         h, dk, dv = self.nh, self.dk, self.dv
-        y = rt.buf("retention.in", n, self.in_dim)
-        if ops.skinny_ok(x, self.w_in):
-            ops.gemm_skinny(x, self.w_in, y)
-        else:
-            ops.linear(x, self.w_in, y)
         o = rt.buf("retention.o", n, h * dv, torch.float32)
         scratch = (
             rt.buf("retention.qn", n, h * dk, torch.float32),
@@ -99,9 +120,23 @@ class Retention(Mixer):
         )
         ops.retention(
             y, 0, self.k_off, self.v_off, ctx.positions, self.inv_freq, self.interleaved, self.key_scale, self.decay, cache.state, o,
-            ctx.query_start_loc, ctx.state_slots, ctx.num_seqs, h, dk, dv, scratch, max_query_len=ctx.max_query_len,
+            ctx.query_start_loc, ctx.state_slots, ctx.num_seqs, h, dk, dv, scratch, max_query_len=ctx.max_query_len, activation=self.activation,
         )  # fmt: skip
-        out = rt.buf("retention.out", n, h * dv)
         gate = y[:, self.g_off : self.g_off + h * dv] if self.gate else None
-        ops.retention_gate(o, gate, self.eps, out, h, dv, self.gate)
+        if self.norm == "joint":
+            ops.wide_norm_gate(o, self.norm_w, self.eps, out, gate=gate, activation=self.gate, mult=mult)
+        elif mult == 1.0:
+            ops.retention_gate(o, gate, self.eps, out, h, dv, self.gate)
+        else:
+            raise RuntimeError("retention with heads normed one by one is not scaled")
+
+    def forward(self, ctx, x: torch.Tensor, cache):
+        rt, n = self.rt, x.shape[0]
+        y = rt.buf("retention.in", n, self.in_dim)
+        if ops.skinny_ok(x, self.w_in):
+            ops.gemm_skinny(x, self.w_in, y)
+        else:
+            ops.linear(x, self.w_in, y)
+        out = rt.buf("retention.out", n, self.inner_width)
+        self.mix(ctx, y, cache, out)
         return project(rt, "retention.proj", out, self.w_o, ctx)

@@ -16,7 +16,8 @@ import math
 
 import torch
 
-from .base import PositionEncoding, register_position_encoding
+from .. import ops
+from .base import PositionEncoding, WeightDecl, register_position_encoding
 
 
 def rotary_inv_freq(rotary_dim: int, theta: float) -> torch.Tensor:
@@ -70,3 +71,24 @@ class RotaryEmbedding(PositionEncoding):
 
     def table(self) -> torch.Tensor:
         return self.inv_freq
+
+
+@register_position_encoding("learned")
+class LearnedPositions(PositionEncoding):
+    """A learned vector per position, added to the residual stream after the embedding lookup.  params: ``rows`` (positions
+    there are; a later one raises the device error flag), ``hidden_size``.  Tensor: ``weight [rows, hidden_size]``."""
+
+    def __init__(self, params, prefix=""):
+        super().__init__(params, prefix)
+        self.rows, self.hidden = int(params["rows"]), int(params["hidden_size"])
+
+    @classmethod
+    def weight_decls(cls, params):
+        return {"weight": WeightDecl((int(params["rows"]), int(params["hidden_size"])))}
+
+    def bind(self, weights, rt):
+        super().bind(weights, rt)
+        self.weight = weights["weight"].contiguous()
+
+    def embed(self, ctx, resid):
+        ops.add_position_rows(resid, self.weight, ctx.positions, self.rt.err)
