@@ -43,7 +43,7 @@ def parse_args(argv=None):
     ap.add_argument("--dtype", required=True, choices=["bfloat16", "float32"])
     ap.add_argument("--out", required=True, help="folder for the <step>.f32 files")
     ap.add_argument("--max-tokens", type=int, required=True, help="most tokens live requests hold at any time")
-    ap.add_argument("--max-live", type=int, default=16, help="most requests live at a time")
+    ap.add_argument("--max-live", type=int, default=4, help="most requests live at a time")
     ap.add_argument("--block-size", type=int, default=PAGE, help="tokens per page of the cache")
     ap.add_argument("--num-blocks", type=int, default=None, help="pages of the pool (default: what --max-tokens needs)")
     ap.add_argument("--cuda-graphs", action="store_true", help="replay steps as captured CUDA graphs, as generation does")
