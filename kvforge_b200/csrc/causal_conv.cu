@@ -7,7 +7,7 @@ using namespace kvf;
 namespace {
 
 // ---------------------------------------------------------------- short causal convolution
-// y[n, c] = act( b[c] + sum_j w[c, j] * u[t - (taps-1) + j, c] ), t the place of row n in its sequence; places
+// y[n, c] = act( b[c] + sum_j w[j, c] * u[t - (taps-1) + j, c] ), t the place of row n in its sequence; places
 // before this step's first row come from the state (the last taps-1 inputs of the sequence, oldest
 // first, [taps-1][C] floats), which is zero before a sequence's start.  `bias` (b) may be null.
 template <typename T, int VEC> struct VecIO;
@@ -33,6 +33,21 @@ template <typename T> struct VecIO<T, 1> {
   static __device__ __forceinline__ void store(T* p, const float* f) { p[0] = from_float<T>(f[0]); }
 };
 
+// VEC neighbouring floats (whole 16-byte loads when VEC is a multiple of four), zeros from null
+template <int VEC>
+__device__ __forceinline__ void load_floats(const float* p, float* f) {
+  if constexpr (VEC % 4 == 0) {
+#pragma unroll
+    for (int e = 0; e < VEC; e += 4) {
+      const float4 v = p ? *reinterpret_cast<const float4*>(p + e) : make_float4(0.f, 0.f, 0.f, 0.f);
+      f[e] = v.x; f[e + 1] = v.y; f[e + 2] = v.z; f[e + 3] = v.w;
+    }
+  } else {
+#pragma unroll
+    for (int e = 0; e < VEC; ++e) f[e] = p ? p[e] : 0.f;
+  }
+}
+
 // A thread owns VEC neighbouring channels (one 16-byte load) of `rows` consecutive token rows; TAPS > 0: the
 // taps are known at compile time and a thread keeps its weights in registers.  Each output is one chain of
 // fused multiply-adds over the taps, oldest first, whichever form runs.
@@ -51,14 +66,16 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const T* __restrict__ 
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
   if (c >= C) return;
   float cb[VEC];
-#pragma unroll
-  for (int e = 0; e < VEC; ++e) cb[e] = bias ? bias[c + e] : 0.f;
+  load_floats<VEC>(bias ? bias + c : nullptr, cb);
   float wr[VEC][TAPS > 0 ? TAPS : 1];
   if (TAPS > 0) {
 #pragma unroll
-    for (int e = 0; e < VEC; ++e)
+    for (int j = 0; j < TAPS; ++j) {
+      float t[VEC];
+      load_floats<VEC>(w + (size_t)j * C + c, t);
 #pragma unroll
-      for (int j = 0; j < TAPS; ++j) wr[e][j] = w[(size_t)(c + e) * TAPS + j];
+      for (int e = 0; e < VEC; ++e) wr[e][j] = t[e];
+    }
   }
   if (TAPS > 0 && rows == CONV_ROWS) {
     // all of the tile's rows in one sequence: its rows + taps - 1 inputs are loaded once, together, and every row's
@@ -122,7 +139,7 @@ __global__ void __launch_bounds__(128) causal_conv_kernel(const T* __restrict__ 
         for (int e = 0; e < VEC; ++e) u[e] = st ? st[(size_t)(taps - 1 + src) * C + c + e] : 0.f;
       }
 #pragma unroll
-      for (int e = 0; e < VEC; ++e) acc[e] = fmaf(TAPS > 0 ? wr[e][TAPS > 0 ? j : 0] : w[(size_t)(c + e) * taps + j], u[e], acc[e]);
+      for (int e = 0; e < VEC; ++e) acc[e] = fmaf(TAPS > 0 ? wr[e][TAPS > 0 ? j : 0] : w[(size_t)j * C + c + e], u[e], acc[e]);
     }
     if (act == 1) {
 #pragma unroll
@@ -151,12 +168,14 @@ __global__ void __launch_bounds__(128) causal_conv_few_kernel(const T* __restric
   if (c >= C || q_len <= 0 || q_len > CONV_FEW) return;
   float* st = slot >= 0 ? state + (size_t)slot * state_stride : nullptr;
   float wr[VEC][TAPS], cb[VEC];
+  load_floats<VEC>(bias ? bias + c : nullptr, cb);
 #pragma unroll
-  for (int e = 0; e < VEC; ++e) cb[e] = bias ? bias[c + e] : 0.f;
+  for (int j = 0; j < TAPS; ++j) {
+    float t[VEC];
+    load_floats<VEC>(w + (size_t)j * C + c, t);
 #pragma unroll
-  for (int e = 0; e < VEC; ++e)
-#pragma unroll
-    for (int j = 0; j < TAPS; ++j) wr[e][j] = w[(size_t)(c + e) * TAPS + j];
+    for (int e = 0; e < VEC; ++e) wr[e][j] = t[e];
+  }
   float u[TAPS - 1 + CONV_FEW][VEC];  // the state's inputs, then this step's rows
 #pragma unroll
   for (int i = 0; i < TAPS - 1; ++i)
@@ -263,7 +282,7 @@ __global__ void __launch_bounds__(256) conv_state_kernel(const T* __restrict__ x
     if (taps <= 0 || (unsigned)B > 65535u) return (int)cudaErrorInvalidValue;                                          \
     constexpr int V = ConvVec<T>::N;                                                                                   \
     const bool vec = C % V == 0 && x_stride % V == 0 && out_stride % V == 0 && ((uintptr_t)x % 16) == 0 &&             \
-                     ((uintptr_t)out % 16) == 0;                                                                       \
+                     ((uintptr_t)out % 16) == 0 && ((uintptr_t)w % 16) == 0 && ((uintptr_t)bias % 16) == 0;            \
     if (max_q_len > 0 && max_q_len <= CONV_FEW && taps >= 2 && taps <= 4) {                                            \
       return vec ? launch_conv_few<T, V>((const T*)x, x_stride, w, bias, state, state_stride, qsl, state_slots, B, C, taps,  \
                                          act, (T*)out, out_stride, st)                                                 \

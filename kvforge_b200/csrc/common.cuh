@@ -114,6 +114,13 @@ __device__ __forceinline__ void bf16x8_to_float(const uint4& u, float* f) {
   }
 }
 
+// 0.5 z (1 + tanh(u)) with u = sqrt(2/pi) (z + 0.044715 z^3), as z / (1 + exp(-2 u)): for results that are rounded to
+// bfloat16 right after (the fast exponential and division are a few units in the last place of a float off).
+__device__ __forceinline__ float gelu_tanh_fast(float z) {
+  const float u2 = 1.5957691216057308f * fmaf(0.044715f * z * z, z, z);
+  return __fdividef(z, 1.f + __expf(-u2));
+}
+
 // One pair of a rotary encoding: (x1, x2) turned by the angle whose cosine and sine are given.
 // The roundings are spelled out (a product, then a fused multiply-add) so that every kernel
 // that rotates gives the same bits, whichever of them a step's token count selects.

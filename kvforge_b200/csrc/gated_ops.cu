@@ -106,8 +106,8 @@ __global__ void __launch_bounds__(256) norm_step_kernel(const NormStepParams p) 
   }
 }
 
-// The same pass for rows of up to 4 * 256 * NIT numbers whose rows start on 16-byte boundaries: a thread owns
-// four neighbouring numbers of each of up to NIT quarters of the row and keeps them in registers; everything a
+// The same pass for rows of up to 4 * TH * NIT numbers whose rows start on 16-byte boundaries: a thread (of TH) owns
+// four neighbouring numbers of each of up to NIT stretches of the row and keeps them in registers; everything a
 // row needs from memory is asked for before the first number is used.  The sums run in the same order whatever
 // else is in the batch.
 template <typename T> struct Vec4;
@@ -159,8 +159,8 @@ __device__ __forceinline__ void reg_stats(const float (&x)[NIT][4], const bool (
   rstd = 1.f / sqrtf(block_sum(q, red) / (float)W + eps);
 }
 
-template <typename T, int NIT>
-__global__ void __launch_bounds__(256) norm_step_vec_kernel(const NormStepParams p) {
+template <typename T, int NIT, int TH>
+__global__ void __launch_bounds__(TH) norm_step_vec_kernel(const NormStepParams p) {
   pdl_launch();
   pdl_wait();
   __shared__ float red[32];
@@ -176,7 +176,7 @@ __global__ void __launch_bounds__(256) norm_step_vec_kernel(const NormStepParams
   float hv[NIT][4], a[NIT][4], g[NIT][4], pw[NIT][4], nw[NIT][4];
 #pragma unroll
   for (int it = 0; it < NIT; ++it) {
-    const int i = (it * 256 + threadIdx.x) * 4;
+    const int i = (it * TH + threadIdx.x) * 4;
     live[it] = i < W;
 #pragma unroll
     for (int e = 0; e < 4; ++e) hv[it][e] = a[it][e] = g[it][e] = 0.f, pw[it][e] = nw[it][e] = 1.f;
@@ -197,15 +197,24 @@ __global__ void __launch_bounds__(256) norm_step_vec_kernel(const NormStepParams
     if (p.post_w) Vec4<float>::load(p.post_w + i, pw[it]);
   }
   if (yp) {
-    for (int s = 0; s < p.nsplit; ++s) {
+    // a few slices' loads in flight at a time, added in slice order
+    constexpr int SL = NIT == 1 ? (TH <= 512 ? 10 : 5) : NIT == 2 ? 5 : 2;
+    for (int s0 = 0; s0 < p.nsplit; s0 += SL) {
+      float t[SL][NIT][4];
 #pragma unroll
-      for (int it = 0; it < NIT; ++it) {
-        if (!live[it]) continue;
-        float t[4];
-        Vec4<float>::load(yp + (size_t)s * p.split_stride + (it * 256 + threadIdx.x) * 4, t);
+      for (int k = 0; k < SL; ++k)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) a[it][e] += t[e];
-      }
+        for (int it = 0; it < NIT; ++it) {
+          // no branch around a load: past the last slice it is read once more, past the row's end its start, and neither is used
+          const int s = min(s0 + k, p.nsplit - 1), i = live[it] ? (it * TH + threadIdx.x) * 4 : 0;
+          Vec4<float>::load(yp + (size_t)s * p.split_stride + i, t[k][it]);
+        }
+#pragma unroll
+      for (int k = 0; k < SL; ++k)
+#pragma unroll
+        for (int it = 0; it < NIT; ++it)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) a[it][e] += live[it] && s0 + k < p.nsplit ? t[k][it][e] : 0.f;
     }
   }
   if (pending) {
@@ -214,7 +223,7 @@ __global__ void __launch_bounds__(256) norm_step_vec_kernel(const NormStepParams
       for (int it = 0; it < NIT; ++it) {
         if (!live[it]) continue;
         float t[4];
-        Vec4<float>::load(p.y_bias + (it * 256 + threadIdx.x) * 4, t);
+        Vec4<float>::load(p.y_bias + (it * TH + threadIdx.x) * 4, t);
 #pragma unroll
         for (int e = 0; e < 4; ++e) a[it][e] += t[e];
       }
@@ -231,7 +240,7 @@ __global__ void __launch_bounds__(256) norm_step_vec_kernel(const NormStepParams
     for (int it = 0; it < NIT; ++it) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) hv[it][e] += p.post_w ? (a[it][e] - mean) * rstd * pw[it][e] : a[it][e];
-      if (live[it] && !p.rows && !p.store_normed) Vec4<float>::store(h + (it * 256 + threadIdx.x) * 4, hv[it]);
+      if (live[it] && !p.rows && !p.store_normed) Vec4<float>::store(h + (it * TH + threadIdx.x) * 4, hv[it]);
     }
   }
   if (!p.out && !p.store_normed) return;
@@ -241,7 +250,7 @@ __global__ void __launch_bounds__(256) norm_step_vec_kernel(const NormStepParams
 #pragma unroll
   for (int it = 0; it < NIT; ++it) {
     if (!live[it]) continue;
-    const int i = (it * 256 + threadIdx.x) * 4;
+    const int i = (it * TH + threadIdx.x) * 4;
     float x[4];
 #pragma unroll
     for (int e = 0; e < 4; ++e) x[e] = p.next_w ? (hv[it][e] - mean) * rstd * nw[it][e] : hv[it][e];
@@ -353,7 +362,7 @@ __device__ __forceinline__ float unary_act(float z, int kind, float ap, float aq
   return 0.5f * z * (1.f + tanhf(0.7978845608028654f * (z + 0.044715f * z * z * z)));
 }
 
-template <typename T>
+template <typename T, int V>
 __global__ void __launch_bounds__(256) unary_act_kernel(const T* __restrict__ in, long long in_stride, T* __restrict__ out,
                                                          long long out_stride, long long rows, int cols, int kind,
                                                          const float* __restrict__ ab, const float* __restrict__ bias) {
@@ -364,18 +373,22 @@ __global__ void __launch_bounds__(256) unary_act_kernel(const T* __restrict__ in
     ap = softplus_f(ab[0]);
     aq = 0.5f + softplus_f(ab[1]);
   }
-  const long long total = rows * cols;
-  for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < total; idx += (long long)gridDim.x * blockDim.x) {
-    const long long r = idx / cols;
-    const int c = (int)(idx - r * cols);
-    out[r * out_stride + c] = from_float<T>(unary_act(to_float<T>(in[r * in_stride + c]) + (bias ? bias[c] : 0.f), kind, ap, aq));
+  const long long r = blockIdx.x;
+  for (int c = (blockIdx.y * blockDim.x + threadIdx.x) * V; c < cols; c += gridDim.y * blockDim.x * V) {
+    float z[V];
+    if constexpr (V == 4) {
+      Vec4<T>::load(in + r * in_stride + c, z);
+    } else {
+      z[0] = to_float<T>(in[r * in_stride + c]);
+    }
+#pragma unroll
+    for (int e = 0; e < V; ++e) z[e] = unary_act(z[e] + (bias ? bias[c + e] : 0.f), kind, ap, aq);
+    if constexpr (V == 4) {
+      Vec4<T>::store(out + r * out_stride + c, z);
+    } else {
+      out[r * out_stride + c] = from_float<T>(z[0]);
+    }
   }
-}
-
-unsigned grid_for(long long total) {
-  long long g = (total + 255) / 256;
-  if (g > 148 * 16) g = 148 * 16;
-  return (unsigned)(g < 1 ? 1 : g);
 }
 
 }  // namespace
@@ -398,9 +411,13 @@ KVF_API int kvf_gated_set_pdl(int enabled) {
     p.nsplit = nsplit; p.z = z; p.z_stride = z_stride; p.z_bias = z_bias; p.y_bias = y_bias; p.post_w = post_w; p.next_w = next_w;       \
     p.out = out; p.out_stride = out_stride; p.W = W; p.centred = centred; p.store_normed = store_normed; p.eps = eps; \
     if (norm_step_vec_ok<T>(p)) {                                                                                     \
-      if (W <= 1024) return launch(norm_step_vec_kernel<T, 1>, dim3(n_rows), dim3(256), 0, st, p);                    \
-      if (W <= 2048) return launch(norm_step_vec_kernel<T, 2>, dim3(n_rows), dim3(256), 0, st, p);                    \
-      return launch(norm_step_vec_kernel<T, 4>, dim3(n_rows), dim3(256), 0, st, p);                                   \
+      /* few rows of slices in bfloat16: a thread for every four numbers, so that all slices of a row are asked for at once */ \
+      const bool few = sizeof(T) == 2 && y_parts && n_rows <= 148;                                                    \
+      if (W <= 1024) return launch(norm_step_vec_kernel<T, 1, 256>, dim3(n_rows), dim3(256), 0, st, p);               \
+      if (W <= 2048) return few ? launch(norm_step_vec_kernel<T, 1, 512>, dim3(n_rows), dim3(512), 0, st, p)          \
+                                : launch(norm_step_vec_kernel<T, 2, 256>, dim3(n_rows), dim3(256), 0, st, p);         \
+      return few ? launch(norm_step_vec_kernel<T, 1, 1024>, dim3(n_rows), dim3(1024), 0, st, p)                       \
+                 : launch(norm_step_vec_kernel<T, 4, 256>, dim3(n_rows), dim3(256), 0, st, p);                        \
     }                                                                                                                 \
     const size_t smem = (size_t)2 * W * sizeof(float);                                                                \
     auto kern = norm_step_kernel<T>;                                                                                  \
@@ -427,8 +444,13 @@ KVF_API int kvf_gated_set_pdl(int enabled) {
                                   int cols, int kind, const float* ab, const float* bias, cudaStream_t st) {          \
     if (rows <= 0 || cols <= 0) return 0;                                                                             \
     if (kind < 0 || kind > 2 || (kind == 0 && !ab)) return (int)cudaErrorInvalidValue;                                \
-    return launch(unary_act_kernel<T>, dim3(grid_for(rows * cols)), dim3(256), 0, st, (const T*)in, in_stride, (T*)out, \
-                  out_stride, rows, cols, kind, ab, bias);                                                                  \
+    constexpr size_t TB = 4 * sizeof(T);                                                                              \
+    const bool vec = cols % 4 == 0 && in_stride % 4 == 0 && out_stride % 4 == 0 && ((uintptr_t)in % TB) == 0 && ((uintptr_t)out % TB) == 0; \
+    const int per = 256 * (vec ? 4 : 1);                                                                              \
+    if (rows > 0x7fffffffLL) return (int)cudaErrorInvalidValue;                                                       \
+    dim3 grid((unsigned)rows, (cols + per - 1) / per < 65535 ? (cols + per - 1) / per : 65535);                       \
+    return launch(vec ? unary_act_kernel<T, 4> : unary_act_kernel<T, 1>, grid, dim3(256), 0, st, (const T*)in, in_stride, (T*)out, \
+                  out_stride, rows, cols, kind, ab, bias);                                                            \
   }
 
 KVF_GATED_API(f32, float)

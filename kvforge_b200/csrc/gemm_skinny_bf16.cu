@@ -14,6 +14,7 @@
 //   3  bfloat16 act[M, N/2] = silu(g) * u     W holds gate and up rows interleaved in blocks
 //                                             of 8 ([g0..7, u0..7, g8..15, ...]), so a thread
 //                                             finds g_i and u_i in its own accumulators
+//   4  bfloat16 y[M, N] = gelu_tanh(x W^T + bias)   bias float [N] or null
 // Any N; K a multiple of 8; rows and chunks past the edges are zero-filled.
 #include "common.cuh"
 
@@ -34,6 +35,7 @@ struct SkinnyParams {
   int k_per_split;  // multiple of BK
   int mode;
   long long split_stride;  // elements between partial slices
+  const float* bias;
 };
 
 __device__ __forceinline__ uint32_t s_u32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -162,7 +164,9 @@ __global__ void __launch_bounds__(THREADS) gemm_skinny_kernel(const SkinnyParams
           const int f = f0 + 8 * h;
           if (f >= p.N) continue;
           const float v = acc[j][2 * h + e];
-          if (p.mode == 0)
+          if (p.mode == 4)
+            reinterpret_cast<bf16*>(p.out)[(size_t)t * p.ldo + f] = __float2bfloat16_rn(gelu_tanh_fast(v + (p.bias ? p.bias[f] : 0.f)));
+          else if (p.mode == 0)
             reinterpret_cast<bf16*>(p.out)[(size_t)t * p.ldo + f] = __float2bfloat16_rn(v);
           else
             reinterpret_cast<float*>(p.out)[(size_t)blockIdx.y * p.split_stride + (size_t)t * p.ldo + f] = v;
@@ -190,9 +194,9 @@ int launch_skinny(const SkinnyParams& p, int ksplit, cudaStream_t st) {
 // mode as at the top of this file; ldo = row stride of the output in elements; for mode 2
 // `ksplit` slices of K are written split_stride elements apart.  M <= 64, K % 8 == 0.
 KVF_API int kvf_gemm_skinny_bf16(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int ldw,
-                                 int ldo, int mode, int ksplit, long long split_stride, cudaStream_t st) {
+                                 int ldo, int mode, int ksplit, long long split_stride, const float* bias, cudaStream_t st) {
   if (M <= 0 || N <= 0) return 0;
-  if (M > 64 || K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || mode < 0 || mode > 3 || ksplit < 1)
+  if (M > 64 || K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || mode < 0 || mode > 4 || ksplit < 1)
     return (int)cudaErrorInvalidValue;
   if ((((uintptr_t)x) & 15) || (((uintptr_t)w) & 15)) return (int)cudaErrorInvalidValue;
   if (mode != 2 && ksplit != 1) return (int)cudaErrorInvalidValue;
@@ -200,7 +204,7 @@ KVF_API int kvf_gemm_skinny_bf16(const void* x, const void* w, void* out, int M,
   SkinnyParams p;
   p.x = (const bf16*)x; p.w = (const bf16*)w; p.out = out;
   p.M = M; p.N = N; p.K = K; p.ldx = ldx; p.ldw = ldw; p.ldo = ldo;
-  p.mode = mode; p.split_stride = split_stride;
+  p.mode = mode; p.split_stride = split_stride; p.bias = bias;
   const int k_iters = (K + BK - 1) / BK;
   p.k_per_split = ((k_iters + ksplit - 1) / ksplit) * BK;
   if ((long long)(ksplit - 1) * p.k_per_split >= K) return (int)cudaErrorInvalidValue;  // an empty slice

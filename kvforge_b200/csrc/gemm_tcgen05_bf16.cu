@@ -14,7 +14,7 @@
 //            ready" mbarrier;
 //   warps 2-5  wait for the accumulator, read it with tcgen05.ld (each warp its quarter of the
 //            128 rows, 32 columns at a time), apply the epilogue and store.
-// Epilogues: bfloat16 y; or act[M, N/2] = silu(g) * u for W with gate and up rows interleaved
+// Epilogues: bfloat16 y; the tanh form of gelu on y plus a bias; or act[M, N/2] = silu(g) * u for W with gate and up rows interleaved
 // in blocks of 8 (a thread holds 32 consecutive columns of a row, so g_i and u_i meet in it).
 //
 // Rows of x past M, rows of W past N and k past K are zero-filled by TMA, so any M and N and
@@ -45,9 +45,11 @@ struct TcParams {
   int M, N, K;
   int ldo;
   // 0: bfloat16 y; 3: bfloat16 silu(g)*u; 4: bfloat16 gelu(y); 5: float y to the rows that `scatter` names; 6: bfloat16 relu(y)^2;
+  // 8: bfloat16 gelu_tanh(y + bias), bias float [N] or null
   // 7: as 3 with g' = min(g, limit), u' = clamp(u, -limit, limit) and g' / (1 + exp(-alpha g')) * (u' + shift)
   int mode;
   float act_limit, act_alpha, act_shift;
+  const float* bias;
   int* err;
   // grouped form: `tiles` holds (expert, first row, rows) per row tile, meta[0] their number (at most max_row_tiles);
   // N is then the number of output columns of ONE expert
@@ -302,6 +304,25 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x, const __grid_cons
             r[i] = __float_as_uint(0.5f * z * (1.f + erff(z * 0.70710678118654752440f)));
           }
         }
+        if (p.mode == 8) {
+          if (p.bias) {
+            if (col + 32 <= p.N) {
+#pragma unroll
+              for (int i = 0; i < 32; i += 4) {
+                const float4 b4 = *reinterpret_cast<const float4*>(p.bias + col + i);
+                r[i] = __float_as_uint(__uint_as_float(r[i]) + b4.x);
+                r[i + 1] = __float_as_uint(__uint_as_float(r[i + 1]) + b4.y);
+                r[i + 2] = __float_as_uint(__uint_as_float(r[i + 2]) + b4.z);
+                r[i + 3] = __float_as_uint(__uint_as_float(r[i + 3]) + b4.w);
+              }
+            } else {
+#pragma unroll
+              for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(__uint_as_float(r[i]) + (col + i < p.N ? p.bias[col + i] : 0.f));
+            }
+          }
+#pragma unroll
+          for (int i = 0; i < 32; ++i) r[i] = __float_as_uint(gelu_tanh_fast(__uint_as_float(r[i])));
+        }
         if (p.mode == 6) {
 #pragma unroll
           for (int i = 0; i < 32; ++i) {
@@ -424,18 +445,20 @@ int launch_tc(const CUtensorMap& mx, const CUtensorMap& mw, const TcParams& p, c
 
 // x: [M, K] (row stride ldx), w: [N, K] (row stride ldw), bfloat16, 16-byte aligned, K % 8 == 0,
 // strides multiples of 8.  mode 0: out bfloat16 [M, N]; mode 3: out bfloat16 [M, N/2] =
-// silu(gate) * up for w in the interleaved gate/up layout (N % 16 == 0).  err: device flag
+// silu(gate) * up for w in the interleaved gate/up layout (N % 16 == 0); mode 8: out bfloat16 [M, N] =
+// gelu_tanh(y + bias) (bias float [N], 16-byte aligned, or null).  err: device flag
 // (bit 4 is raised if a wait inside the kernel ran out).
 KVF_API int kvf_gemm_tcgen05_bf16(const void* x, const void* w, void* out, int M, int N, int K, int ldx, int ldw,
-                                  int ldo, int mode, int* err, cudaStream_t st) {
+                                  int ldo, int mode, const float* bias, int* err, cudaStream_t st) {
   if (M <= 0 || N <= 0) return 0;
-  if (K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || (ldo & 7) || (mode != 0 && mode != 3))
+  if (K <= 0 || (K & 7) || (ldx & 7) || (ldw & 7) || (ldo & 7) || (mode != 0 && mode != 3 && mode != 8))
     return (int)cudaErrorInvalidValue;
-  if ((((uintptr_t)x) | ((uintptr_t)w) | ((uintptr_t)out)) & 15) return (int)cudaErrorInvalidValue;
+  if ((((uintptr_t)x) | ((uintptr_t)w) | ((uintptr_t)out) | ((uintptr_t)bias)) & 15) return (int)cudaErrorInvalidValue;
   if (mode == 3 && (N & 15)) return (int)cudaErrorInvalidValue;
   TcParams p;
   p.out = out; p.M = M; p.N = N; p.K = K; p.ldo = ldo; p.mode = mode; p.err = err;
   p.act_limit = p.act_alpha = p.act_shift = 0.f;
+  p.bias = bias;
   p.tiles = nullptr; p.meta = nullptr; p.scatter = nullptr; p.max_row_tiles = 0;
   CUtensorMap mx, mw;
   int rc = make_map(&mx, x, M, K, ldx, BM);
@@ -466,6 +489,7 @@ KVF_API int kvf_gemm_grouped_tcgen05_bf16(const void* x, const void* w, void* ou
   TcParams p;
   if (gelu == 3 && (N & 15)) return (int)cudaErrorInvalidValue;
   p.out = out; p.M = P; p.N = N; p.K = K; p.ldo = ldo; p.mode = gelu == 3 ? 7 : gelu == 2 ? 6 : gelu ? 4 : 5; p.err = err;
+  p.bias = nullptr;
   p.act_limit = act_limit; p.act_alpha = act_alpha; p.act_shift = act_shift;
   p.tiles = tiles; p.meta = meta; p.scatter = gelu ? nullptr : scatter; p.max_row_tiles = max_row_tiles;
   CUtensorMap mx, mw;

@@ -70,7 +70,7 @@ struct JointParams {
 };
 
 template <typename T, int V>
-__global__ void __launch_bounds__(256) joint_norm_cache_kernel(const JointParams p) {
+__global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParams p) {
   pdl_launch();
   extern __shared__ __align__(16) float row[];  // q and k of the token
   __shared__ float red[64];
@@ -190,7 +190,10 @@ int joint_norm_cache(const JointParams& p, int n_tokens, cudaStream_t st) {
     cudaError_t e = cudaFuncSetAttribute(kern, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem);
     if (e != cudaSuccess) return (int)e;
   }
-  return launch(kern, dim3(n_tokens), dim3(256), smem, st, p);
+  // few tokens: a thread for every four numbers, so that all slices of a row are asked for at once
+  const int units = p.width / (vec ? 4 : 1);
+  const int threads = n_tokens > 148 || units <= 256 ? 256 : units <= 512 ? 512 : 1024;
+  return launch(kern, dim3(n_tokens), dim3(threads), smem, st, p);
 }
 
 // ---------------------------------------------------------------- a logistic gate on an attention layer's result

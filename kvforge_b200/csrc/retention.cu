@@ -8,9 +8,9 @@
 //
 //   prepare : a warp per (token, head of q, k or v): rotation, scaling, widening to float.  Nothing here depends
 //             on the state, so it runs over all tokens at once.
-//   walk    : csrc/decay_walk.cuh.
+//   walk    : csrc/decay_walk.cuh, or for many tokens csrc/decay_chunks.cuh.
 //   gate    : every head's read-out divided by its root mean square and multiplied by act(gate).
-#include "decay_walk.cuh"
+#include "decay_chunks.cuh"
 
 using namespace kvf;
 
@@ -96,13 +96,15 @@ __global__ void __launch_bounds__(128) retention_gate_kernel(const float* __rest
 // x: rows of the projections (q heads from q_off, k heads from k_off, v heads from v_off; H heads each of dk, dk, dv).
 // qn, kn [N][H*dk] and vn [N][H*dv]: float scratch.  state: float, slot i at state + i * state_stride, [H][dk][dv].
 // out: float [N][H*dv] (row stride out_stride).  decay: float [H].  max_q_len: the most rows a sequence of the step brings
-// (0: unknown); a step of single tokens stages one token, not sixteen.  Two launches.
+// (0: unknown); a step of single tokens stages one token, not sixteen.  With `raw` (float scratch [N][H][64]) and log_decay
+// (float [H]) the chunked form runs.  Two launches, three in the chunked form.
 #define KVF_RETENTION_API(SUF, T)                                                                                       \
   KVF_API int kvf_retention_##SUF(const void* x, long long x_stride, int q_off, int k_off, int v_off,                   \
                                   const int* positions, const float* inv_freq, int rot, int split_pairs,                \
                                   float k_scale, int act, const float* decay, float* state, long long state_stride, float* out,  \
                                   long long out_stride, const int* qsl, const int* state_slots, int B, long long N,     \
                                   int H, int dk, int dv, float* qn, float* kn, float* vn, int max_q_len,                \
+                                  const float* log_decay, float* raw,                                                   \
                                   cudaStream_t st) {                                                                    \
     if (B <= 0 || N <= 0) return 0;                                                                                     \
     if (H <= 0 || dk <= 0 || dk > 512 || dv <= 0 || rot < 0 || rot > dk || (rot & 1) || (unsigned)B > 65535u ||         \
@@ -113,6 +115,9 @@ __global__ void __launch_bounds__(128) retention_gate_kernel(const float* __rest
                     x_stride, q_off, k_off, v_off, positions, inv_freq, rot, split_pairs, k_scale, act, N, H, dk, dv, qn,    \
                     kn, vn);                                                                                            \
     if (rc) return rc;                                                                                                  \
+    if (raw)                                                                                                            \
+      return decay_chunks<false>(qn, kn, vn, log_decay, raw, state, state_stride, out, out_stride, qsl, state_slots, B, \
+                                 N, H, 1, dk, dv, st);                                                                  \
     return decay_walk<false>(qn, kn, vn, decay, state, state_stride, out, out_stride, qsl, state_slots, B, H, 1, dk, dv, \
                              max_q_len, st);                                                                            \
   }

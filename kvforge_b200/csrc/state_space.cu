@@ -5,12 +5,12 @@
 //   y_t = S_t^T C_t + D_h x_t
 //
 //   prepare   : a CTA per token: step sizes and decays, d x, B and C as floats.  Nothing here depends on the state.
-//   walk      : decay_walk with one decay a token and head.
+//   walk      : decay_walk with one decay a token and head, or for many tokens decay_chunks.
 //   wide_norm : what follows a recurrence: the read-out (plus D x), gated before or after a norm over wide parts of the
 //               row (one part, or several equal ones), times a weight.
 //
 // Everything is float whatever the storage type T of projections and results.
-#include "decay_walk.cuh"
+#include "decay_chunks.cuh"
 
 using namespace kvf;
 
@@ -50,7 +50,7 @@ template <> struct Run<bf16, 4> {
 template <typename T, int V>
 __global__ void __launch_bounds__(256) state_space_prepare_kernel(const T* __restrict__ x, long long ldx, const T* __restrict__ dt,
                                                                    long long lddt, const float* __restrict__ dt_bias,
-                                                                   const float* __restrict__ a_log, int H, int dv, int gn,
+                                                                   const float* __restrict__ a_log, int log_form, int H, int dv, int gn,
                                                                    float* __restrict__ decay, float* __restrict__ cn,
                                                                    float* __restrict__ bn, float* __restrict__ vn) {
   pdl_launch();
@@ -60,7 +60,8 @@ __global__ void __launch_bounds__(256) state_space_prepare_kernel(const T* __res
   for (int h = threadIdx.x; h < H; h += blockDim.x) {
     const float d = softplus_exact(to_float<T>(dt[n * lddt + h]) + dt_bias[h]);
     step[h] = d;
-    decay[n * H + h] = expf(-expf(a_log[h]) * d);
+    const float l = -expf(a_log[h]) * d;
+    decay[n * H + h] = log_form ? l : expf(l);
   }
   __syncthreads();
   const T* row = x + n * ldx;
@@ -183,13 +184,14 @@ int wide_norm_gate(const WideNormParams& p, long long n_tokens, cudaStream_t st)
 
 // x: rows of  x [H*dv] | B [G*N] | C [G*N]; dt: rows of [H]; out: float [N_tokens][H*dv] (row stride out_stride), the
 // read-out without the D term.  state: float, slot i at state + i * state_stride, [H][N][dv].  Scratch: decay [tokens][H],
-// cn and bn [tokens][G*N], vn [tokens][H*dv].  Two launches.
+// cn and bn [tokens][G*N], vn [tokens][H*dv], and for the chunked form raw [tokens][G][64] (else null).  Two launches,
+// three in the chunked form.
 #define KVF_STATE_SPACE_API(SUF, T)                                                                                     \
   KVF_API int kvf_state_space_##SUF(const void* x, long long ldx, const void* dt, long long lddt, const float* dt_bias, \
                                     const float* a_log, float* state, long long state_stride, float* out,               \
                                     long long out_stride, const int* qsl, const int* state_slots, int B,                \
                                     long long n_tokens, int H, int G, int ns, int dv, float* decay, float* cn,          \
-                                    float* bn, float* vn, int max_q_len, cudaStream_t st) {                             \
+                                    float* bn, float* vn, int max_q_len, float* raw, cudaStream_t st) {                             \
     if (B <= 0 || n_tokens <= 0) return 0;                                                                              \
     if (H <= 0 || G <= 0 || H % G || ns <= 0 || ns > 512 || dv <= 0 || (unsigned)B > 65535u || (unsigned)H > 65535u ||  \
         n_tokens > 0x7fffffffLL)                                                                                        \
@@ -200,8 +202,11 @@ int wide_norm_gate(const WideNormParams& p, long long n_tokens, cudaStream_t st)
                      al(cn, 16);                                                                                        \
     int rc = launch(vec ? state_space_prepare_kernel<T, 4> : state_space_prepare_kernel<T, 1>,                          \
                     dim3((unsigned)n_tokens), dim3(256), (size_t)H * sizeof(float), st, (const T*)x, ldx,               \
-                    (const T*)dt, lddt, dt_bias, a_log, H, dv, gn, decay, cn, bn, vn);                                  \
+                    (const T*)dt, lddt, dt_bias, a_log, raw ? 1 : 0, H, dv, gn, decay, cn, bn, vn);                                  \
     if (rc) return rc;                                                                                                  \
+    if (raw)                                                                                                            \
+      return decay_chunks<true>(cn, bn, vn, decay, raw, state, state_stride, out, out_stride, qsl, state_slots, B,      \
+                                n_tokens, H, H / G, ns, dv, st);                                                        \
     return decay_walk<true>(cn, bn, vn, decay, state, state_stride, out, out_stride, qsl, state_slots, B, H, H / G, ns, \
                             dv, max_q_len, st);                                                                         \
   }                                                                                                                     \

@@ -33,9 +33,9 @@ _SIGNATURES = {
     "kvf_paged_attention_decode_fused_bf16": "pppppppiiiiiiiifiiiipppp",
     "kvf_paged_attention_decode_tma_bf16": "pppppppiiiiiiiilfiiiippppiip",
     "kvf_gemm_nt_f32": "pppiiiiiip",
-    "kvf_gemm_skinny_bf16": "pppiiiiiiiilp",
+    "kvf_gemm_skinny_bf16": "pppiiiiiiiilpp",
     "kvf_set_pdl": "i",
-    "kvf_gemm_tcgen05_bf16": "pppiiiiiiipp",
+    "kvf_gemm_tcgen05_bf16": "pppiiiiiiippp",
     "kvf_sample_f32": "pliippppppp",
     "kvf_argmax_f32": "pliipipp",
     "kvf_scale_softcap_f32": "plffp",
@@ -75,11 +75,11 @@ _SIGNATURES = {
     "kvf_talking_set_pdl": "i",
     "kvf_gated_set_pdl": "i",
     # library "decay"
-    "kvf_retention_{s}": "pliiippiifipplplppiliiipppip",
+    "kvf_retention_{s}": "pliiippiifipplplppiliiipppippp",
     "kvf_retention_gate_{s}": "plplfiliiplp",
     "kvf_tanh_norm_{s}": "pppilfppppplip",
     "kvf_decay_set_pdl": "i",
-    "kvf_state_space_{s}": "plplppplplppiliiiippppip",
+    "kvf_state_space_{s}": "plplppplplppiliiiippppipp",
     "kvf_wide_norm_gate_{s}": "plpplipliipffliiplp",
     # library "joint"
     "kvf_joint_norm_cache_{s}": "plpilipppiifpppiiiiiilpp",
@@ -885,12 +885,21 @@ def skinny_splits(n_out: int, k: int, m: int = 8) -> int:
     return s
 
 
-def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | Partials, mode: str = "plain") -> None:
+def _check_bias(bias: torch.Tensor | None, n: int, mode: str) -> None:
+    if bias is None:
+        return
+    _need(bias, torch.float32, "product bias")
+    if mode != "gelu_tanh" or bias.numel() != n:
+        raise ValueError("a product's bias belongs to its activation and has one entry a column")
+
+
+def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | Partials, mode: str = "plain", bias: torch.Tensor | None = None) -> None:
     """``x [M<=64, K] @ w [N, K]^T`` in bfloat16 with float accumulation.
 
     ``out``: a bfloat16 or float ``[M, N]`` tensor, ``Partials`` (``[S, M, N]`` float, one slice
     of K each), or with ``mode="silu"`` a bfloat16 ``[M, N/2]`` tensor that receives
-    ``silu(gate) * up`` for ``w`` in the interleaved gate/up layout.
+    ``silu(gate) * up`` for ``w`` in the interleaved gate/up layout; with ``mode="gelu_tanh"`` a bfloat16 ``[M, N]`` tensor that
+    receives ``gelu_tanh(x w^T + bias)`` (``bias`` float ``[N]`` or ``None``).
     """
     m, k = x.shape
     if not (x.dtype == torch.bfloat16 and w.dtype == torch.bfloat16 and 0 < m <= SKINNY_MAX_M and k % 8 == 0
@@ -916,6 +925,10 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | Partials, 
             code = 3
         elif tuple(out.shape) != (m, n):
             raise ValueError("gemm_skinny: out shape")
+        elif mode == "gelu_tanh":
+            if out.dtype != torch.bfloat16:
+                raise TypeError("gemm_skinny: an activation's result is bfloat16")
+            code = 4
         elif out.dtype == torch.bfloat16:
             code = 0
         elif out.dtype == torch.float32:
@@ -923,8 +936,9 @@ def gemm_skinny(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor | Partials, 
         else:
             raise TypeError("gemm_skinny: out must be bfloat16 or float32")
         ldo, optr = out.stride(0), _ptr(out)
+    _check_bias(bias, n, mode)
     name = "kvf_gemm_skinny_bf16"
-    _check(_fn(name)(_ptr(x), _ptr(w), optr, m, n, k, x.stride(0), w.stride(0), ldo, code, ksplit, stride, _stream()), name)
+    _check(_fn(name)(_ptr(x), _ptr(w), optr, m, n, k, x.stride(0), w.stride(0), ldo, code, ksplit, stride, _ptr(bias), _stream()), name)
 
 
 TCGEN05_MIN_TILES = 120  # below this many 128 x 256 output tiles the persistent grid leaves SMs idle
@@ -941,10 +955,13 @@ def tcgen05_ok(x: torch.Tensor, w: torch.Tensor, min_tiles: int = TCGEN05_MIN_TI
     )  # fmt: skip
 
 
-def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str = "plain", err: torch.Tensor | None = None) -> None:
+def gemm_tcgen05(
+    x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str = "plain", err: torch.Tensor | None = None, bias: torch.Tensor | None = None
+) -> None:
     """``x [M, K] @ w [N, K]^T`` in bfloat16 on the tcgen05 tensor cores (TMA loads, float
     accumulation in tensor memory).  ``out``: bfloat16 ``[M, N]``, or with ``mode="silu"``
-    bfloat16 ``[M, N/2] = silu(gate) * up`` for ``w`` in the interleaved gate/up layout."""
+    bfloat16 ``[M, N/2] = silu(gate) * up`` for ``w`` in the interleaved gate/up layout, or with ``mode="gelu_tanh"``
+    ``gelu_tanh(x w^T + bias)`` (``bias`` float ``[N]`` or ``None``)."""
     if not tcgen05_ok(x, w, min_tiles=0):
         raise ValueError("gemm_tcgen05: needs bfloat16, K % 8 == 0, unit inner strides, 16-byte aligned rows")
     m, k = x.shape
@@ -961,9 +978,10 @@ def gemm_tcgen05(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor, mode: str 
     else:
         if tuple(out.shape) != (m, n):
             raise ValueError("gemm_tcgen05: out shape")
-        code = 0
+        code = 8 if mode == "gelu_tanh" else 0
+    _check_bias(bias, n, mode)
     name = "kvf_gemm_tcgen05_bf16"
-    _check(_fn(name)(_ptr(x), _ptr(w), _ptr(out), m, n, k, x.stride(0), w.stride(0), out.stride(0), code, _ptr(err), _stream()), name)
+    _check(_fn(name)(_ptr(x), _ptr(w), _ptr(out), m, n, k, x.stride(0), w.stride(0), out.stride(0), code, _ptr(bias), _ptr(err), _stream()), name)
 
 
 def linear(x: torch.Tensor, w: torch.Tensor, out: torch.Tensor) -> None:
@@ -1143,8 +1161,8 @@ def causal_conv(
 ) -> None:  # fmt: skip
     """Short causal convolution over time per channel of a flat batch, and the state moved on.
 
-    ``x [N, C]`` (rows may be a slice of a wider buffer), ``weight`` float ``[C, taps]`` whose last
-    column multiplies the current token, ``bias`` float ``[C]`` or ``None``, ``state`` float ``[slots, (taps-1)*C]``: the last
+    ``x [N, C]`` (rows may be a slice of a wider buffer), ``weight`` float ``[taps, C]`` (a tap's channels side by
+    side) whose last row multiplies the current token, ``bias`` float ``[C]`` or ``None``, ``state`` float ``[slots, (taps-1)*C]``: the last
     ``taps-1`` inputs of each sequence, oldest first, zeros before its start.  ``out [N, C]`` gets
     the sums (``activation``: ``None`` or ``"silu"``); afterwards the state holds this step's last
     inputs.  Sequences without rows and slots below zero are left alone.  ``max_query_len`` (0 =
@@ -1154,8 +1172,8 @@ def causal_conv(
     _rows2d(out, x.dtype, "out")
     _need(weight, torch.float32, "conv weight")
     n, c = x.shape
-    taps = weight.shape[1]
-    if tuple(weight.shape) != (c, taps) or tuple(out.shape) != (n, c):
+    taps = weight.shape[0]
+    if tuple(weight.shape) != (taps, c) or tuple(out.shape) != (n, c):
         raise ValueError("causal_conv: shapes do not agree")
     if bias is not None:
         _need(bias, torch.float32, "conv bias")
@@ -2026,6 +2044,33 @@ def tanh_norm(
     )
 
 
+CHUNK_TOKENS = 64  # tokens of a chunk of the chunked form of a recurrence
+# Steps of at most this many sequences, one of which brings at least so many tokens, take it (bfloat16 storage).  One sequence of
+# 2,048 tokens: 64 heads of 128 x 64 with a decay a token 523 us by the walk and 334 us by chunks (the kernels around it
+# included), 16 heads of 128 x 128 448 and 306 us.  Four sequences of 512: 340 and 338 us; eight of 256: 305 and 305 us:
+# the walk's chains hide one another, and the chunked form's CTAs fill an SM each.
+CHUNKS_MAX_SEQS = 2
+CHUNKS_MIN_QUERY = 256
+
+
+def chunks_pay(num_seqs: int, max_query_len: int) -> bool:
+    """Whether a step's shape makes the chunked form the faster one."""
+    return num_seqs <= CHUNKS_MAX_SEQS and max_query_len >= CHUNKS_MIN_QUERY
+
+
+def chunks_ok(dk: int, dv: int, state: torch.Tensor) -> bool:
+    """Whether the chunked form (``csrc/decay_chunks.cuh``) takes a state of ``dk`` rows of ``dv`` numbers a head that lies so."""
+    return dk <= 128 and dk % 4 == 0 and dv % 4 == 0 and state.data_ptr() % 16 == 0 and state.stride(0) % 4 == 0
+
+
+def _check_chunks(raw: torch.Tensor, n: int, key_heads: int, dk: int, dv: int, state: torch.Tensor, out: torch.Tensor) -> None:
+    _need(raw, torch.float32, "scratch raw")
+    if tuple(raw.shape) != (n, key_heads * CHUNK_TOKENS):
+        raise ValueError(f"scratch raw must be float [{n}, {key_heads * CHUNK_TOKENS}]")
+    if not chunks_ok(dk, dv, state) or out.stride(0) % 4:
+        raise ValueError("the chunked form does not take these sizes")
+
+
 RETENTION_MAX_KEY_DIM = 512  # rows of a head's state that the walk holds in the registers of 32 lanes
 
 
@@ -2033,7 +2078,7 @@ def retention(
     x: torch.Tensor, q_off: int, k_off: int, v_off: int, positions: torch.Tensor, inv_freq: torch.Tensor | None, interleaved: bool,
     k_scale: float, decay: torch.Tensor, state: torch.Tensor, out: torch.Tensor, qsl: torch.Tensor, state_slots: torch.Tensor,
     num_seqs: int, num_heads: int, dk: int, dv: int, scratch: tuple[torch.Tensor, torch.Tensor, torch.Tensor] | None = None,
-    max_query_len: int = 0, activation: str | None = None,
+    max_query_len: int = 0, activation: str | None = None, log_decay: torch.Tensor | None = None, raw: torch.Tensor | None = None,
 ) -> None:  # fmt: skip
     """Retention over a flat batch, token by token per sequence, on the float state ``S [heads, dk, dv]`` of each
     sequence's slot: ``S <- decay[h] S + k v^T``, ``out = S^T q`` (float ``[N, H*dv]``).  Rows of ``x`` hold the
@@ -2041,7 +2086,9 @@ def retention(
     ``v_off``; with ``activation="silu"`` all of them pass silu.  The first ``2*len(inv_freq)`` dims of q and k turn with the position (split pairs ``(i, i + rot/2)``
     unless ``interleaved``), then k is multiplied by ``k_scale``; all of that in float.  ``scratch``: float buffers
     ``(qn [N, H*dk], kn [N, H*dk], vn [N, H*dv])``; without it they are allocated here.  ``max_query_len`` (0 = unknown):
-    the most rows a sequence of the step brings (a step of single tokens stages less).  Two launches."""
+    the most rows a sequence of the step brings (a step of single tokens stages less).  With ``raw`` (float scratch
+    ``[N, H*64]``) and ``log_decay`` (float ``[H]``) the recurrence runs chunk by chunk instead of token by token
+    (``chunks_ok`` says for which sizes).  Two launches, three in the chunked form."""
     s = _suffix(x.dtype)
     _rows2d(x, None, "x")
     n = x.shape[0]
@@ -2076,15 +2123,20 @@ def retention(
         _need(t, torch.float32, f"scratch {what}")
         if tuple(t.shape) != (n, w):
             raise ValueError(f"retention: scratch {what} must be float [{n}, {w}]")
+    if raw is not None:
+        _check_chunks(raw, n, h, dk, dv, state, out)
+        _need(log_decay, torch.float32, "log_decay")
+        if log_decay.numel() != h:
+            raise ValueError("retention: one logarithm per head")
     name = f"kvf_retention_{s}"
     _check(
         _fn(name, DECAY_LIB)(
             _ptr(x), x.stride(0), int(q_off), int(k_off), int(v_off), _ptr(positions), _ptr(inv_freq) if rot else None, rot,
             0 if interleaved else 1, float(k_scale), 1 if activation == "silu" else 0, _ptr(decay), sptr, sstride, _ptr(out), out.stride(0), _ptr(qsl), _ptr(state_slots),
-            int(num_seqs), n, h, int(dk), int(dv), _ptr(qn), _ptr(kn), _ptr(vn), int(max_query_len), _stream(),
+            int(num_seqs), n, h, int(dk), int(dv), _ptr(qn), _ptr(kn), _ptr(vn), int(max_query_len), _ptr(log_decay), _ptr(raw), _stream(),
         ),
         name,
-        2,
+        3 if raw is not None else 2,
     )  # fmt: skip
 
 
@@ -2118,13 +2170,15 @@ def state_space(
     x: torch.Tensor, dt: torch.Tensor, dt_bias: torch.Tensor, a_log: torch.Tensor, state: torch.Tensor, out: torch.Tensor,
     qsl: torch.Tensor, state_slots: torch.Tensor, num_seqs: int, num_heads: int, groups: int, n_state: int, dv: int,
     scratch: tuple[torch.Tensor, torch.Tensor, torch.Tensor, torch.Tensor] | None = None, max_query_len: int = 0,
+    raw: torch.Tensor | None = None,
 ) -> None:  # fmt: skip
     """A state space per head whose step size follows the token, over a flat batch, on the float state ``S [heads, n_state,
     dv]`` of each sequence's slot: ``d = softplus(dt + dt_bias)``, ``S <- exp(-exp(a_log) d) S + B (d x)^T``, ``out = S^T C``
     (float ``[N, H*dv]``; the term that passes ``x`` on is ``wide_norm_gate``'s).  Rows of ``x`` hold ``x [H*dv] | B
     [groups*n_state] | C [groups*n_state]`` after their convolution; head ``h`` takes group ``h // (H / groups)``; ``dt``
     holds rows of ``H`` logits.  ``scratch``: float buffers ``(decay [N, H], cn [N, G*n_state], bn [N, G*n_state], vn
-    [N, H*dv])``; without it they are allocated here.  ``max_query_len`` as in ``retention``.  Two launches."""
+    [N, H*dv])``; without it they are allocated here.  ``max_query_len`` as in ``retention``.  With ``raw`` (float
+    scratch ``[N, groups*64]``) the chunked form runs.  Two launches, three in the chunked form."""
     s = _suffix(x.dtype)
     _rows2d(x, None, "x")
     _rows2d(dt, x.dtype, "dt")
@@ -2150,16 +2204,18 @@ def state_space(
         _need(t, torch.float32, f"scratch {what}")
         if tuple(t.shape) != (n, w):
             raise ValueError(f"state_space: scratch {what} must be float [{n}, {w}]")
+    if raw is not None:
+        _check_chunks(raw, n, g, n_state, dv, state, out)
     decay, cn, bn, vn = scratch
     name = f"kvf_state_space_{s}"
     _check(
         _fn(name, DECAY_LIB)(
             _ptr(x), x.stride(0), _ptr(dt), dt.stride(0), _ptr(dt_bias), _ptr(a_log), sptr, sstride, _ptr(out), out.stride(0), _ptr(qsl),
             _ptr(state_slots), int(num_seqs), n, h, g, int(n_state), int(dv), _ptr(decay), _ptr(cn), _ptr(bn), _ptr(vn), int(max_query_len),
-            _stream(),
+            _ptr(raw), _stream(),
         ),
         name,
-        2,
+        3 if raw is not None else 2,
     )  # fmt: skip
 
 

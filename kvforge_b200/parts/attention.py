@@ -183,7 +183,7 @@ class PagedAttention(Mixer):
         self.w_o = weights["o_proj.weight"].contiguous()
         self.w_conv = None
         if self.taps:
-            self.w_conv = torch.cat([weights["q_proj.conv"], weights["k_proj.conv"], weights["v_proj.conv"]], dim=0).contiguous()
+            self.w_conv = torch.cat([weights["q_proj.conv"], weights["k_proj.conv"], weights["v_proj.conv"]], dim=0).t().contiguous()
         self.q_norm_w = weights.get("q_norm.weight") if self.qk_eps is not None else None
         self.k_norm_w = weights.get("k_norm.weight") if self.qk_eps is not None else None
         bias = ops.DistanceBias(weights["rel"].contiguous(), distance_buckets(*self.bias_shape).to(rt.device)) if self.bias_shape is not None else None

@@ -135,7 +135,7 @@ class GatedDeltaRule(Mixer):
         self.w_a2 = W.get("a2")
         self.w_g2 = W.get("g2")
         self.w_o = W["o"].contiguous()
-        self.w_conv = torch.cat([W["q.conv"], W["k.conv"], W["v.conv"]], dim=0).contiguous()
+        self.w_conv = torch.cat([W["q.conv"], W["k.conv"], W["v.conv"]], dim=0).t().contiguous()
         self.a_log, self.dt_bias, self.norm_w = W["A_log"], W["dt_bias"], W["norm"]
         del dev, dt
 

@@ -117,6 +117,15 @@ class PlainMLP(FeedForward):
     def forward(self, ctx, x: torch.Tensor):
         rt = self.rt
         n = x.shape[0]
+        if self.activation == "gelu_tanh" and self.extra_w is None:
+            # the activation as the accumulator leaves the product: a few tokens, many tokens
+            act = rt.buf("pmlp.act", n, self.inter)
+            if ops.skinny_ok(x, self.w_up):
+                ops.gemm_skinny(x, self.w_up, act, mode="gelu_tanh", bias=self.b_up)
+                return self._down(act, ctx)
+            if ops.tcgen05_ok(x, self.w_up) and self.inter % 8 == 0:
+                ops.gemm_tcgen05(x, self.w_up, act, mode="gelu_tanh", err=rt.err, bias=self.b_up)
+                return self._down(act, ctx)
         u = rt.buf("pmlp.up", n, self.w_up.shape[0])
         if ops.skinny_ok(x, self.w_up):
             ops.gemm_skinny(x, self.w_up, u)
@@ -125,5 +134,8 @@ class PlainMLP(FeedForward):
         self.extra_out = u[:, self.extra_off : self.extra_off + self.extra_w.shape[0]] if self.extra_w is not None else None
         act = rt.buf("pmlp.act", n, self.inter)
         ops.unary_act(u[:, : self.inter], act, self.activation, self.ab, self.b_up)
-        y = project(rt, "pmlp.out", act, self.w_down, None if self.has_bias else ctx)
+        return self._down(act, ctx)
+
+    def _down(self, act: torch.Tensor, ctx):
+        y = project(self.rt, "pmlp.out", act, self.w_down, None if self.has_bias else ctx)
         return ops.Biased(y, self.b_down) if self.has_bias else y

@@ -88,6 +88,10 @@ class Retention(Mixer):
         self.norm_w = weights["norm"].contiguous() if self.norm == "joint" else None
         self.w_o = weights["o"].contiguous()
         self.decay = torch.tensor(self.decay_values, dtype=torch.float32, device=rt.device)
+        # the chunked form works with logarithms: decays in (0, 1]
+        self.log_decay = None
+        if all(0.0 < a <= 1.0 for a in self.decay_values):
+            self.log_decay = torch.tensor(self.decay_values, dtype=torch.float64).log().to(device=rt.device, dtype=torch.float32)
         if self.position_spec is not None and self.position is None:
             self.position = build_part("position", self.position_spec)
             self.position.bind({}, rt)
@@ -118,9 +122,15 @@ class Retention(Mixer):
             rt.buf("retention.kn", n, h * dk, torch.float32),
             rt.buf("retention.vn", n, h * dv, torch.float32),
         )
+        # many tokens of few sequences in bfloat16: chunk by chunk; 32-bit: token by token, the same bits however a sequence is cut
+        raw = None
+        chunked = rt.dtype == torch.bfloat16 and self.log_decay is not None and ops.chunks_pay(ctx.num_seqs, ctx.max_query_len)
+        if chunked and ops.chunks_ok(dk, dv, cache.state):
+            raw = rt.buf("retention.raw", n, h * ops.CHUNK_TOKENS, torch.float32)
         ops.retention(
             y, 0, self.k_off, self.v_off, ctx.positions, self.inv_freq, self.interleaved, self.key_scale, self.decay, cache.state, o,
             ctx.query_start_loc, ctx.state_slots, ctx.num_seqs, h, dk, dv, scratch, max_query_len=ctx.max_query_len, activation=self.activation,
+            log_decay=self.log_decay, raw=raw,
         )  # fmt: skip
         gate = y[:, self.g_off : self.g_off + h * dv] if self.gate else None
         if self.norm == "joint":

@@ -70,7 +70,7 @@ class StateSpace(Mixer):
         self.w_in, (self.z_off, self.x_off, self.dt_off) = stack_rows([z, xbc, dt])
         self.in_dim = self.w_in.shape[0]
         self.w_o = weights["o"].contiguous()
-        self.w_conv, self.b_conv = weights["conv"].contiguous(), weights["conv.b"].contiguous()
+        self.w_conv, self.b_conv = weights["conv"].t().contiguous(), weights["conv.b"].contiguous()
         self.dt_bias, self.a_log, self.skip, self.norm_w = (weights[k].contiguous() for k in ("dt_bias", "A_log", "D", "norm"))
 
     def forward(self, ctx, x: torch.Tensor, cache):
@@ -91,9 +91,13 @@ class StateSpace(Mixer):
         f32 = torch.float32
         read = rt.buf("ssm.read", n, self.inner, f32)
         scratch = (rt.buf("ssm.decay", n, H, f32), rt.buf("ssm.cn", n, gn, f32), rt.buf("ssm.bn", n, gn, f32), rt.buf("ssm.vn", n, self.inner, f32))
+        # many tokens of few sequences in bfloat16: chunk by chunk; 32-bit: token by token, the same bits however a sequence is cut
+        state, raw = cache.state[:, self.conv_floats :], None
+        if rt.dtype == torch.bfloat16 and ops.chunks_pay(ctx.num_seqs, ctx.max_query_len) and ops.chunks_ok(self.N, dv, state):
+            raw = rt.buf("ssm.raw", n, self.G * ops.CHUNK_TOKENS, f32)
         ops.state_space(
-            xbc, y[:, self.dt_off : self.dt_off + H], self.dt_bias, self.a_log, cache.state[:, self.conv_floats :], read, ctx.query_start_loc,
-            ctx.state_slots, ctx.num_seqs, H, self.G, self.N, dv, scratch, max_query_len=ctx.max_query_len,
+            xbc, y[:, self.dt_off : self.dt_off + H], self.dt_bias, self.a_log, state, read, ctx.query_start_loc,
+            ctx.state_slots, ctx.num_seqs, H, self.G, self.N, dv, scratch, max_query_len=ctx.max_query_len, raw=raw,
         )  # fmt: skip
         out = rt.buf("ssm.out", n, self.inner)
         ops.wide_norm_gate(

@@ -284,7 +284,7 @@ def test_short_convolution_with_state(dtype, taps, act, c):
         x = torch.cat([seqs[i][at[i] : at[i] + lens[i]] for i in range(3)] + [torch.randn(3, c, generator=g)]).to(dev, dt)
         qsl, sl = flat_batch(lens + [0, 0], slots + [5, -1], dev)
         out = torch.full_like(x, 7.0)
-        ops.causal_conv(x, w.to(dev), view, qsl, sl, 5, out, activation=act, max_query_len=max(lens) if step in (1, 2) else 0)
+        ops.causal_conv(x, w.t().contiguous().to(dev), view, qsl, sl, 5, out, activation=act, max_query_len=max(lens) if step in (1, 2) else 0)
         assert bool((out[-3:] == 7.0).all())
         o = 0
         for i in range(3):
@@ -319,7 +319,7 @@ def test_short_convolution_of_a_step_with_many_rows(dtype, taps):
         x = torch.cat([u[: ls[i]] if step == 0 else u[lens[i][0] :] for i, u in enumerate(seqs)]).to(dev, dt)
         qsl, sl = flat_batch(ls, [3, 0, 4, 1], dev)
         out = torch.empty_like(x)
-        ops.causal_conv(x, w.to(dev), state, qsl, sl, 4, out)
+        ops.causal_conv(x, w.t().contiguous().to(dev), state, qsl, sl, 4, out)
         o = 0
         for i in range(4):
             got[i].append(out[o : o + ls[i]].float().cpu())

@@ -174,6 +174,30 @@ def test_long_decoding(models):
             check(steps, outs, ref, scale, TOL[dtype])
 
 
+def test_long_prompts_in_bfloat16(models):
+    """Prompts long enough for the recurrences' chunked form, whole and cut so that portions of it follow single tokens and end
+    inside a chunk; eager and as captured graphs (whose padding belongs to no sequence)."""
+    from kvforge_b200 import ops
+
+    for name in ("a", "d", "e"):
+        case = CASES[name]
+        folder, _, _, _, w = models[name]
+        reqs = {"long": tokens(case["config"]["vocab"], 390, 8)}
+        ref = {"long": plain_logits(case["config"], w, reqs["long"])}
+        scale = float(ref["long"].pow(2).mean().sqrt())
+        pos, cut = 0, []
+        for n in (1, 270, 1, 2, 90, 26):
+            cut.append({"step": len(cut), "entries": [{"id": "long", "tokens": reqs["long"][pos : pos + n], "want": list(range(n))}], "end": ["long"] if pos + n == 390 else []})
+            pos += n
+        assert pos == 390 and ops.chunks_pay(1, 270) and not ops.chunks_pay(1, 90)
+        for steps in (traces.whole(reqs), cut):
+            outs, _ = run_trace(folder, "bfloat16", steps, case["block_size"])
+            check(steps, outs, ref, scale, TOL["bfloat16"])
+            last = traces.last_only(steps)
+            outs, _ = run_trace(folder, "bfloat16", last, case["block_size"], cuda_graphs=True)
+            check(last, outs, ref, scale, TOL["bfloat16"])
+
+
 def test_the_trace_program_reads_a_folder_and_writes_logits(models, tmp_path):
     folder, reqs, ref, scale, _ = models["b"]
     steps = traces.portions(dict(list(reqs.items())[:3]))
@@ -435,6 +459,62 @@ def test_lightning_attention_through_the_state(dtype, heads, dk, dv, t):
     two_requests(part, rt, x, ref, x2, ref2, cache, dtype)
 
 
+@pytest.mark.parametrize("per_token", [False, True])
+@pytest.mark.parametrize("heads,groups,dk,dv", [(4, 4, 16, 24), (6, 2, 20, 12), (3, 1, 4, 4), (2, 2, 128, 100), (8, 1, 128, 64), (5, 5, 100, 36), (40, 2, 64, 128)])
+def test_recurrences_chunk_by_chunk(per_token, heads, groups, dk, dv):
+    """The chunked form in 32-bit against the plain walks: sequences of 1 to 300 tokens side by side (chunks that are full, end early
+    or hold one token), states carried from step to step at places that are no chunk's edge, decays from none at all to ones
+    that leave nothing of a token's past, a slot of no sequence left alone."""
+    from kvforge_b200 import ops
+
+    if not per_token and groups != heads:
+        pytest.skip("heads with a fixed decay have keys of their own")
+    g = torch.Generator().manual_seed(heads + dk)
+    i32 = lambda v: torch.tensor(v, dtype=torch.int32, device="cuda")  # noqa: E731
+    lens, parts = [300, 1, 130, 64, 67], [[200, 1, 30, 64, 2], [100, 0, 100, 0, 65]]
+    n = sum(lens)
+    r = lambda *s: torch.randn(*s, generator=g)  # noqa: E731
+    q, k, v = r(n, groups, dk), r(n, groups, dk) / dk**0.5, r(n, heads, dv)
+    starts = [sum(lens[:i]) for i in range(len(lens))]
+    decay = torch.tensor([[1.0, 0.9995, 0.9, 0.5, 1e-6][h % 5] for h in range(heads)])
+    a_log, bias = 1.5 * r(heads), r(heads)
+    dt = 2.0 * r(n, heads)
+    dt[::7] += 12.0  # now and then a step that forgets everything
+    ref = torch.zeros(n, heads, dv, dtype=torch.float64)
+    for s0, m in zip(starts, lens):
+        rows = slice(s0, s0 + m)
+        if per_token:
+            d = plain.softplus(dt[rows].double() + bias.double())
+            ref[rows] = plain.state_space_walk(v[rows].double(), k[rows].double(), q[rows].double(), d, a_log.double(), torch.zeros(heads, dtype=torch.float64))
+        else:
+            ref[rows] = plain.fixed_decay_walk(q[rows].double(), k[rows].double(), v[rows].double(), decay.double().tolist())
+    state = torch.zeros(7, heads * dk * dv + 4, device="cuda")
+    view = state[:, 4:]
+    slots = [5, 0, 3, 6, 1]
+    got = torch.zeros(n, heads, dv)
+    done = [0] * len(lens)
+    for part in parts:
+        idx = [s0 + d + j for s0, d, m in zip(starts, done, part) for j in range(m)]
+        qsl = [0]
+        for m in part:
+            qsl.append(qsl[-1] + m)
+        rows, out = len(idx), torch.full((len(idx), heads * dv), float("nan"), device="cuda")
+        raw = torch.full((rows, groups * ops.CHUNK_TOKENS), float("nan"), device="cuda")
+        if per_token:
+            x = torch.cat([v[idx].reshape(rows, -1), k[idx].reshape(rows, -1), q[idx].reshape(rows, -1)], dim=1).cuda()
+            ops.state_space(x, dt[idx].cuda(), bias.cuda(), a_log.cuda(), view, out, i32(qsl), i32(slots), len(lens), heads, groups, dk, dv, max_query_len=max(part), raw=raw)
+        else:
+            x = torch.cat([q[idx].reshape(rows, -1), k[idx].reshape(rows, -1), v[idx].reshape(rows, -1)], dim=1).cuda()
+            ops.retention(x, 0, heads * dk, 2 * heads * dk, i32([0] * rows), None, False, 1.0, decay.cuda(), view, out, i32(qsl), i32(slots), len(lens), heads, dk, dv,
+                          max_query_len=max(part), log_decay=decay.double().log().float().cuda(), raw=raw)  # fmt: skip
+        got[idx] = out.cpu().reshape(rows, heads, dv)
+        done = [d + m for d, m in zip(done, part)]
+    assert rel_rows(got, ref) < 2e-5
+    for rid, (s0, m) in enumerate(zip(starts, lens)):
+        assert rel_rows(got[s0 : s0 + m], ref[s0 : s0 + m]) < 5e-5, rid
+    assert float(state[[2, 4]].abs().max()) == 0.0 and float(state[:, :4].abs().max()) == 0.0
+
+
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 def test_wide_norm_and_gate(dtype):
     """Parts and the whole row, the gate before and after the norm, with and without what passes the recurrence by, a constant,
@@ -505,7 +585,7 @@ def test_convolution_with_a_bias(dtype, taps, c, act):
         state = torch.zeros(3, (taps - 1) * c, device="cuda")
         out = torch.empty(t, c, dtype=dtype, device="cuda")
         for lo, hi in cuts:
-            ops.causal_conv(x[lo:hi].cuda(), w.cuda(), state, i32([0, hi - lo]), i32([1]), 1, out[lo:hi], activation=act, max_query_len=hi - lo, bias=b.cuda())
+            ops.causal_conv(x[lo:hi].cuda(), w.t().contiguous().cuda(), state, i32([0, hi - lo]), i32([1]), 1, out[lo:hi], activation=act, max_query_len=hi - lo, bias=b.cuda())
         assert torch.allclose(out.cpu().double(), want, atol=part_tol(dtype), rtol=part_tol(dtype)), cuts
 
 
