@@ -12,8 +12,8 @@ Added: cache *groups*.  Layers that keep the same thing per token form a group w
 and tables of its own.  A ``full`` group keeps every key.  A ``window`` group keeps the last
 ``window`` keys: ``append_slots`` gives pages back once every position in them lies before
 ``write_start - window + 1`` (no later query can see them); the table entry becomes ``-1``.
-A ``chunk`` group's queries see the keys of their own chunk of ``window`` positions (counted from
-position 0): a page comes back once every position in it lies before the chunk of ``write_start``.
+A ``chunk`` group's queries see the keys of their own chunk of ``window`` positions (which
+begins at a multiple of it): a page comes back once every position in it lies before the chunk of ``write_start``.
 A window group may also keep the first ``keep_first`` positions of every request for good
 (queries see them at any distance): the pages that hold them are never given back.
 """

@@ -7,7 +7,7 @@
 // ctx_b keys in its pages after this step's writes and q_b = qsl[b+1]-qsl[b] queries;
 // query i sits at position p = ctx_b - q_b + i and sees key j iff j <= p (and
 // j > p - window when window > 0, or j < keep_first: the first keys of a sequence may stay
-// visible at any distance).  window < 0 stands for chunks of -window positions counted from position 0:
+// visible at any distance).  window < 0 stands for chunks of -window positions, which begin at its multiples:
 // query i then sees key j iff j <= p and both lie in the same chunk (csrc/common.cuh first_key).  S = scale * (q . k) in float, plus, when a table is given, a learned
 // bias by distance: bias[head][min(p - j, far)], `bias` float [nh][far + 1] (a head's values for
 // neighbouring keys lie side by side); softmax in float, O = P V in float, one rounding to T.

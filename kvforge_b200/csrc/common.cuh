@@ -95,7 +95,7 @@ __device__ __forceinline__ float block_max(float v, float* scratch) {
 }
 
 // The first key that a query at position `pos` sees (it sees no key after itself): span > 0: the last `span` keys, itself
-// included (a sliding window); span < 0: the keys of its own chunk of -span positions, chunks counted from position 0;
+// included (a sliding window); span < 0: the keys of its own chunk of -span positions, chunks begin at the multiples of their size;
 // span == 0: every key.  It never falls as `pos` grows.
 __device__ __forceinline__ int first_key(int pos, int span) {
   if (span == 0 || pos < 0) return 0;

@@ -571,7 +571,7 @@ def paged_attention(
 ) -> None:
     """Paged GQA attention of a flat batch (the contract is at the top of
     ``csrc/attention_generic.cu``).  ``window`` (0: none): a query sees the last ``window`` keys.  ``chunk`` (0: none; not
-    with a window): a query sees the keys of its own chunk of ``chunk`` positions, counted from position 0.
+    with a window): a query sees the keys of its own chunk, a stretch of ``chunk`` positions that begins at a multiple of it.
 
     ``dv``: size of a value head when it differs from ``d`` (``vcache`` is then
     ``[num_blocks, nkv, block_size, dv]`` and ``out`` ``[N, nh*dv]``); only the FP32-pipe kernel

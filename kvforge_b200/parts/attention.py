@@ -75,7 +75,7 @@ class PagedAttention(Mixer):
     """params: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``; optional
     ``position`` (a position-encoding ``PartSpec`` or ``None``), ``window`` (keys a query
     sees, itself included; ``None`` = all), ``chunk`` (instead of a window: a query sees the keys of its own chunk of
-    so many positions, chunks counted from position 0 of the sequence), ``scale`` (default ``1/sqrt(head_dim)``),
+    so many positions, which begin at its multiples), ``scale`` (default ``1/sqrt(head_dim)``),
     ``v_head_dim`` (size of a value head, default ``head_dim``) and ``conv`` (taps of a short causal
     convolution over time on every channel of q, k and v, between the projection and the rotation;
     its last ``conv - 1`` inputs are the mixer's state per request; tensors ``q_proj.conv`` ...),

@@ -64,7 +64,7 @@ class WeightDecl:
 class CacheNeed:
     """What a mixer keeps per token.  ``kind``: ``full`` (every key), ``window`` (the last
     ``window`` keys, and for good the first ``keep_first``), ``chunk`` (the keys of the query's own chunk
-    of ``window`` positions, chunks counted from position 0) or ``none``."""
+    of ``window`` positions, chunks begin at the multiples of their size) or ``none``."""
 
     kind: str
     kv_heads: int = 0

@@ -80,7 +80,7 @@ def whole_causal(t: int):
 
 
 def chunked_causal(t: int, size: int):
-    """A position sees itself and the earlier positions of its own chunk; chunks are counted from position 0."""
+    """A position sees itself and the earlier positions of its own chunk (positions ``c * size`` to ``c * size + size - 1``)."""
     i, j = torch.arange(t)[:, None], torch.arange(t)[None, :]
     return (j <= i) & (i // size == j // size)
 

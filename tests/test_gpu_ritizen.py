@@ -316,7 +316,7 @@ def pages(nb, nkv, bs, dk, dv, dtype):
 
 @pytest.mark.parametrize("dtype", [torch.float32, torch.bfloat16])
 @pytest.mark.parametrize("chunk", [None, 1, 7, 33, 64, 70])
-@pytest.mark.parametrize("nh,nkv,dk,dv,t,bs", [(6, 3, 24, 16, 45, 4), (3, 1, 9, 13, 60, 8), (8, 2, 64, 64, 200, 16), (6, 2, 64, 64, 150, 16), (4, 2, 128, 128, 150, 16), (2, 2, 16, 40, 50, 4)])
+@pytest.mark.parametrize("nh,nkv,dk,dv,t,bs", [(6, 3, 24, 16, 45, 4), (3, 1, 9, 13, 60, 8), (8, 2, 64, 64, 200, 16), (9, 3, 64, 64, 150, 16), (4, 2, 128, 128, 150, 16), (2, 2, 16, 40, 50, 4)])
 def test_attention_with_joint_norms_gates_and_chunks(dtype, chunk, nh, nkv, dk, dv, t, bs):
     """One gate a head without biases, and one a channel with them; the whole sequence in one step, then portions and single
     tokens on top of the cache, against the plain mixer; heads of 64 and of 128 on pages of 16 go to the tensor-core
