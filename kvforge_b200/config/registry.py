@@ -88,6 +88,11 @@ def _ensure_builtin() -> None:
 
     if RITIZEN not in ARCHITECTURES:
         register_architecture(RITIZEN, RitizenConfig.from_dict, ritizen_spec)
+    from ..models.latuzen import latuzen_spec
+    from .latuzen_config import ARCHITECTURE as LATUZEN, LatuzenConfig
+
+    if LATUZEN not in ARCHITECTURES:
+        register_architecture(LATUZEN, LatuzenConfig.from_dict, latuzen_spec)
 
 
 _LLAMA3_32 = RopeScaling(factor=32.0, low_freq_factor=1.0, high_freq_factor=4.0, original_max_position_embeddings=8192)
@@ -144,3 +149,7 @@ PRESETS.update(SONALIX_PRESETS)
 from .ritizen_config import RITIZEN_PRESETS  # noqa: E402
 
 PRESETS.update(RITIZEN_PRESETS)
+
+from .latuzen_config import LATUZEN_PRESETS  # noqa: E402
+
+PRESETS.update(LATUZEN_PRESETS)

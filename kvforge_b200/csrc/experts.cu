@@ -10,6 +10,9 @@
 //             g' = min(g, limit), u' = clamp(u, -limit, limit), g' / (1 + exp(-alpha g')) * (u' + shift)
 //   combine : resid[token] += sum_k weight_k * y[token, k]   (float, k in order)
 //
+// The router may have more outputs than there are experts: a choice beyond the last expert is an identity expert, whose result is
+// the token's own input; its pair enters no product, and combine takes x[token] for it.
+//
 // A pair's row of a product depends on that row and on its expert's weights alone (its products are
 // added in the order of k: by one thread on the FP32 pipes, by the tensor cores' own order in bfloat16),
 // so a token's result does not depend on what else is in the batch or on where its pairs land in the order.  Router, scores, choice and the weighted sum are float
@@ -55,7 +58,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ x,
                                                          const float* __restrict__ router, const float* __restrict__ correction,
                                                          int n_tokens, int W, int E, int top, int groups, int keep,
                                                          float norm_eps, int vec, int flags, int* __restrict__ ids, float* __restrict__ wts,
-                                                         const float* __restrict__ logit_bias) {
+                                                         const float* __restrict__ logit_bias, float scale) {
   pdl_launch();
   pdl_wait();
   extern __shared__ float sm[];
@@ -124,7 +127,8 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ x,
     __syncwarp();
   }
   if (groups > 1 && keep < groups) {
-    // a group is ranked by the sum of the top two shifted scores among its members; the `keep` best-ranked stay
+    // a group is ranked by the sum of the top two shifted scores among its members (flags bit 3: by the largest alone); the
+    // `keep` best-ranked stay
     const int per = E / groups;
     for (int g = lane; g < groups; g += 32) {
       float a = -INFINITY, b = -INFINITY;
@@ -137,7 +141,7 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ x,
           b = v;
         }
       }
-      gs[g] = per > 1 ? a + b : a;
+      gs[g] = per > 1 && !(flags & 8) ? a + b : a;
       ga[g] = 0.f;
     }
     __syncwarp();
@@ -188,16 +192,16 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ x,
     float sum = 0.f;
     for (int k = 0; k < top; ++k) sum += expf(my_w[k] - mx);
     __syncwarp();
-    for (int k = lane; k < top; k += 32) my_w[k] = expf(my_w[k] - mx) / sum;
+    for (int k = lane; k < top; k += 32) my_w[k] = expf(my_w[k] - mx) / sum * scale;
     return;
   }
-  if (flags & 2) return;  // the weights are the chosen scores as they are
-  const float inv = 1.f / (total + norm_eps);
+  if ((flags & 2) && scale == 1.f) return;  // the weights are the chosen scores as they are
+  const float inv = (flags & 2) ? scale : scale / (total + norm_eps);
   for (int k = lane; k < top; k += 32) my_w[k] *= inv;
 }
 
-// One CTA.  ids [P] -> order [P] (pairs by expert), tiles: (expert, first sorted row, rows) per tile of
-// tm rows, meta[0] = number of tiles.
+// One CTA.  ids [P] -> order [P] (pairs by expert, those of identity experts (ids from E on) left out), tiles: (expert, first
+// sorted row, rows) per tile of tm rows, meta[0] = number of tiles, meta[1] = pairs in the order.
 __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ ids, int P, int E, int tm, int* __restrict__ order,
                                                          int* __restrict__ tiles, int* __restrict__ meta) {
   pdl_launch();
@@ -208,7 +212,8 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ 
   int* tbase = off + E;   // [E]
   for (int e = threadIdx.x; e < E; e += blockDim.x) cnt[e] = 0;
   __syncthreads();
-  for (int p = threadIdx.x; p < P; p += blockDim.x) atomicAdd(&cnt[ids[p]], 1);
+  for (int p = threadIdx.x; p < P; p += blockDim.x)
+    if (ids[p] < E) atomicAdd(&cnt[ids[p]], 1);
   __syncthreads();
   if (threadIdx.x == 0) {
     int run = 0, t = 0;
@@ -219,6 +224,7 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ 
       t += (cnt[e] + tm - 1) / tm;
     }
     meta[0] = t;
+    meta[1] = run;
   }
   __syncthreads();
   for (int e = threadIdx.x; e < E; e += blockDim.x) {
@@ -234,7 +240,7 @@ __global__ void __launch_bounds__(1024) moe_sort_kernel(const int* __restrict__ 
   __syncthreads();
   for (int p = threadIdx.x; p < P; p += blockDim.x) {
     const int e = ids[p];
-    order[off[e] + atomicAdd(&cnt[e], 1)] = p;
+    if (e < E) order[off[e] + atomicAdd(&cnt[e], 1)] = p;
   }
 }
 
@@ -499,12 +505,12 @@ inline int mma_tile_rows(int P, int E) {
 }
 
 // xs[i, :] = x[order[i] / top, :]: the rows of the pairs in the order of the experts (16-byte copies), for a
-// product that wants an expert's rows side by side.
-__global__ void moe_gather_kernel(const bf16* __restrict__ x, long long x_stride, const int* __restrict__ order, int top, int P,
-                                  int W, bf16* __restrict__ xs) {
+// product that wants an expert's rows side by side; meta[1] of them.
+__global__ void moe_gather_kernel(const bf16* __restrict__ x, long long x_stride, const int* __restrict__ order,
+                                  const int* __restrict__ meta, int top, int W, bf16* __restrict__ xs) {
   pdl_launch();
   pdl_wait();
-  const int chunks = W / 8;
+  const int chunks = W / 8, P = meta[1];
   for (long long idx = (long long)blockIdx.x * blockDim.x + threadIdx.x; idx < (long long)P * chunks; idx += (long long)gridDim.x * blockDim.x) {
     const int i = (int)(idx / chunks), c = (int)(idx - (long long)i * chunks);
     const uint4 v = *reinterpret_cast<const uint4*>(x + (size_t)(order[i] / top) * x_stride + c * 8);
@@ -512,8 +518,11 @@ __global__ void moe_gather_kernel(const bf16* __restrict__ x, long long x_stride
   }
 }
 
+// With ids, a pair whose expert is E or beyond takes its token's row of x instead of a row of y (which then holds nothing).
+template <typename T>
 __global__ void moe_combine_kernel(float* __restrict__ resid, const float* __restrict__ y, const float* __restrict__ wts,
-                                   long long total, int W, int top) {
+                                   long long total, int W, int top, const int* __restrict__ ids, int E, const T* __restrict__ x,
+                                   long long x_stride) {
   pdl_launch();
   pdl_wait();
   if ((W & 3) == 0) {  // four columns a thread; each column's sum is the same chain over k as below
@@ -524,7 +533,13 @@ __global__ void moe_combine_kernel(float* __restrict__ resid, const float* __res
       float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
       for (int k = 0; k < top; ++k) {
         const float g = wts[n * top + k];
-        const float4 v = *reinterpret_cast<const float4*>(y + ((size_t)n * top + k) * W + c);
+        float4 v;
+        if (ids && ids[n * top + k] >= E) {
+          const T* own = x + (size_t)n * x_stride + c;
+          v = make_float4(to_float<T>(own[0]), to_float<T>(own[1]), to_float<T>(own[2]), to_float<T>(own[3]));
+        } else {
+          v = *reinterpret_cast<const float4*>(y + ((size_t)n * top + k) * W + c);
+        }
         s.x = fmaf(g, v.x, s.x);
         s.y = fmaf(g, v.y, s.y);
         s.z = fmaf(g, v.z, s.z);
@@ -544,7 +559,10 @@ __global__ void moe_combine_kernel(float* __restrict__ resid, const float* __res
     const long long n = idx / W;
     const int c = (int)(idx - n * W);
     float s = 0.f;
-    for (int k = 0; k < top; ++k) s = fmaf(wts[n * top + k], y[((size_t)n * top + k) * W + c], s);
+    for (int k = 0; k < top; ++k) {
+      const bool own = ids && ids[n * top + k] >= E;
+      s = fmaf(wts[n * top + k], own ? to_float<T>(x[(size_t)n * x_stride + c]) : y[((size_t)n * top + k) * W + c], s);
+    }
     resid[idx] += s;
   }
 }
@@ -596,7 +614,8 @@ int run_products<bf16>(const bf16* x, long long x_stride, const bf16* w_up, cons
 #define KVF_EXPERTS_API(SUF, T)                                                                                       \
   KVF_API int kvf_moe_route_##SUF(const void* x, long long x_stride, const float* router, const float* correction,    \
                                   int n_tokens, int W, int E, int top, int groups, int keep, float norm_eps,          \
-                                  int flags, int* ids, float* wts, const float* logit_bias, cudaStream_t st) {        \
+                                  int flags, int* ids, float* wts, const float* logit_bias, float scale,              \
+                                  cudaStream_t st) {                                                                  \
     if (n_tokens <= 0) return 0;                                                                                      \
     if (E <= 0 || top <= 0 || top > E || groups <= 0 || E % groups || keep <= 0 || keep > groups ||                   \
         top > keep * (E / groups))                                                                                    \
@@ -607,14 +626,16 @@ int run_products<bf16>(const bf16* x, long long x_stride, const bf16* w_up, cons
     const int vec = (W % 8 == 0) && (x_stride % 8 == 0) && ((((uintptr_t)x) | ((uintptr_t)router)) % 16 == 0);        \
     if (rt == 1)                                                                                                      \
       return launch(moe_route_kernel<T, 1>, dim3(n_tokens), dim3(256), smem, st, (const T*)x, x_stride, router,       \
-                    correction, n_tokens, W, E, top, groups, keep, norm_eps, vec, flags, ids, wts, logit_bias);       \
+                    correction, n_tokens, W, E, top, groups, keep, norm_eps, vec, flags, ids, wts, logit_bias,        \
+                    scale);                                                                                           \
     return launch(moe_route_kernel<T, 4>, dim3((n_tokens + 3) / 4), dim3(256), smem, st, (const T*)x, x_stride,       \
-                  router, correction, n_tokens, W, E, top, groups, keep, norm_eps, vec, flags, ids, wts, logit_bias); \
+                  router, correction, n_tokens, W, E, top, groups, keep, norm_eps, vec, flags, ids, wts, logit_bias,  \
+                  scale);                                                                                             \
   }                                                                                                                   \
   KVF_API int kvf_moe_experts_##SUF(const void* x, long long x_stride, const void* w_up, const void* w_down,          \
                                     const int* ids, const float* wts, int n_tokens, int W, int ff, int E, int top,    \
                                     int* order, int* tiles, int* meta, void* act, float* y, float* resid,             \
-                                    int act_kind, float act_limit, float act_alpha, float act_shift,                  \
+                                    int act_kind, float act_limit, float act_alpha, float act_shift, int identity,    \
                                     cudaStream_t st) {                                                                \
     if (n_tokens <= 0) return 0;                                                                                      \
     if (act_kind == ACT_GATED && (ff & 7)) return (int)cudaErrorInvalidValue; /* gate and up rows in blocks of 8 */   \
@@ -628,8 +649,8 @@ int run_products<bf16>(const bf16* x, long long x_stride, const bf16* w_up, cons
     const long long total = (long long)n_tokens * W;                                                                  \
     long long g = (total + 255) / 256;                                                                                \
     if (g > 148 * 16) g = 148 * 16;                                                                                   \
-    return launch(moe_combine_kernel, dim3((unsigned)g), dim3(256), 0, st, resid, (const float*)y, wts, total, W,     \
-                  top);                                                                                               \
+    return launch(moe_combine_kernel<T>, dim3((unsigned)g), dim3(256), 0, st, resid, (const float*)y, wts, total, W,  \
+                  top, identity ? ids : (const int*)nullptr, E, (const T*)x, x_stride);                               \
   }
 
 KVF_EXPERTS_API(f32, float)
@@ -642,19 +663,21 @@ KVF_API int kvf_moe_sort(const int* ids, int P, int E, int tm, int* order, int* 
   return launch(moe_sort_kernel, dim3(1), dim3(1024), (size_t)3 * E * sizeof(int), st, ids, P, E, tm, order, tiles, meta);
 }
 
-KVF_API int kvf_moe_gather_bf16(const void* x, long long x_stride, const int* order, int top, int P, int W, void* xs,
+KVF_API int kvf_moe_gather_bf16(const void* x, long long x_stride, const int* order, const int* meta, int top, int P, int W, void* xs,
                                 cudaStream_t st) {
   if (P <= 0) return 0;
   if ((W & 7) || (x_stride & 7) || ((((uintptr_t)x) | ((uintptr_t)xs)) & 15)) return (int)cudaErrorInvalidValue;
   long long g = ((long long)P * (W / 8) + 255) / 256;
   if (g > 148 * 16) g = 148 * 16;
-  return launch(moe_gather_kernel, dim3((unsigned)g), dim3(256), 0, st, (const bf16*)x, x_stride, order, top, P, W, (bf16*)xs);
+  return launch(moe_gather_kernel, dim3((unsigned)g), dim3(256), 0, st, (const bf16*)x, x_stride, order, meta, top, W, (bf16*)xs);
 }
 
-KVF_API int kvf_moe_combine(float* resid, const float* y, const float* wts, int n_tokens, int W, int top, cudaStream_t st) {
+// ids (null: every choice is an expert with weights), E, x: see moe_combine_kernel
+KVF_API int kvf_moe_combine_bf16(float* resid, const float* y, const float* wts, int n_tokens, int W, int top, const int* ids, int E,
+                                 const void* x, long long x_stride, cudaStream_t st) {
   const long long total = (long long)n_tokens * W;
   if (total <= 0) return 0;
   long long g = (total + 255) / 256;
   if (g > 148 * 16) g = 148 * 16;
-  return launch(moe_combine_kernel, dim3((unsigned)g), dim3(256), 0, st, resid, y, wts, total, W, top);
+  return launch(moe_combine_kernel<bf16>, dim3((unsigned)g), dim3(256), 0, st, resid, y, wts, total, W, top, ids, E, (const bf16*)x, x_stride);
 }

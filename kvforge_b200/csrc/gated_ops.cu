@@ -1,7 +1,7 @@
 // What a layer needs around its matrix products when every sublayer's result is gated, normed and only then
 // added to the residual stream, and when queries and keys are rotated and then normed per head:
 //
-//   norm_step    : resid += norm_post((y + y_bias) * sigmoid(z + b)) ; out = norm_next(resid)   (one pass over a row)
+//   norm_step    : resid += norm_post((y + y_bias) * sigmoid(z + b)) ; out = norm_next(resid) + next_b   (one pass over a row)
 //   qk_prepare   : rotation of split pairs, per-head RMS norm without a weight, keys and values to the cache
 //   unary_act    : xIELU, squared ReLU or tanh-GELU on the rows of an inner activation
 //
@@ -26,6 +26,7 @@ struct NormStepParams {
   const float* z_bias;     // [W] or null
   const float* post_w;     // weight of the norm of the gated result, or null: the result is added as it is
   const float* next_w;     // weight of the norm whose rows go to `out`, or null: `out` gets the stream itself
+  const float* next_b;     // [W] bias of that norm, or null
   void* out;               // [*, out_stride] storage type, or null
   long long out_stride;
   int W;
@@ -100,7 +101,8 @@ __global__ void __launch_bounds__(256) norm_step_kernel(const NormStepParams p) 
   if (p.next_w) row_stats(v, W, p.centred, p.eps, red, mean, rstd);
   T* o = p.out ? (T*)p.out + (size_t)r * p.out_stride : nullptr;
   for (int i = threadIdx.x; i < W; i += blockDim.x) {
-    const float x = p.next_w ? (v[i] - mean) * rstd * p.next_w[i] : v[i];
+    float x = p.next_w ? (v[i] - mean) * rstd * p.next_w[i] : v[i];
+    if (p.next_b) x += p.next_b[i];
     if (o) o[i] = from_float<T>(x);
     if (p.store_normed && !p.rows) h[i] = x;
   }
@@ -173,16 +175,17 @@ __global__ void __launch_bounds__(TH) norm_step_vec_kernel(const NormStepParams 
   const float* yp = p.y_parts ? p.y_parts + (size_t)src * W : nullptr;
   const T* z = (pending && p.z) ? (const T*)p.z + (size_t)src * p.z_stride : nullptr;
   bool live[NIT];
-  float hv[NIT][4], a[NIT][4], g[NIT][4], pw[NIT][4], nw[NIT][4];
+  float hv[NIT][4], a[NIT][4], g[NIT][4], pw[NIT][4], nw[NIT][4], nb[NIT][4];
 #pragma unroll
   for (int it = 0; it < NIT; ++it) {
     const int i = (it * TH + threadIdx.x) * 4;
     live[it] = i < W;
 #pragma unroll
-    for (int e = 0; e < 4; ++e) hv[it][e] = a[it][e] = g[it][e] = 0.f, pw[it][e] = nw[it][e] = 1.f;
+    for (int e = 0; e < 4; ++e) hv[it][e] = a[it][e] = g[it][e] = nb[it][e] = 0.f, pw[it][e] = nw[it][e] = 1.f;
     if (!live[it]) continue;
     Vec4<float>::load(h + i, hv[it]);
     if (p.next_w) Vec4<float>::load(p.next_w + i, nw[it]);
+    if (p.next_b) Vec4<float>::load(p.next_b + i, nb[it]);
     if (!pending) continue;
     if (y) Vec4<T>::load(y + i, a[it]);
     if (z) {
@@ -253,7 +256,7 @@ __global__ void __launch_bounds__(TH) norm_step_vec_kernel(const NormStepParams 
     const int i = (it * TH + threadIdx.x) * 4;
     float x[4];
 #pragma unroll
-    for (int e = 0; e < 4; ++e) x[e] = p.next_w ? (hv[it][e] - mean) * rstd * nw[it][e] : hv[it][e];
+    for (int e = 0; e < 4; ++e) x[e] = (p.next_w ? (hv[it][e] - mean) * rstd * nw[it][e] : hv[it][e]) + nb[it][e];
     if (o) Vec4<T>::store(o + i, x);
     if (p.store_normed && !p.rows) Vec4<float>::store(h + i, x);
   }
@@ -264,7 +267,7 @@ bool norm_step_vec_ok(const NormStepParams& p) {
   auto al = [](const void* q, size_t n) { return q == nullptr || ((uintptr_t)q % n) == 0; };
   constexpr size_t TB = 4 * sizeof(T);
   return p.W % 4 == 0 && p.W <= 4 * 256 * 4 && al(p.resid, 16) && al(p.y_parts, 16) && al(p.z_bias, 16) && al(p.y_bias, 16) && al(p.post_w, 16) &&
-         al(p.next_w, 16) && al(p.y, TB) && al(p.z, TB) && al(p.out, TB) && p.y_stride % 4 == 0 && p.z_stride % 4 == 0 &&
+         al(p.next_w, 16) && al(p.next_b, 16) && al(p.y, TB) && al(p.z, TB) && al(p.out, TB) && p.y_stride % 4 == 0 && p.z_stride % 4 == 0 &&
          p.out_stride % 4 == 0 && p.split_stride % 4 == 0;
 }
 
@@ -401,14 +404,14 @@ KVF_API int kvf_gated_set_pdl(int enabled) {
 #define KVF_GATED_API(SUF, T)                                                                                          \
   KVF_API int kvf_norm_step_##SUF(float* resid, const int* rows, const void* y, const float* y_parts, long long y_stride, \
                                   long long split_stride, int nsplit, const void* z, long long z_stride,              \
-                                  const float* z_bias, const float* y_bias, const float* post_w, const float* next_w, void* out, \
+                                  const float* z_bias, const float* y_bias, const float* post_w, const float* next_w, const float* next_b, void* out, \
                                   long long out_stride, int n_rows, int W, int centred, int store_normed, float eps,  \
                                   cudaStream_t st) {                                                                  \
     if (n_rows <= 0) return 0;                                                                                        \
-    if (W <= 0 || (y && y_parts) || (store_normed && rows)) return (int)cudaErrorInvalidValue;                        \
+    if (W <= 0 || (y && y_parts) || (store_normed && rows) || (next_b && !next_w)) return (int)cudaErrorInvalidValue;                        \
     NormStepParams p;                                                                                                 \
     p.resid = resid; p.rows = rows; p.y = y; p.y_parts = y_parts; p.y_stride = y_stride; p.split_stride = split_stride; \
-    p.nsplit = nsplit; p.z = z; p.z_stride = z_stride; p.z_bias = z_bias; p.y_bias = y_bias; p.post_w = post_w; p.next_w = next_w;       \
+    p.nsplit = nsplit; p.z = z; p.z_stride = z_stride; p.z_bias = z_bias; p.y_bias = y_bias; p.post_w = post_w; p.next_w = next_w; p.next_b = next_b; \
     p.out = out; p.out_stride = out_stride; p.W = W; p.centred = centred; p.store_normed = store_normed; p.eps = eps; \
     if (norm_step_vec_ok<T>(p)) {                                                                                     \
       /* few rows of slices in bfloat16: a thread for every four numbers, so that all slices of a row are asked for at once */ \

@@ -10,8 +10,9 @@ namespace {
 
 // ---------------------------------------------------------------- per-head norm, rotation, cache write
 // Rows of `qkv` hold nh query heads and nkv key heads of dk and nkv value heads of dv.  A warp owns
-// one (token, head).  Query and key heads: x <- x / sqrt(mean(x^2) + eps) * w (w of dk floats shared
-// by all heads; skipped without w), then the first `rot` dims turn by the angle pos * inv_freq[i], in
+// one (token, head).  Query and key heads: x <- x / sqrt(sum(x^2) / count + eps) * w (w of dk floats shared
+// by all heads; skipped without w; count: the numbers of a head that are not padding, padded places hold zeros), then the
+// first `rot` dims turn by the angle pos * inv_freq[i] and are multiplied by `magnitude`, in
 // interleaved pairs (2i, 2i+1) or, with split_pairs, in pairs (i, i + rot/2) (skipped when rot == 0).
 // Queries are written back in place; keys and values go to their slot of the paged cache
 // ([blocks][nkv][block_size][dk] and [...][dv]); a slot below zero (padding) is skipped, one beyond the
@@ -29,7 +30,7 @@ __global__ void __launch_bounds__(128) head_norm_cache_kernel(T* __restrict__ qk
                                                                int dv, int block_size, long long num_slots,
                                                                int* __restrict__ err, int split_pairs,
                                                                T* __restrict__ v_keep, const T* __restrict__ v_first,
-                                                               const float* __restrict__ v_lambda) {
+                                                               const float* __restrict__ v_lambda, float count, float magnitude) {
   pdl_launch();
   pdl_wait();
   const int heads = nh + 2 * nkv;
@@ -79,7 +80,7 @@ __global__ void __launch_bounds__(128) head_norm_cache_kernel(T* __restrict__ qk
     }
     ss = warp_sum(ss);
   }
-  const float r = w ? 1.f / sqrtf(ss / (float)dk + eps) : 1.f;
+  const float r = w ? 1.f / sqrtf(ss / count + eps) : 1.f;
   const float pos = (float)positions[n];
   T* dst = x;
   if (is_k) {
@@ -99,7 +100,7 @@ __global__ void __launch_bounds__(128) head_norm_cache_kernel(T* __restrict__ qk
       float sn, cs;
       sincosf(pos * inv_freq[i], &sn, &cs);
       float ya, yb;
-      rotate_pair(a, b, cs, sn, ya, yb);
+      rotate_pair(a, b, cs * magnitude, sn * magnitude, ya, yb);
       a = ya;
       b = yb;
     }
@@ -247,14 +248,15 @@ inline unsigned grid_for(long long total, int threads) {
                                         const int* slots, void* kcache, void* vcache, int n_tokens, int nh, int nkv, \
                                         int dk, int dv, int block_size, long long num_slots, int* err,               \
                                         int split_pairs, void* v_keep, const void* v_first, const float* v_lambda,   \
-                                        cudaStream_t st) {                                                           \
+                                        int count, float magnitude, cudaStream_t st) {                               \
     if (n_tokens <= 0) return 0;                                                                                     \
     if (dk <= 0 || (dk & 1) || rot < 0 || rot > dk || (rot & 1)) return (int)cudaErrorInvalidValue;                  \
-    if (v_first && !v_lambda) return (int)cudaErrorInvalidValue;                                                     \
+    if ((v_first && !v_lambda) || count <= 0 || count > dk) return (int)cudaErrorInvalidValue;                       \
     const long long units = (long long)n_tokens * (nh + 2 * nkv);                                                    \
     return launch(head_norm_cache_kernel<T>, dim3((unsigned)((units + 3) / 4)), dim3(128), 0, st, (T*)qkv,           \
                   row_stride, positions, q_w, k_w, eps, inv_freq, rot, slots, (T*)kcache, (T*)vcache, n_tokens, nh,  \
-                  nkv, dk, dv, block_size, num_slots, err, split_pairs, (T*)v_keep, (const T*)v_first, v_lambda);    \
+                  nkv, dk, dv, block_size, num_slots, err, split_pairs, (T*)v_keep, (const T*)v_first, v_lambda,     \
+                  (float)count, magnitude);                                                                          \
   }                                                                                                                  \
   KVF_API int kvf_row_rmsnorm_##SUF(const void* x, long long x_stride, const float* w, float eps, long long n_rows,  \
                                     int r, void* out, long long out_stride, cudaStream_t st) {                       \

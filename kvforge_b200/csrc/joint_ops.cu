@@ -2,7 +2,8 @@
 // heads and whose result is gated before the output projection; and a learned vector per position that joins the
 // residual stream after the embedding.
 //
-//   joint_norm_cache : biases, RMS norm over all query numbers and over all key numbers of a token, keys and values to the cache
+//   joint_norm_cache : biases, RMS norm over all query numbers and over all key numbers of a token, rotation, keys and values to
+//                      the cache
 //   output_gate      : out = mult * y * sigmoid(g), one gate a head or one a channel
 //   add_position_rows: resid[n] += table[position of n]
 //
@@ -47,7 +48,8 @@ template <> struct Pack<bf16, 4> {
 // comes from `y` (storage type) or, when `parts` is given, as the sum of nsplit float slices (slice order; row stride
 // `width`).  q and k become (x + bias) / sqrt(sum x^2 / count + eps) * w  with one sum over all of q and one over all of
 // k (`count`: the numbers of a head that are not padding; padded places hold zeros), without `qw` they are only
-// biased; v is only biased.  q goes back to `y` in place, k and v to the token's slot of the cache
+// biased; v is only biased.  Then the first `rot` numbers of every q and k head turn by the angle pos * inv_freq[i] and are
+// multiplied by `magnitude`, in interleaved pairs (2i, 2i+1) or in split pairs (i, i + rot/2) (rot == 0: none do).  q goes back to `y` in place, k and v to the token's slot of the cache
 // ([blocks][nkv][block_size][dk] and [...][dv]); with `parts` the rest goes to `y` as well.  A slot below zero (padding)
 // writes no key and no value, one beyond the pool raises bit 1 of the error flag.  One CTA a token.
 struct JointParams {
@@ -61,6 +63,10 @@ struct JointParams {
   const float* qw;    // [nh*dk] or null
   const float* kw;    // [nkv*dk]
   float q_count, k_count, eps;
+  const int* positions;
+  const float* inv_freq;  // [rot / 2]
+  int rot, interleaved;
+  float magnitude;
   const int* slots;
   void* kcache;
   void* vcache;
@@ -72,7 +78,7 @@ struct JointParams {
 template <typename T, int V>
 __global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParams p) {
   pdl_launch();
-  extern __shared__ __align__(16) float row[];  // q and k of the token
+  extern __shared__ __align__(16) float row[];  // q and k of the token, then the cosines and sines of its angles
   __shared__ float red[64];
   const int n = blockIdx.x;
   const int q_dim = p.nh * p.dk, k_dim = p.nkv * p.dk, v_dim = p.nkv * p.dv, qk = q_dim + k_dim;
@@ -94,6 +100,18 @@ __global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParam
       Pack<T, V>::load(y + c, f);
     }
   };
+  const int half = p.rot >> 1;
+  float* cs = row + qk;
+  float* sn = cs + half;
+  if (p.rot) {
+    const float pos = (float)p.positions[n];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
+      float s, c;
+      sincosf(pos * p.inv_freq[i], &s, &c);
+      cs[i] = c * p.magnitude;
+      sn[i] = s * p.magnitude;
+    }
+  }
   float sq = 0.f, sk = 0.f;
   for (int c = threadIdx.x * V; c < qk; c += blockDim.x * V) {
     float f[V];
@@ -126,6 +144,8 @@ __global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParam
     sk = warp_sum(lane < nw ? red[32 + lane] : 0.f);
     rq = 1.f / sqrtf(sq / p.q_count + p.eps);
     if (k_dim) rk = 1.f / sqrtf(sk / p.k_count + p.eps);
+  } else if (p.rot) {
+    __syncthreads();  // a pair's numbers and its angle may be another thread's
   }
   long long slot = -1;
   if (p.nkv) {
@@ -136,7 +156,7 @@ __global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParam
     }
   }
   const size_t page = slot >= 0 ? (size_t)(slot / p.block_size) : 0, place = slot >= 0 ? (size_t)(slot % p.block_size) : 0;
-  for (int c = threadIdx.x * V; c < qk; c += blockDim.x * V) {  // a thread reads what it wrote itself
+  for (int c = threadIdx.x * V; c < qk; c += blockDim.x * V) {  // nobody writes the row any more
     float f[V];
     Pack<float, V>::load(row + c, f);
     const bool is_q = c < q_dim;
@@ -146,6 +166,40 @@ __global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParam
       const float r = is_q ? rq : rk;
 #pragma unroll
       for (int e = 0; e < V; ++e) f[e] = f[e] * r * w[e];
+    }
+    const int j0 = c % p.dk;  // V numbers of one head from its j0 on
+    if (j0 < p.rot) {
+      const float* w = is_q ? p.qw : p.kw;
+      const int c_of_w = is_q ? c : c - q_dim;
+      const float r = is_q ? rq : rk;
+      if (V == 4 && p.interleaved && j0 + 4 <= p.rot) {  // whole pairs
+#pragma unroll
+        for (int e = 0; e < V; e += 2) {
+          float a, b;
+          const int i = (j0 + e) >> 1;
+          rotate_pair(f[e], f[(e + 1) % V], cs[i], sn[i], a, b);
+          f[e] = a;
+          f[(e + 1) % V] = b;
+        }
+      } else {
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          const int j = j0 + e;
+          if (j >= p.rot) continue;
+          const bool first = p.interleaved ? !(j & 1) : j < half;
+          const int d = p.interleaved ? (first ? 1 : -1) : (first ? half : -half);  // where the pair's other number is
+          const int i = p.interleaved ? j >> 1 : (first ? j : j - half);
+          float other = row[c + e + d];
+          if (p.qw) other = other * r * w[c_of_w + e + d];
+          const float own = p.qw ? row[c + e] * r * w[c_of_w + e] : row[c + e];
+          float a, b;
+          if (first)
+            rotate_pair(own, other, cs[i], sn[i], a, b);
+          else
+            rotate_pair(other, own, cs[i], sn[i], a, b);
+          f[e] = first ? a : b;
+        }
+      }
     }
     if (is_q) {
       Pack<T, V>::store(y + c, f);
@@ -183,7 +237,7 @@ int joint_norm_cache(const JointParams& p, int n_tokens, cudaStream_t st) {
   const bool vec = p.dk % 4 == 0 && p.dv % 4 == 0 && p.ldy % 4 == 0 && p.width % 4 == 0 && p.split_stride % 4 == 0 &&
                    al(p.y, 4 * sizeof(T)) && al(p.parts, 16) && al(p.bias, 16) && al(p.qw, 16) && al(p.kw, 16) &&
                    al(p.kcache, 4 * sizeof(T)) && al(p.vcache, 4 * sizeof(T));
-  const size_t smem = (size_t)(p.nh + p.nkv) * p.dk * sizeof(float);
+  const size_t smem = ((size_t)(p.nh + p.nkv) * p.dk + p.rot) * sizeof(float);
   if (smem > 200 * 1024) return (int)cudaErrorInvalidValue;
   auto kern = vec ? joint_norm_cache_kernel<T, 4> : joint_norm_cache_kernel<T, 1>;
   if (smem > 48 * 1024) {
@@ -254,16 +308,18 @@ KVF_API int kvf_joint_set_pdl(int enabled) {
 #define KVF_JOINT_API(SUF, T)                                                                                           \
   KVF_API int kvf_joint_norm_cache_##SUF(void* y, long long ldy, const float* parts, int nsplit, long long split_stride, \
                                          int width, const float* bias, const float* qw, const float* kw, int q_count,   \
-                                         int k_count, float eps, const int* slots, void* kcache, void* vcache,          \
+                                         int k_count, float eps, const int* positions, const float* inv_freq, int rot,  \
+                                         int interleaved, float magnitude, const int* slots, void* kcache, void* vcache, \
                                          int n_tokens, int nh, int nkv, int dk, int dv, int block_size,                 \
                                          long long num_slots, int* err, cudaStream_t st) {                              \
     if (n_tokens <= 0) return 0;                                                                                        \
     if (nh <= 0 || nkv < 0 || dk <= 0 || dv <= 0 || (nkv && (!slots || !kcache || !vcache || block_size <= 0)) ||       \
-        (parts && nsplit <= 0) || (qw && (q_count <= 0 || (nkv && (!kw || k_count <= 0)))))                             \
+        rot < 0 || rot > dk || (rot & 1) || (rot && (!positions || !inv_freq)) || (parts && nsplit <= 0) || (qw && (q_count <= 0 || (nkv && (!kw || k_count <= 0)))))                             \
       return (int)cudaErrorInvalidValue;                                                                                \
     JointParams p;                                                                                                      \
     p.y = y; p.ldy = ldy; p.parts = parts; p.nsplit = nsplit; p.split_stride = split_stride; p.width = width;           \
     p.bias = bias; p.qw = qw; p.kw = kw; p.q_count = (float)q_count; p.k_count = (float)k_count; p.eps = eps;           \
+    p.positions = positions; p.inv_freq = inv_freq; p.rot = rot; p.interleaved = interleaved; p.magnitude = magnitude;  \
     p.slots = slots; p.kcache = kcache; p.vcache = vcache; p.nh = nh; p.nkv = nkv; p.dk = dk; p.dv = dv;                \
     p.block_size = block_size; p.num_slots = num_slots; p.err = err;                                                    \
     return joint_norm_cache<T>(p, n_tokens, st);                                                                        \

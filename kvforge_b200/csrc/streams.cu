@@ -177,7 +177,8 @@ __global__ void replicate_kernel(const float* __restrict__ src, float* __restric
 
 // ---------------------------------------------------------------- mean of normed branches
 // out[n, :] = T( (1/nb) * sum_b rmsnorm(y_b[n, :]) * w_b[:] ) for the results y_b of nb mixers that read
-// the same input; a result is a tensor in the storage type or the float slices of a split-K product.
+// the same input; a result is a tensor in the storage type or the float slices of a split-K product.  With `resid` the mean
+// joins that float stream instead (resid[n, :] += ..., never rounded to T).
 constexpr int MAX_BRANCHES = 4;
 struct BranchParams {
   const void* y[MAX_BRANCHES];
@@ -188,6 +189,7 @@ struct BranchParams {
   int nb, W;
   float eps;
   void* out;
+  float* resid;
 };
 
 // A thread owns at most CPT columns of a row and keeps them in registers for every branch; all loads first.
@@ -248,7 +250,10 @@ __global__ void __launch_bounds__(256) branch_norm_mean_rows_kernel(const Branch
 #pragma unroll
     for (int b = 0; b < MAX_BRANCHES; ++b)
       if (b < p.nb) acc += v[b][k] * inv[b] * wv[b][k];
-    o[c] = from_float<T>(acc * share);
+    if (p.resid)
+      p.resid[n * W + c] += acc * share;
+    else
+      o[c] = from_float<T>(acc * share);
   }
 }
 
@@ -281,7 +286,10 @@ __global__ void __launch_bounds__(256) branch_norm_mean_kernel(const BranchParam
   for (int c = threadIdx.x; c < W; c += blockDim.x) {
     float acc = 0.f;
     for (int b = 0; b < p.nb; ++b) acc += rowbuf[(size_t)b * W + c] * inv[b] * p.w[b][c];
-    o[c] = from_float<T>(acc * share);
+    if (p.resid)
+      p.resid[n * W + c] += acc * share;
+    else
+      o[c] = from_float<T>(acc * share);
   }
 }
 
@@ -393,8 +401,9 @@ int launch_hc(const HcParams& p, int n_rows, int S, cudaStream_t st) {
   }                                                                                                                    \
   KVF_API int kvf_branch_norm_mean_##SUF(const void* const* y, const float* const* partials, const int* nsplit,        \
                                          const long long* split_stride, const float* const* w, int nb, long long N,    \
-                                         int W, float eps, void* out, cudaStream_t st) {                               \
+                                         int W, float eps, void* out, float* resid, cudaStream_t st) {                 \
     if (N <= 0) return 0;                                                                                              \
+    if ((out == nullptr) == (resid == nullptr)) return (int)cudaErrorInvalidValue;                                     \
     if (nb <= 0 || nb > MAX_BRANCHES || (size_t)nb * W * sizeof(float) > 160 * 1024) return (int)cudaErrorInvalidValue; \
     BranchParams p;                                                                                                    \
     for (int b = 0; b < nb; ++b) {                                                                                     \
@@ -402,7 +411,7 @@ int launch_hc(const HcParams& p, int n_rows, int S, cudaStream_t st) {
       p.w[b] = w[b];                                                                                                   \
       if (!p.y[b] && !p.partials[b]) return (int)cudaErrorInvalidValue;                                                \
     }                                                                                                                  \
-    p.nb = nb; p.W = W; p.eps = eps; p.out = out;                                                                      \
+    p.nb = nb; p.W = W; p.eps = eps; p.out = out; p.resid = resid;                                                     \
     if (W <= 8192) {                                                                                                   \
       const dim3 g((unsigned)N);                                                                                       \
       /* small CTAs, so that many rows share an SM and their loads overlap */                                          \
@@ -453,7 +462,7 @@ KVF_API int kvf_softcap_f32(float* x, long long n, float cap, cudaStream_t st) {
 
 // Turn programmatic dependent launch on or off for every launch of this library (its own flag: the flag is one
 // per shared library).
-KVF_API int kvf_mixers_set_pdl(int enabled) {
+KVF_API int kvf_streams_set_pdl(int enabled) {
   kvf::g_pdl_enabled = enabled ? 1 : 0;
   return 0;
 }

@@ -119,6 +119,8 @@ class StepContext:
     # The step's float residual stream [N, hidden], set by the model before its blocks run.  A mixer
     # or feed-forward may add its result into it directly and return ``ops.ADDED`` instead of a tensor.
     residual: torch.Tensor | None = None
+    # Room for the float slices of split products that a block hands on as one set (``parts.projection.SliceRow``).
+    slices: object | None = None
     # Upper bound on any context (fixes grid sizes of captured decode steps).
     context_bound: int = 0
     # Per registered tile size a ``QueryTiles``.  Empty when every sequence brings one token.

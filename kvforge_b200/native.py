@@ -38,9 +38,10 @@ LIBRARIES: dict[str, tuple[list[str], list[str]]] = {
     "noalloc": (["attention_decode_noalloc.cu"], []),
     # the short causal convolution of mixers with a running state
     "conv": (["causal_conv.cu"], []),
-    # what mixers with a running state, several residual streams and the general rotary form need; a
-    # library of its own, so that a model without them never compiles it
-    "mixers": (["sequence_mix_f32.cu", "sequence_mix_bf16.cu", "streams.cu"], []),
+    # the delta rule and its read-out; a library of its own, so that a model without them never compiles it
+    "mixers": (["sequence_mix_f32.cu", "sequence_mix_bf16.cu"], []),
+    # several residual streams, the mean of normed branches, the general rotary form, a soft cap on logits
+    "streams": (["streams.cu"], []),
     # attention layers with normed heads or latent keys and values, and the feed-forward of routed experts; a
     # library of its own for the same reason
     "routed": (["head_ops.cu", "experts.cu"], []),
@@ -53,6 +54,8 @@ LIBRARIES: dict[str, tuple[list[str], list[str]]] = {
     "decay": (["retention.cu", "state_space.cu", "tanh_norm.cu"], []),
     # attention whose queries and keys are normed as one vector and whose result is gated, learned positions
     "joint": (["joint_ops.cu"], []),
+    # a matrix memory with exponential gates
+    "memory": (["matrix_memory.cu"], []),
 }
 
 _loaded: dict[str, ctypes.CDLL] = {}

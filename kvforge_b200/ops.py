@@ -42,31 +42,32 @@ _SIGNATURES = {
     # library "conv"
     "kvf_causal_conv_{s}": "pippplppiiiiipiip",
     "kvf_conv_set_pdl": "i",
-    # library "mixers"
+    # libraries "mixers" and "streams"
     "kvf_gated_delta_{s}": "pppipipippiplpippiiiiiffiippppilp",
     "kvf_gated_head_norm_{s}": "pipipfiliipip",
     "kvf_hc_step_{s}": "pppilppppppiiifp",
-    "kvf_branch_norm_mean_{s}": "pppppilifpp",
+    "kvf_branch_norm_mean_{s}": "pppppilifppp",
     "kvf_rope_cache_general_{s}": "pipppppiiiiiiiilpp",
     "kvf_replicate_streams": "ppliip",
     "kvf_softcap_f32": "plfp",
     "kvf_mixers_set_pdl": "i",
+    "kvf_streams_set_pdl": "i",
     # library "routed"
-    "kvf_head_norm_cache_{s}": "plpppfpipppiiiiiilpipppp",
+    "kvf_head_norm_cache_{s}": "plpppfpipppiiiiiilpipppifp",
     "kvf_latent_prepare_{s}": "pliippfpipppiiiiiilpiplp",
     "kvf_row_rmsnorm_{s}": "plpfliplp",
     "kvf_head_gate_{s}": "pplliip",
     "kvf_add_row_f32": "pplip",
-    "kvf_moe_route_{s}": "plppiiiiiifipppp",
-    "kvf_moe_experts_{s}": "plppppiiiiippppppifffp",
+    "kvf_moe_route_{s}": "plppiiiiiifipppfp",
+    "kvf_moe_experts_{s}": "plppppiiiiippppppifffip",
     "kvf_moe_max_tiles": "ii",
     "kvf_moe_sort": "piiipppp",
-    "kvf_moe_gather_bf16": "plpiiipp",
-    "kvf_moe_combine": "pppiiip",
+    "kvf_moe_gather_bf16": "plppiiipp",
+    "kvf_moe_combine_bf16": "pppiiipiplp",
     "kvf_gemm_grouped_tcgen05_bf16": "pppiiiiiiipppipfffp",
     "kvf_routed_set_pdl": "i",
     # library "gated"
-    "kvf_norm_step_{s}": "pppplliplpppppliiiifp",
+    "kvf_norm_step_{s}": "pppplliplppppppliiiifp",
     "kvf_qk_prepare_{s}": "pliiippiifpppiiiiiilpp",
     "kvf_unary_act_{s}": "plplliippp",
     "kvf_talking_attention_{s}": "pppppppppiiiiiiiiiifiiiippp",
@@ -82,10 +83,15 @@ _SIGNATURES = {
     "kvf_state_space_{s}": "plplppplplppiliiiippppipp",
     "kvf_wide_norm_gate_{s}": "plpplipliipffliiplp",
     # library "joint"
-    "kvf_joint_norm_cache_{s}": "plpilipppiifpppiiiiiilpp",
+    "kvf_joint_norm_cache_{s}": "plpilipppiifppiifpppiiiiiilpp",
     "kvf_output_gate_{s}": "plplifpliiip",
     "kvf_add_position_rows_{s}": "pppiiipp",
     "kvf_joint_set_pdl": "i",
+    # library "memory"
+    "kvf_matrix_memory_{s}": "pliiifplilippfplplppiliiippppppipp",
+    "kvf_memory_read_{s}": "plpplpfliiplp",
+    "kvf_memory_columns": "i",
+    "kvf_memory_set_pdl": "i",
 }
 _CTYPES = {"p": ctypes.c_void_p, "i": ctypes.c_int, "l": ctypes.c_longlong, "f": ctypes.c_float}
 
@@ -167,7 +173,8 @@ def set_pdl(enabled: bool) -> None:
 # every shared library has a flag of its own; it follows the core's once the library is loaded
 _PDL_SETTERS = {
     "conv": "kvf_conv_set_pdl", "mixers": "kvf_mixers_set_pdl", "routed": "kvf_routed_set_pdl", "gated": "kvf_gated_set_pdl",
-    "talking": "kvf_talking_set_pdl", "decay": "kvf_decay_set_pdl", "joint": "kvf_joint_set_pdl",
+    "talking": "kvf_talking_set_pdl", "decay": "kvf_decay_set_pdl", "joint": "kvf_joint_set_pdl", "streams": "kvf_streams_set_pdl",
+    "memory": "kvf_memory_set_pdl",
 }  # fmt: skip
 _library_pdl: dict[str, bool] = {}
 
@@ -1136,6 +1143,7 @@ def splitmix64(z: int) -> int:
 # ------------------------------------------------------------------ mixers with a running state (library "mixers")
 
 MIXERS_LIB = "mixers"
+STREAMS_LIB = "streams"
 CONV_LIB = "conv"
 
 
@@ -1351,7 +1359,7 @@ def stream_step(
         raise ValueError("stream_step: fewer stream rows than output rows")
     name = f"kvf_hc_step_{s}"
     _check(
-        _fn(name, MIXERS_LIB)(
+        _fn(name, STREAMS_LIB)(
             _ptr(streams), yptr, pptr, nsplit, stride, _ptr(mix), _ptr(ow), _ptr(read), _ptr(norm_weight), _ptr(out), _ptr(rows),
             n_rows, num_streams, w, float(eps), _stream(),
         ),
@@ -1367,15 +1375,20 @@ def replicate_streams(src: torch.Tensor, streams: torch.Tensor, num_streams: int
     if tuple(streams.shape) != (n, num_streams * w):
         raise ValueError("replicate_streams: shapes do not agree")
     name = "kvf_replicate_streams"
-    _check(_fn(name, MIXERS_LIB)(_ptr(src), _ptr(streams), n, num_streams, w, _stream()), name)
+    _check(_fn(name, STREAMS_LIB)(_ptr(src), _ptr(streams), n, num_streams, w, _stream()), name)
 
 
-def branch_norm_mean(results: list, weights: list[torch.Tensor], eps: float, out: torch.Tensor) -> None:
+def branch_norm_mean(results: list, weights: list[torch.Tensor], eps: float, out: torch.Tensor, add: bool = False) -> None:
     """``out = T(mean_b rmsnorm(results[b]) * weights[b])`` over the model width: the results of
-    mixers that ran side by side on the same input (tensors in the storage type or ``Partials``)."""
-    s = _suffix(out.dtype)
-    _need(out, None, "out")
+    mixers that ran side by side on the same input (tensors in the storage type or ``Partials``).  ``add``: ``out`` is the float
+    residual stream and the mean is added to it."""
+    _need(out, torch.float32 if add else None, "out")
     n, w = out.shape
+    kinds = {y.dtype for y in results if not isinstance(y, Partials)} or {torch.float32 if add else out.dtype}
+    if len(kinds) > 1:
+        raise TypeError("branch_norm_mean: results must have one storage type")
+    (storage,) = kinds
+    s = _suffix(storage)
     nb = len(results)
     if not 0 < nb <= MAX_BRANCHES or len(weights) != nb:
         raise ValueError(f"branch_norm_mean: between 1 and {MAX_BRANCHES} branches, a weight each")
@@ -1392,19 +1405,19 @@ def branch_norm_mean(results: list, weights: list[torch.Tensor], eps: float, out
                 raise ValueError("branch_norm_mean: partials must be [S, N, W] with dense rows")
             ys[b], ps[b], ns[b], ss[b] = None, y.t.data_ptr(), y.nsplit, y.split_stride
         else:
-            _need(y, out.dtype, "branch result")
+            _need(y, storage if add else out.dtype, "branch result")
             if tuple(y.shape) != (n, w):
                 raise ValueError("branch_norm_mean: result shape")
             ys[b], ps[b], ns[b], ss[b] = y.data_ptr(), None, 0, 0
     name = f"kvf_branch_norm_mean_{s}"
-    _check(_fn(name, MIXERS_LIB)(ys, ps, ns, ss, ws, nb, n, w, float(eps), _ptr(out), _stream()), name)
+    _check(_fn(name, STREAMS_LIB)(ys, ps, ns, ss, ws, nb, n, w, float(eps), None if add else _ptr(out), _ptr(out) if add else None, _stream()), name)
 
 
 def softcap(logits: torch.Tensor, cap: float) -> None:
     """``logits <- cap * tanh(logits / cap)`` in place (float)."""
     _need(logits, torch.float32, "logits")
     name = "kvf_softcap_f32"
-    _check(_fn(name, MIXERS_LIB)(_ptr(logits), logits.numel(), float(cap), _stream()), name)
+    _check(_fn(name, STREAMS_LIB)(_ptr(logits), logits.numel(), float(cap), _stream()), name)
 
 
 def rope_cache_general(
@@ -1436,7 +1449,7 @@ def rope_cache_general(
         num_slots = kcache.shape[0] * block_size
     name = f"kvf_rope_cache_general_{s}"
     _check(
-        _fn(name, MIXERS_LIB)(
+        _fn(name, STREAMS_LIB)(
             _ptr(qkv), qkv.stride(0), _ptr(positions), _ptr(inv_freq), _ptr(slots), _ptr(kcache), _ptr(vcache), n, nh, nkv,
             dk, dv, rot, 1 if interleaved else 0, block_size, num_slots, _ptr(err), _stream(),
         ),
@@ -1464,6 +1477,7 @@ def head_norm_cache(
     inv_freq: torch.Tensor | None, slots: torch.Tensor | None, kcache: torch.Tensor | None, vcache: torch.Tensor | None,
     nh: int, nkv: int, dk: int, dv: int, block_size: int, err: torch.Tensor | None = None, interleaved: bool = True,
     v_keep: torch.Tensor | None = None, v_first: torch.Tensor | None = None, v_lambda: torch.Tensor | None = None,
+    count: int | None = None, magnitude: float = 1.0,
 ) -> None:  # fmt: skip
     """What follows the q/k/v product of an attention layer whose queries and keys are normed per
     head: rows of ``qkv`` hold ``nh`` query heads and ``nkv`` key heads of ``dk`` and ``nkv`` value heads
@@ -1473,7 +1487,8 @@ def head_norm_cache(
     (``None``: no rotation); queries in place, keys and values to ``slots`` of
     ``kcache [blocks, nkv, block_size, dk]`` / ``vcache [..., dv]``.  ``v_keep [N, nkv*dv]``: the values as projected
     are copied there as well (for later layers of the step).  ``v_first [N, nkv*dv]`` with ``v_lambda`` (a float
-    scalar on the device): the cached value is ``(1 - lambda) v + lambda v_first``."""
+    scalar on the device): the cached value is ``(1 - lambda) v + lambda v_first``.  ``count``: the numbers of a query or key
+    head that are not padding (default: all; padded places hold zeros).  ``magnitude``: what turned pairs are multiplied by."""
     s = _suffix(qkv.dtype)
     _rows2d(qkv, None, "qkv")
     n = qkv.shape[0]
@@ -1513,7 +1528,7 @@ def head_norm_cache(
         _fn(name, ROUTED_LIB)(
             _ptr(qkv), qkv.stride(0), _ptr(positions), _ptr(q_weight), _ptr(k_weight), float(eps), _ptr(inv_freq) if rot else None, rot,
             _ptr(slots), _ptr(kcache), _ptr(vcache), n, nh, nkv if slots is not None else 0, dk, dv, block_size, num_slots, _ptr(err),
-            0 if interleaved else 1, _ptr(v_keep), _ptr(v_first), _ptr(v_lambda) if v_first is not None else None, _stream(),
+            0 if interleaved else 1, _ptr(v_keep), _ptr(v_first), _ptr(v_lambda) if v_first is not None else None, int(count or dk), float(magnitude), _stream(),
         ),
         name,
     )  # fmt: skip
@@ -1599,7 +1614,7 @@ def moe_max_tiles(n_pairs: int, num_experts: int) -> int:
 def moe_route(
     x: torch.Tensor, router: torch.Tensor, correction: torch.Tensor | None, top: int, groups: int, keep: int, norm_eps: float,
     ids: torch.Tensor, weights: torch.Tensor, softmax: bool = False, normalize: bool = True, bias: torch.Tensor | None = None,
-    chosen_softmax: bool = False,
+    chosen_softmax: bool = False, group_rank: str = "top2", scale: float = 1.0,
 ) -> None:  # fmt: skip
     """Per token of ``x [N, W]``: logits ``router [E, W] x`` in float, scores ``s = sigmoid(z)``; the ``top``
     experts with the largest ``s + correction`` among the best ``keep`` of ``groups`` equal groups of
@@ -1608,7 +1623,8 @@ def moe_route(
     (``weights`` float ``[N, top]``).  ``softmax``: the scores are ``softmax(z)`` over all experts instead;
     ``normalize=False``: the weights are the chosen scores as they are.  ``bias`` (float ``[E]``) is added to the
     logits.  ``chosen_softmax``: the logits themselves rank the experts and the weights are a softmax over the chosen
-    logits alone (``softmax``, ``normalize`` and ``norm_eps`` then play no part)."""
+    logits alone (``softmax``, ``normalize`` and ``norm_eps`` then play no part).  ``group_rank``: ``"top2"`` as above, or ``"max"``
+    (a group's rank is its largest ``s + correction``).  ``scale``: the weights are multiplied by it."""
     s = _suffix(x.dtype)
     _rows2d(x, None, "x")
     _need(router, torch.float32, "router")
@@ -1628,10 +1644,12 @@ def moe_route(
     _need(weights, torch.float32, "weights")
     if tuple(ids.shape) != (n, top) or tuple(weights.shape) != (n, top):
         raise ValueError("moe_route: ids and weights must be [N, top]")
-    flags = 4 if chosen_softmax else (1 if softmax else 0) | (0 if normalize else 2)
+    if group_rank not in ("top2", "max"):
+        raise ValueError("moe_route: group_rank is 'top2' or 'max'")
+    flags = (4 if chosen_softmax else (1 if softmax else 0) | (0 if normalize else 2)) | (8 if group_rank == "max" else 0)
     name = f"kvf_moe_route_{s}"
     _check(
-        _fn(name, ROUTED_LIB)(_ptr(x), x.stride(0), _ptr(router), _ptr(correction), n, w, e, int(top), int(groups), int(keep), float(norm_eps), flags, _ptr(ids), _ptr(weights), _ptr(bias), _stream()),
+        _fn(name, ROUTED_LIB)(_ptr(x), x.stride(0), _ptr(router), _ptr(correction), n, w, e, int(top), int(groups), int(keep), float(norm_eps), flags, _ptr(ids), _ptr(weights), _ptr(bias), float(scale), _stream()),
         name,
     )
 
@@ -1657,7 +1675,7 @@ GROUPED_TCGEN05_MIN_ROWS = 64
 
 def moe_experts(
     x: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, ids: torch.Tensor, weights: torch.Tensor, scratch: dict, resid: torch.Tensor,
-    err: torch.Tensor | None = None, activation: str = "gelu", gated: GatedActivation | None = None,
+    err: torch.Tensor | None = None, activation: str = "gelu", gated: GatedActivation | None = None, identity: bool = False,
 ) -> None:  # fmt: skip
     """``resid[n] += sum_k weights[n, k] * w_down[e] act(w_up[e] x[n])`` with ``e = ids[n, k]`` and ``act`` the exact
     GELU (``"gelu"``) or the square of relu (``"relu2"``): the pairs are
@@ -1666,8 +1684,8 @@ def moe_experts(
     int32 ``[N*top]``, ``tiles`` int32 ``[3*max_tiles]``, ``meta`` int32 ``[4]``, ``act [N*top, ff]``, ``y`` float
     ``[N*top, W]``, and for many bfloat16 rows ``xs [N*top, W]`` (the pairs' rows side by side by expert).  With
     ``activation="gated"`` ``w_up`` is ``[E, 2*ff, W]``, gate and up rows alternating in blocks of 8, and ``gated`` says how
-    they are joined.  Four
-    launches, five through the tensor-memory product (``err``: the device flag its bounded waits raise)."""
+    they are joined.  ``identity``: ``ids`` may name outputs of the router beyond the last expert; such a choice's
+    result is ``x[n]`` itself.  Four launches, five through the tensor-memory product (``err``: the device flag its bounded waits raise)."""
     s = _suffix(x.dtype)
     if activation not in EXPERT_ACTIVATIONS:
         raise ValueError(f"moe_experts: activation {activation!r} is not one of {sorted(EXPERT_ACTIVATIONS)}")
@@ -1705,18 +1723,18 @@ def moe_experts(
         row_tiles = pairs // GROUPED_TILE_ROWS + e
         st = _stream()
         _check(_fn("kvf_moe_sort", ROUTED_LIB)(_ptr(ids), pairs, e, GROUPED_TILE_ROWS, _ptr(order), _ptr(tiles), _ptr(meta), st), "kvf_moe_sort")
-        _check(_fn("kvf_moe_gather_bf16", ROUTED_LIB)(_ptr(x), x.stride(0), _ptr(order), top, pairs, w, _ptr(xs), st), "kvf_moe_gather_bf16")
+        _check(_fn("kvf_moe_gather_bf16", ROUTED_LIB)(_ptr(x), x.stride(0), _ptr(order), _ptr(meta), top, pairs, w, _ptr(xs), st), "kvf_moe_gather_bf16")
         g = _fn("kvf_gemm_grouped_tcgen05_bf16")
         fl = (float(ga.limit), float(ga.alpha), float(ga.shift))
         _check(g(_ptr(xs), _ptr(w_up), _ptr(act), pairs, ff * (2 if is_gated else 1), w, e, w, ff, 1 + act_kind, _ptr(tiles), _ptr(meta), None, row_tiles, _ptr(err), *fl, st), "kvf_gemm_grouped_tcgen05_bf16")
         _check(g(_ptr(act), _ptr(w_down), _ptr(y), pairs, w, ff, e, ff, w, 0, _ptr(tiles), _ptr(meta), _ptr(order), row_tiles, _ptr(err), *fl, st), "kvf_gemm_grouped_tcgen05_bf16")
-        _check(_fn("kvf_moe_combine", ROUTED_LIB)(_ptr(resid), _ptr(y), _ptr(weights), n, w, top, st), "kvf_moe_combine")
+        _check(_fn("kvf_moe_combine_bf16", ROUTED_LIB)(_ptr(resid), _ptr(y), _ptr(weights), n, w, top, _ptr(ids) if identity else None, e, _ptr(x), x.stride(0), st), "kvf_moe_combine_bf16")
         return
     name = f"kvf_moe_experts_{s}"
     _check(
         _fn(name, ROUTED_LIB)(
             _ptr(x), x.stride(0), _ptr(w_up), _ptr(w_down), _ptr(ids), _ptr(weights), n, w, ff, e, top, _ptr(order), _ptr(tiles), _ptr(meta),
-            _ptr(act), _ptr(y), _ptr(resid), act_kind, float(ga.limit), float(ga.alpha), float(ga.shift), _stream(),
+            _ptr(act), _ptr(y), _ptr(resid), act_kind, float(ga.limit), float(ga.alpha), float(ga.shift), 1 if identity else 0, _stream(),
         ),
         name,
         4,
@@ -1761,13 +1779,14 @@ def norm_step(
     centred: bool = True,
     rows: torch.Tensor | None = None,
     store_normed: bool = False,
+    next_b: torch.Tensor | None = None,
 ) -> None:
     """One pass over every row of the float residual stream ``resid [N, W]``:
 
     * ``pending`` (``None``, ``ADDED``, a tensor, ``Partials``, ``Biased`` or a ``GatedWrite``) is gated, normed and added
       (the sum is written back unless ``rows`` picks rows);
-    * ``out`` (storage type, rows may be a view of a wider buffer) gets the row normed with ``next_w``
-      (``None``: the row itself); with ``store_normed`` the normed row also replaces the residual row.
+    * ``out`` (storage type, rows may be a view of a wider buffer) gets the row normed with ``next_w``, plus ``next_b`` if
+      given (``next_w=None``: the row itself); with ``store_normed`` the normed row also replaces the residual row.
 
     The norm is the layer norm ``(x - mean) / sqrt(var + eps) * w`` with the variance of the deviations
     (``centred``), or the RMS norm ``x / sqrt(mean(x^2) + eps) * w``."""
@@ -1822,6 +1841,10 @@ def norm_step(
         _need(next_w, torch.float32, "norm weight")
         if next_w.numel() != w:
             raise ValueError("norm_step: norm weight must have W entries")
+    if next_b is not None:
+        _need(next_b, torch.float32, "norm bias")
+        if next_b.numel() != w or next_w is None:
+            raise ValueError("norm_step: a norm's bias has W entries and goes with a weight")
     if rows is not None:
         _need(rows, torch.int32, "rows")
         if rows.numel() < n_rows:
@@ -1832,7 +1855,7 @@ def norm_step(
     _check(
         _fn(name, GATED_LIB)(
             _ptr(resid), _ptr(rows), yptr, pptr, ystride, sstride, nsplit, zptr, zstride,
-            _ptr(gw.z_bias) if gw else None, _ptr(y_bias), _ptr(gw.post_w) if gw else None, _ptr(next_w), optr, ostride,
+            _ptr(gw.z_bias) if gw else None, _ptr(y_bias), _ptr(gw.post_w) if gw else None, _ptr(next_w), _ptr(next_b), optr, ostride,
             n_rows, w, 1 if centred else 0, 1 if store_normed else 0, float(eps), _stream(),
         ),
         name,
@@ -2270,12 +2293,15 @@ JOINT_LIB = "joint"
 def joint_norm_cache(
     y: torch.Tensor, parts: Partials | None, bias: torch.Tensor | None, q_weight: torch.Tensor | None, k_weight: torch.Tensor | None,
     q_count: int, k_count: int, eps: float, slots: torch.Tensor | None, kcache: torch.Tensor | None, vcache: torch.Tensor | None,
-    nh: int, nkv: int, dk: int, dv: int, block_size: int, err: torch.Tensor | None = None,
+    nh: int, nkv: int, dk: int, dv: int, block_size: int, err: torch.Tensor | None = None, positions: torch.Tensor | None = None,
+    inv_freq: torch.Tensor | None = None, interleaved: bool = False, magnitude: float = 1.0,
 ) -> None:  # fmt: skip
     """What follows the input product of an attention layer whose query rows (and key rows) are normed as one vector.
     Rows hold ``q [nh*dk] | k [nkv*dk] | v [nkv*dv] | rest`` (``nkv == 0``: ``q | rest``): those of ``y`` (storage type), or the sum
     of the slices ``parts`` (``y`` then receives queries and rest).  ``bias`` (float, as wide as q, k and v together, or ``None``)
-    joins first; then ``q / sqrt(sum(q^2) / q_count + eps) * q_weight`` and the same for k (``q_weight=None``: no norm); queries
+    joins first; then ``q / sqrt(sum(q^2) / q_count + eps) * q_weight`` and the same for k (``q_weight=None``: no norm); then
+    (with ``inv_freq``) the first ``2*len(inv_freq)`` numbers of every query and key head turn with the position, in split pairs
+    ``(i, i + rot/2)`` or ``interleaved`` ones, and are multiplied by ``magnitude``; queries
     are written to ``y``, keys and values to ``slots`` of ``kcache [blocks, nkv, block_size, dk]`` / ``vcache [..., dv]``."""
     s = _suffix(y.dtype)
     _rows2d(y, None, "y")
@@ -2297,6 +2323,13 @@ def joint_norm_cache(
                 raise ValueError(f"joint_norm_cache: the {what} must have {size} entries")
     if q_weight is not None and nkv and k_weight is None:
         raise ValueError("joint_norm_cache: queries and keys are normed together or not at all")
+    rot = 0
+    if inv_freq is not None and inv_freq.numel():
+        _need(inv_freq, torch.float32, "inv_freq")
+        _need(positions, torch.int32, "positions")
+        rot = 2 * inv_freq.numel()
+        if rot > dk or positions.numel() < n:
+            raise ValueError("joint_norm_cache: more frequencies than dk/2, or too few positions")
     num_slots = 0
     if nkv:
         _need(slots, torch.int32, "slots")
@@ -2309,6 +2342,7 @@ def joint_norm_cache(
     _check(
         _fn(name, JOINT_LIB)(
             _ptr(y), y.stride(0), pptr, nsplit, stride, width, _ptr(bias), _ptr(q_weight), _ptr(k_weight), int(q_count), int(k_count), float(eps),
+            _ptr(positions) if rot else None, _ptr(inv_freq) if rot else None, rot, 1 if interleaved else 0, float(magnitude),
             _ptr(slots) if nkv else None, _ptr(kcache) if nkv else None, _ptr(vcache) if nkv else None, n, nh, nkv, dk, dv, block_size, num_slots,
             _ptr(err), _stream(),
         ),
@@ -2347,3 +2381,110 @@ def add_position_rows(resid: torch.Tensor, table: torch.Tensor, positions: torch
         raise ValueError("add_position_rows: shapes do not agree")
     name = f"kvf_add_position_rows_{s}"
     _check(_fn(name, JOINT_LIB)(_ptr(resid), _ptr(table), _ptr(positions), n, w, table.shape[0], _ptr(err), _stream()), name)
+
+
+# ------------------------------------------------------------------ library "memory"
+# a matrix memory with exponential gates
+
+MEMORY_LIB = "memory"
+MEMORY_MAX_KEY_DIM = RETENTION_MAX_KEY_DIM  # the same walk
+
+
+def memory_columns(dv: int) -> int:
+    """Columns of a head's state for values of ``dv`` numbers: ``dv`` of the matrix, one of the key sum, zeros up to a multiple of four."""
+    return (dv + 4) // 4 * 4
+
+
+def matrix_memory(
+    x: torch.Tensor, q_off: int, k_off: int, v_off: int, q_scale: float, logits: "torch.Tensor | Partials", f_off: int, i_bias: torch.Tensor,
+    f_bias: torch.Tensor, cap: float, state: torch.Tensor, out: torch.Tensor, floor: torch.Tensor, qsl: torch.Tensor, state_slots: torch.Tensor,
+    num_seqs: int, num_heads: int, dk: int, dv: int, scratch: tuple[torch.Tensor, ...] | None = None, max_query_len: int = 0,
+    raw: torch.Tensor | None = None,
+) -> None:  # fmt: skip
+    """A matrix memory with exponential gates over a flat batch, on each sequence's slot of the float ``state``
+    (``[heads, dk, memory_columns(dv)]``, then the heads' running maxima).  Rows of ``x`` hold ``H`` query heads of ``dk`` from column
+    ``q_off`` (multiplied by ``q_scale`` in float), key heads from ``k_off``, value heads of ``dv`` from ``v_off``; ``logits`` (float rows, or
+    ``Partials``) the input gates' logits from column 0 and the forget gates' from ``f_off``.  ``i = cap tanh((zi + i_bias) / cap)``,
+    ``f = logsigmoid(cap tanh((zf + f_bias) / cap))``, ``m <- max(f + m, i)``, ``S <- e^(f + m_before - m) S + e^(i - m) k v^T``, the key
+    sum likewise.  ``out`` (float ``[N, H*memory_columns(dv)]``) gets ``S^T q`` and, in column ``dv`` of a head, the key sum times q;
+    ``floor`` (float ``[N, H]``) gets ``e^(-m)``.  ``scratch``: float ``(decay [N, H], inflow [N, H], qn [N, H*dk], kn [N, H*dk], vn
+    [N, H*memory_columns(dv)])``; without it they are allocated here.  ``max_query_len``: the most rows a sequence brings (0 = unknown).
+    With ``raw`` (float scratch ``[N, H*64]``) the chunked form runs.  Two launches for single tokens, three otherwise, four in the chunked form."""
+    s = _suffix(x.dtype)
+    _rows2d(x, None, "x")
+    n, h, dvx = x.shape[0], int(num_heads), memory_columns(dv)
+    if not 0 < dk <= MEMORY_MAX_KEY_DIM or dv <= 0:
+        raise ValueError(f"matrix_memory: key heads of 1 to {MEMORY_MAX_KEY_DIM} numbers")
+    if max(q_off, k_off) + h * dk > x.shape[1] or v_off + h * dv > x.shape[1]:
+        raise ValueError("matrix_memory: the columns do not fit the rows")
+    if isinstance(logits, Partials):
+        z, nsplit, sstride = logits.t, logits.nsplit, logits.split_stride
+        _need(z, torch.float32, "gate logits", contiguous=False)
+        if z.shape[1] != n or z.stride(2) != 1:
+            raise ValueError("matrix_memory: slices of gate logits must be [S, N, *]")
+        ldz, width = z.stride(1), z.shape[2]
+    else:
+        z, nsplit, sstride = logits, 1, 0
+        _rows2d(z, torch.float32, "gate logits")
+        if z.shape[0] != n:
+            raise ValueError("matrix_memory: a row of gate logits per token")
+        ldz, width = z.stride(0), z.shape[1]
+    if f_off < h or f_off + h > width or not cap > 0:
+        raise ValueError("matrix_memory: the gates' columns do not fit, or the cap is not positive")
+    for t, what in ((i_bias, "input gate bias"), (f_bias, "forget gate bias")):
+        _need(t, torch.float32, what)
+        if t.numel() != h:
+            raise ValueError(f"matrix_memory: one {what} per head")
+    _rows2d(out, torch.float32, "out")
+    _need(floor, torch.float32, "floor")
+    if tuple(out.shape) != (n, h * dvx) or tuple(floor.shape) != (n, h):
+        raise ValueError("matrix_memory: out must be float [N, H*memory_columns(dv)], floor [N, H]")
+    sptr, sstr = _state_view(state, h * dk * dvx + h, "memory state")
+    _need(qsl, torch.int32, "query_start_loc")
+    _need(state_slots, torch.int32, "state_slots")
+    sizes = (h, h, h * dk, h * dk, h * dvx)
+    if scratch is None:
+        scratch = tuple(torch.empty((n, w), dtype=torch.float32, device=x.device) for w in sizes)
+    for t, w, what in zip(scratch, sizes, ("decay", "inflow", "qn", "kn", "vn")):
+        _need(t, torch.float32, f"scratch {what}")
+        if tuple(t.shape) != (n, w):
+            raise ValueError(f"matrix_memory: scratch {what} must be float [{n}, {w}]")
+    if raw is not None:
+        _check_chunks(raw, n, h, dk, dvx, state, out)
+    decay, inflow, qn, kn, vn = scratch
+    name = f"kvf_matrix_memory_{s}"
+    _check(
+        _fn(name, MEMORY_LIB)(
+            _ptr(x), x.stride(0), int(q_off), int(k_off), int(v_off), float(q_scale), _ptr(z), ldz, nsplit, sstride, int(f_off), _ptr(i_bias),
+            _ptr(f_bias), float(cap), sptr, sstr, _ptr(out), out.stride(0), _ptr(qsl), _ptr(state_slots), int(num_seqs), n, h, int(dk), int(dv),
+            _ptr(decay), _ptr(inflow), _ptr(floor), _ptr(qn), _ptr(kn), _ptr(vn), int(max_query_len), _ptr(raw), _stream(),
+        ),
+        name,
+        2 if max_query_len == 1 else 3 if raw is None else 4,
+    )  # fmt: skip
+
+
+def memory_read(o: torch.Tensor, floor: torch.Tensor, weight: torch.Tensor, eps: float, out: torch.Tensor, num_heads: int, dv: int, gate: torch.Tensor | None = None) -> None:
+    """What follows ``matrix_memory``: per token and head ``y = o[:dv] / (max(|o[dv]|, floor) + 1e-6)``, ``y / sqrt(mean(y^2) + eps)`` times
+    ``weight`` (float ``[H*dv]``) and ``sigmoid(gate)`` (storage type, ``None``: no gate), rounded once into ``out [N, H*dv]`` (gate and out may
+    be column ranges of wider rows)."""
+    s = _suffix(out.dtype)
+    _rows2d(o, torch.float32, "o")
+    _rows2d(out, None, "out")
+    _need(floor, torch.float32, "floor")
+    _need(weight, torch.float32, "norm weight")
+    n, h = o.shape[0], int(num_heads)
+    if o.shape[1] != h * memory_columns(dv) or tuple(out.shape) != (n, h * dv) or tuple(floor.shape) != (n, h) or weight.numel() != h * dv:
+        raise ValueError("memory_read: shapes do not agree")
+    if gate is not None:
+        _rows2d(gate, out.dtype, "gate")
+        if tuple(gate.shape) != (n, h * dv):
+            raise ValueError("memory_read: gate shape")
+    name = f"kvf_memory_read_{s}"
+    _check(
+        _fn(name, MEMORY_LIB)(
+            _ptr(o), o.stride(0), _ptr(floor), _ptr(gate), gate.stride(0) if gate is not None else 0, _ptr(weight), float(eps), n, h, int(dv),
+            _ptr(out), out.stride(0), _stream(),
+        ),
+        name,
+    )  # fmt: skip

@@ -1,10 +1,10 @@
 """The parts a model is put together from.  Importing the package registers the built-in
 ones (token embedding, rotary encoding, RMSNorm over one or several residual streams, paged
-attention, gated attention, latent attention, the gated delta rule, retention, the state space, mixers side by side, gated
+attention, gated attention, latent attention, the gated delta rule, retention, the state space, the matrix memory, mixers side by side, gated
 and plain feed-forward, routed experts, the pre-norm block over one or several streams, the post-norm, parallel and sandwich
 blocks, linear head)."""
 
-from . import attention, block, delta, embedding, experts, gated_attention, head, latent, mlp, norm, parallel, retention, rope, state_space, talking  # noqa: F401  (registration)
+from . import attention, block, delta, embedding, experts, gated_attention, head, latent, matrix_memory, mlp, norm, parallel, retention, rope, state_space, talking  # noqa: F401  (registration)
 from .base import (  # noqa: F401
     CacheNeed,
     LayerCache,

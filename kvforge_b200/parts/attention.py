@@ -70,6 +70,15 @@ def decode_scratch(rt, ctx, nh: int, nkv: int, d: int, dv: int, tickets: torch.T
     return (acc, ml, tickets), reach, split
 
 
+def pad_head_rows(t: torch.Tensor, heads: int, size: int, padded: int) -> torch.Tensor:
+    """Rows (or entries) of ``heads`` heads of ``size``, each followed by zeros up to ``padded``."""
+    if size == padded:
+        return t
+    out = torch.zeros((heads, padded, *t.shape[1:]), dtype=t.dtype, device=t.device)
+    out[:, :size] = t.reshape(heads, size, *t.shape[1:])
+    return out.reshape(heads * padded, *t.shape[1:])
+
+
 @register_mixer("paged_attention")
 class PagedAttention(Mixer):
     """params: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``; optional
@@ -85,7 +94,10 @@ class PagedAttention(Mixer):
     scores by ``distance_buckets`` of the distance between query and key), ``keep_first`` (with a
     window: the first keys of a sequence that every later query sees, at their true positions),
     ``softcap`` (``c``: a scaled score ``s`` becomes ``c * tanh(s / c)``), ``sink`` (true: the tensor ``sink [num_heads]``;
-    ``exp(sink_h)`` joins the softmax's denominator of head ``h`` without a key or a value) and ``value_mix``
+    ``exp(sink_h)`` joins the softmax's denominator of head ``h`` without a key or a value; ``"zero"``: a sink whose score is 0 in every
+    head, so one joins the denominator, and no tensor), ``keep_window`` (the cache keeps at least so many keys because a later
+    layer that reads it sees them), ``pad_heads`` (heads whose size is no multiple of 8 are padded with zeros when the tensors are bound:
+    that changes neither a norm's sum nor a score nor, through zero columns of the output projection, the result) and ``value_mix``
     (``"source"``: the values as projected are also kept for the later layers of the step; ``"mix"``: the values become
     ``(1 - lambda) v + lambda v_source`` with the source layer's values of the same token, before they are cached;
     both declare the scalar tensor ``vmix``, which only ``"mix"`` uses; source and mixing layers have values of one shape).
@@ -94,14 +106,18 @@ class PagedAttention(Mixer):
     of the Llama decoder; anything else (interleaved pairs, a value size of its own, a convolution,
     normed heads, a bias, kept first keys) goes through ``forward_general``: one product, the
     convolution, the rotary kernel (or the one that also norms the heads), and the attention kernel
-    that takes the shape."""
+    that takes the shape.  The general form without a convolution and carried values also has the open form that mixers side by
+    side take: ``take_input`` / ``take_output`` hand the input and output matrices over, ``mix`` computes what lies between the two products."""
 
     def __init__(self, params, prefix=""):
         super().__init__(params, prefix)
         self.hidden = int(params["hidden_size"])
         self.nh = int(params["num_heads"])
         self.nkv = int(params["num_kv_heads"])
-        self.d = int(params["head_dim"])
+        self.d = self.d_true = int(params["head_dim"])
+        self.dv = self.dv_true = int(params.get("v_head_dim") or self.d)
+        if params.get("pad_heads"):
+            self.d, self.dv = -(-self.d // 8) * 8, -(-self.dv // 8) * 8
         if self.nkv <= 0 or self.nh % self.nkv:
             raise ValueError("num_heads must be a multiple of num_kv_heads")
         ops.check_head_dim(self.d)
@@ -111,13 +127,12 @@ class PagedAttention(Mixer):
         self.chunk = params.get("chunk")
         if self.chunk is not None and (int(self.chunk) <= 0 or self.window is not None):
             raise ValueError("chunk must be positive, and does not go with a window")
-        self.scale = float(params.get("scale") or 1.0 / math.sqrt(self.d))  # model.py:74
+        self.scale = float(params.get("scale") or 1.0 / math.sqrt(self.d_true))  # model.py:74
         pos = params.get("position")
         if isinstance(pos, dict):
             pos = PartSpec(pos["kind"], pos.get("params", {}))
         self.position_spec: PartSpec | None = pos
         self.position = None  # shared instance, set by the model before bind
-        self.dv = int(params.get("v_head_dim") or self.d)
         ops.check_head_dim(self.dv)
         self.taps = int(params.get("conv") or 0)
         if self.taps < 0:
@@ -132,7 +147,13 @@ class PagedAttention(Mixer):
         self.softcap = float(params.get("softcap") or 0.0)
         if self.softcap < 0:
             raise ValueError("softcap must be positive")
-        self.has_sink = bool(params.get("sink", False))
+        self.sink = params.get("sink") or False
+        if self.sink not in (False, True, "zero"):
+            raise ValueError("sink is true, false or 'zero'")
+        self.has_sink = bool(self.sink)
+        self.keep_window = int(params.get("keep_window") or 0)
+        if self.keep_window and self.window is None:
+            raise ValueError("keep_window goes with a window")
         self.value_mix = params.get("value_mix")
         if self.value_mix not in (None, "source", "mix"):
             raise ValueError("value_mix is 'source', 'mix' or None")
@@ -160,7 +181,7 @@ class PagedAttention(Mixer):
             out["k_norm.weight"] = WeightDecl((d,), kind="vector", init="ones")
         if params.get("distance_bias"):
             out["rel"] = WeightDecl((int(params["distance_bias"]["rows"]), nh), kind="vector", init="small")
-        if params.get("sink"):
+        if params.get("sink") is True:
             out["sink"] = WeightDecl((nh,), kind="vector", init="small")
         if params.get("value_mix"):
             out["vmix"] = WeightDecl((), kind="vector", init="unit")
@@ -172,13 +193,21 @@ class PagedAttention(Mixer):
             return CacheNeed("chunk", self.nkv, self.d, int(self.chunk), v)
         if self.window is None:
             return CacheNeed("full", self.nkv, self.d, None, v)
-        return CacheNeed("window", self.nkv, self.d, int(self.window), v, keep_first=self.keep_first)
+        return CacheNeed("window", self.nkv, self.d, max(int(self.window), self.keep_window), v, keep_first=self.keep_first)
 
     def state_shape(self):
         return ((self.taps - 1) * self.qkv_dim,) if self.taps > 1 else None
 
     def bind(self, weights, rt):
         super().bind(weights, rt)
+        if (self.d, self.dv) != (self.d_true, self.dv_true):
+            if self.taps or self.value_mix is not None:
+                raise ValueError("padded heads go with neither a convolution nor mixed values")
+            weights = dict(weights)
+            for name, heads, true, padded in (("q_proj.weight", self.nh, self.d_true, self.d), ("k_proj.weight", self.nkv, self.d_true, self.d), ("v_proj.weight", self.nkv, self.dv_true, self.dv), ("q_norm.weight", 1, self.d_true, self.d), ("k_norm.weight", 1, self.d_true, self.d)):
+                if name in weights:
+                    weights[name] = pad_head_rows(weights[name], heads, true, padded)
+            weights["o_proj.weight"] = pad_head_rows(weights["o_proj.weight"].t().contiguous(), self.nh, self.dv_true, self.dv).t()
         self.w_qkv = torch.cat([weights["q_proj.weight"], weights["k_proj.weight"], weights["v_proj.weight"]], dim=0).contiguous()
         self.w_o = weights["o_proj.weight"].contiguous()
         self.w_conv = None
@@ -187,19 +216,27 @@ class PagedAttention(Mixer):
         self.q_norm_w = weights.get("q_norm.weight") if self.qk_eps is not None else None
         self.k_norm_w = weights.get("k_norm.weight") if self.qk_eps is not None else None
         bias = ops.DistanceBias(weights["rel"].contiguous(), distance_buckets(*self.bias_shape).to(rt.device)) if self.bias_shape is not None else None
-        sinks = weights["sink"].contiguous() if self.has_sink else None
+        sinks = None
+        if self.has_sink:
+            sinks = weights["sink"].contiguous() if self.sink is True else torch.zeros(self.nh, dtype=torch.float32, device=rt.device)
         self.v_lambda = weights["vmix"].reshape(1).contiguous() if self.value_mix == "mix" else None
         self._bind_attention(bias, sinks)
-        if self.position_spec is not None and self.position is None:
-            self.position = build_part("position", self.position_spec)
-            self.position.bind({}, rt)
-        table = self.position.table() if self.position is not None else None
-        # no table: q and k are stored and used as the projections leave them
-        self.inv_freq = table if table is not None else torch.empty(0, dtype=torch.float32, device=rt.device)
-        self.interleaved = bool(getattr(self.position, "pairs_interleaved", False))
+        self._bind_position()
+        if self.magnitude != 1.0 and self.qk_eps is None:
+            raise ValueError("a rotation that changes the size of what it turns goes with normed heads")
         self.general = (
             bool(self.taps) or self.dv != self.d or self.interleaved or self.qk_eps is not None or not self.plain_scores or self.value_mix is not None
         )
+
+    def _bind_position(self) -> None:
+        if self.position_spec is not None and self.position is None:
+            self.position = build_part("position", self.position_spec)
+            self.position.bind({}, self.rt)
+        table = self.position.table() if self.position is not None else None
+        # no table: q and k are stored and used as the projections leave them
+        self.inv_freq = table if table is not None else torch.empty(0, dtype=torch.float32, device=self.rt.device)
+        self.interleaved = bool(getattr(self.position, "pairs_interleaved", False))
+        self.magnitude = self.position.magnitude if self.position is not None else 1.0
 
     def _bind_attention(self, bias=None, sinks=None) -> None:
         """What the attention kernels themselves need, whatever comes before and after them."""
@@ -267,13 +304,38 @@ class PagedAttention(Mixer):
     def forward_general(self, ctx, x: torch.Tensor, cache):
         rt = self.rt
         n = x.shape[0]
-        if not cache.writable:
-            raise RuntimeError("a mixer in the general form keeps its own keys and values")
         qkv = rt.buf("attn.qkv", n, self.qkv_dim)
         if ops.skinny_ok(x, self.w_qkv):
             ops.gemm_skinny(x, self.w_qkv, qkv)
         else:
             ops.linear(x, self.w_qkv, qkv)
+        out = rt.buf("attn.out", n, self.o_dim)
+        self.mix(ctx, qkv, cache, out)
+        return project(rt, "attn.proj", out, self.w_o, ctx)
+
+    inner_width = property(lambda self: self.o_dim)
+
+    @property
+    def open_form(self) -> bool:
+        return self.general and not self.taps and self.value_mix is None
+
+    def take_input(self) -> torch.Tensor:
+        w, self.w_qkv = self.w_qkv, None
+        return w
+
+    def take_output(self) -> torch.Tensor:
+        w, self.w_o = self.w_o, None
+        return w
+
+    def mix(self, ctx, qkv: torch.Tensor, cache, out: torch.Tensor, mult: float = 1.0) -> None:
+        """From the input product's rows (a column range of wider rows is fine where there is no convolution) to what the output
+        projection multiplies, ``out [N, inner_width]``."""
+        if mult != 1.0:
+            raise RuntimeError("attention without a gate does not scale its result")
+        rt = self.rt
+        n = qkv.shape[0]
+        if not cache.writable:
+            raise RuntimeError("a mixer in the general form keeps its own keys and values")
         if self.taps:
             mixed = rt.buf("attn.qkv_conv", n, self.qkv_dim)
             ops.causal_conv(qkv, self.w_conv, cache.state, ctx.query_start_loc, ctx.state_slots, ctx.num_seqs, mixed, max_query_len=ctx.max_query_len)
@@ -285,15 +347,14 @@ class PagedAttention(Mixer):
                 qkv, ctx.positions, self.q_norm_w, self.k_norm_w, self.qk_eps or 0.0, self.inv_freq, ctx.slot_mappings[cache.group], cache.k, cache.v,
                 self.nh, self.nkv, self.d, self.dv, ctx.block_size, rt.err, interleaved=self.interleaved,
                 v_keep=carried if self.value_mix == "source" else None, v_first=carried if self.value_mix == "mix" else None, v_lambda=self.v_lambda,
+                count=self.d_true, magnitude=self.magnitude,
             )  # fmt: skip
         else:
             ops.rope_cache_general(
                 qkv, ctx.positions, self.inv_freq, self.interleaved, ctx.slot_mappings[cache.group], cache.k, cache.v,
                 self.nh, self.nkv, self.d, self.dv, ctx.block_size, rt.err,
             )  # fmt: skip
-        out = rt.buf("attn.out", n, self.o_dim)
-        self.attend(ctx, qkv, self.qkv_dim, out, cache)
-        return project(rt, "attn.proj", out, self.w_o, ctx)
+        self.attend(ctx, qkv, qkv.stride(0), out, cache)
 
     def attend(self, ctx, q, q_stride, out, cache) -> None:
         scratch, bound, split = None, None, 256

@@ -87,7 +87,8 @@ class CacheNeed:
         """Whether a mixer with the need ``other`` can read a cache kept for this one: keys and values of one shape, and
         every key that it may see is still there."""
         same = (self.kv_heads, self.head_dim, self.value_dim, self.v_in_k) == (other.kv_heads, other.head_dim, other.value_dim, other.v_in_k)
-        return same and (self.kind == "full" or self.group_key == other.group_key)
+        wider = self.kind == other.kind == "window" and self.window >= other.window and self.keep_first >= other.keep_first
+        return same and (self.kind == "full" or wider or self.group_key == other.group_key)
 
 
 @dataclass
@@ -142,6 +143,9 @@ class Part:
 
 
 class PositionEncoding(Part):
+    # what a mixer that turns q and k multiplies the turned pairs by (some scalings of the frequencies come with one)
+    magnitude = 1.0
+
     def table(self) -> torch.Tensor | None:
         """Float frequencies ``[rot/2]`` for a mixer that turns q and k, or ``None``."""
         return None

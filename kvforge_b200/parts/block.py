@@ -10,6 +10,7 @@ from __future__ import annotations
 
 from .. import ops
 from .base import Block, PartSpec, WeightDecl, build_part, register_block
+from .projection import SliceRow
 
 
 def _spec(v) -> PartSpec:
@@ -83,8 +84,9 @@ class ParallelBlock(Block):
     ``mixer_name``, ``ffn_name`` under the layer's prefix.
 
     Nothing reads the residual stream between the norm and the next layer's norm, so either part may
-    add its result straight into the stream (``ops.ADDED``); of two results that are still pending
-    one is added here and the other is handed to the next norm."""
+    add its result straight into the stream (``ops.ADDED``); the float slices of two split products come to lie
+    one behind the other and are handed to the next norm as one set; of two other results that are still pending
+    one is added here and the other is handed on."""
 
     def __init__(self, params, prefix=""):
         super().__init__(params, prefix)
@@ -102,10 +104,16 @@ class ParallelBlock(Block):
 
     def forward(self, ctx, resid, delta, cache):
         x = self.norm.forward(ctx, resid, delta)
-        a = self.mixer.forward(ctx, x, cache)
         if self.ffn is None:
-            return a
-        f = self.ffn.forward(ctx, x)
+            return self.mixer.forward(ctx, x, cache)
+        ctx.slices = slices = SliceRow(self.norm.rt, resid.shape[1])
+        try:
+            a = self.mixer.forward(ctx, x, cache)
+            f = self.ffn.forward(ctx, x)
+        finally:
+            ctx.slices = None
+        if slices.holds(a) and slices.holds(f):
+            return slices.all()
         if a is ops.ADDED or a is None:
             return f
         if f is ops.ADDED or f is None:

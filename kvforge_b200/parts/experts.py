@@ -10,6 +10,9 @@ of its own that every token passes, may be added to the sum.
 A router may add a bias to its logits (``z = W_router x + b``), and its weights may be a softmax over the chosen
 logits alone (the logits then rank the experts).  A gated expert is ``W_down[e] join(W_gate[e] x, W_up[e] x)`` with
 ``join(g, u) = g' sigmoid(alpha g') (u' + shift)``, ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)``.
+
+The router may have more outputs than there are experts: the last ones are identity experts, which have no tensors and whose
+result is the input itself.
 """
 
 from __future__ import annotations
@@ -34,9 +37,11 @@ class RoutedExperts(FeedForward):
     that runs for every token and is added; its tensors lie under ``shared.``); ``score: "chosen_softmax"`` (the
     logits rank the experts, the weights are a softmax over the chosen logits alone); ``router_bias`` (true: the
     tensor ``router.b [E]`` is added to the logits); ``activation: "gated"`` with ``gated: {"limit": l, "alpha": a,
-    "shift": s}`` (each optional; the defaults make SwiGLU): an expert then also has ``e<i>.gate [ff, W]``.
+    "shift": s}`` (each optional; the defaults make SwiGLU): an expert then also has ``e<i>.gate [ff, W]``; ``identity`` (how many identity
+    experts follow the ``experts``; router, correction and groups are over both), ``group_rank`` (``"top2"``, the default, or ``"max"``: a
+    group is ranked by its largest shifted score) and ``weight_scale`` (the chosen weights are multiplied by it).
 
-    Tensors: ``router [E, W]``, ``correction [E]``, ``e<i>.up [ff, W]``, ``e<i>.down [W, ff]``."""
+    Tensors: ``router [E + identity, W]``, ``correction [E + identity]``, ``e<i>.up [ff, W]``, ``e<i>.down [W, ff]``."""
 
     def __init__(self, params, prefix=""):
         super().__init__(params, prefix)
@@ -63,19 +68,28 @@ class RoutedExperts(FeedForward):
         if isinstance(shared, dict):
             shared = PartSpec(shared["kind"], shared.get("params", {}))
         self.shared = build_part("ffn", shared, prefix + "shared.") if shared is not None else None
-        if not 0 < self.top <= self.experts or self.experts % self.groups or not 0 < self.keep <= self.groups:
+        self.identity = int(p.get("identity") or 0)
+        self.group_rank = p.get("group_rank", "top2")
+        if self.group_rank not in ("top2", "max"):
+            raise ValueError("group_rank must be 'top2' or 'max'")
+        self.weight_scale = float(p.get("weight_scale", 1.0))
+        self.choices = self.experts + self.identity  # what the router has outputs for
+        if self.experts <= 0 or self.identity < 0:
+            raise ValueError("experts must be positive, identity a count")
+        if not 0 < self.top <= self.choices or self.choices % self.groups or not 0 < self.keep <= self.groups:
             raise ValueError("experts must divide into the groups, and top and keep must be within their counts")
-        if self.top > self.keep * (self.experts // self.groups):
+        if self.top > self.keep * (self.choices // self.groups):
             raise ValueError("the groups that stay hold fewer experts than a token uses")
 
     @classmethod
     def weight_decls(cls, params):
         w, e, ff = int(params["hidden_size"]), int(params["experts"]), int(params["intermediate_size"])
-        out = {"router": WeightDecl((e, w), kind="vector", init="normal")}
+        choices = e + int(params.get("identity") or 0)
+        out = {"router": WeightDecl((choices, w), kind="vector", init="normal")}
         if params.get("correction", True):
-            out["correction"] = WeightDecl((e,), kind="vector", init="zeros")
+            out["correction"] = WeightDecl((choices,), kind="vector", init="zeros")
         if params.get("router_bias"):
-            out["router.b"] = WeightDecl((e,), kind="vector", init="zeros")
+            out["router.b"] = WeightDecl((choices,), kind="vector", init="zeros")
         for i in range(e):
             if params.get("activation") == "gated":
                 out[f"e{i}.gate"] = WeightDecl((ff, w))
@@ -124,7 +138,7 @@ class RoutedExperts(FeedForward):
         wts = rt.buf("experts.weights", n, top, torch.float32)
         ops.moe_route(
             x, self.router, self.correction, top, self.groups, self.keep, WEIGHT_SUM_EPS, ids, wts, self.score == "softmax", self.normalize,
-            bias=self.bias, chosen_softmax=self.score == "chosen_softmax",
+            bias=self.bias, chosen_softmax=self.score == "chosen_softmax", group_rank=self.group_rank, scale=self.weight_scale,
         )  # fmt: skip
         scratch = {
             "order": rt.buf("experts.order", n * top, 1, torch.int32, cap=pairs_cap),
@@ -137,22 +151,22 @@ class RoutedExperts(FeedForward):
             scratch["xs"] = rt.buf("experts.xs", n * top, self.hidden, cap=pairs_cap)
         resid = getattr(ctx, "residual", None)
         if resid is not None and resid.shape[0] >= n and resid.shape[1] == self.hidden:
-            ops.moe_experts(x, self.w_up, self.w_down, ids, wts, scratch, resid[:n], rt.err, self.activation, self.gated)
+            ops.moe_experts(x, self.w_up, self.w_down, ids, wts, scratch, resid[:n], rt.err, self.activation, self.gated, self.identity > 0)
             return self.shared.forward(ctx, x) if self.shared is not None else ops.ADDED
         if self.shared is not None:
             # the shared expert first: when its result comes as the float slices of a split product, the routed sum is
             # added into the first slice and the slices are handed on as they are (whoever reads them adds them in order)
             y = self.shared.forward(ctx, x)
             if isinstance(y, ops.Partials) and y.t.dtype == torch.float32 and y.t.shape[1] >= n and y.t.shape[2] == self.hidden:
-                ops.moe_experts(x, self.w_up, self.w_down, ids, wts, scratch, y.t[0, :n], rt.err, self.activation, self.gated)
+                ops.moe_experts(x, self.w_up, self.w_down, ids, wts, scratch, y.t[0, :n], rt.err, self.activation, self.gated, self.identity > 0)
                 return y
             out = rt.buf("experts.out", n, self.hidden, torch.float32)
             out.zero_()
-            ops.moe_experts(x, self.w_up, self.w_down, ids, wts, scratch, out, rt.err, self.activation, self.gated)
+            ops.moe_experts(x, self.w_up, self.w_down, ids, wts, scratch, out, rt.err, self.activation, self.gated, self.identity > 0)
             if y is not None and y is not ops.ADDED:
                 ops.add_residual(out, y[:n])
             return ops.Partials(out.view(1, n, self.hidden))
         out = rt.buf("experts.out", n, self.hidden, torch.float32)
         out.zero_()
-        ops.moe_experts(x, self.w_up, self.w_down, ids, wts, scratch, out, rt.err, self.activation, self.gated)
+        ops.moe_experts(x, self.w_up, self.w_down, ids, wts, scratch, out, rt.err, self.activation, self.gated, self.identity > 0)
         return ops.Partials(out.view(1, n, self.hidden))

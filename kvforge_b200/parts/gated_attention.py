@@ -1,9 +1,9 @@
-"""Grouped-query attention whose query rows (and key rows) are normed as one vector and whose result is gated.
+"""Grouped-query attention whose query rows (and key rows) are normed as one vector and whose result may be gated.
 
 Per layer ``q = W_q x + b_q``, ``k = W_k x + b_k``, ``v = W_v x + b_v`` (the biases are optional); q and k are RMS-normed over
-all their numbers at once, before they are split into heads, with weights as wide as the projections; nothing turns with
-the position.  Attention sees every earlier key, a sliding window of them, or the keys of the query's own chunk.  The
-result is multiplied by ``sigmoid(W_g x)``, one number a head or one a channel, before the output projection.  A layer may
+all their numbers at once, before they are split into heads, with weights as wide as the projections; then the first
+dims of every head may turn with the position.  Attention sees every earlier key, a sliding window of them, or the keys of the query's own chunk.  The
+result may be multiplied by ``sigmoid(W_g x)``, one number a head or one a channel, before the output projection.  A layer may
 use the keys and values of an earlier layer (as that layer's cache holds them) with queries of its own.
 
 The input projections (q, k, v and the gate) are one product.  Heads whose size is no multiple of 8 are padded with zeros
@@ -16,22 +16,13 @@ from __future__ import annotations
 import torch
 
 from .. import ops
-from .attention import PagedAttention
+from .attention import PagedAttention, pad_head_rows
 from .base import CacheNeed, WeightDecl, register_mixer
 from .projection import PART_ROWS, project
 
 
 def _pad8(n: int) -> int:
     return (n + 7) // 8 * 8
-
-
-def pad_head_rows(t: torch.Tensor, heads: int, size: int, padded: int) -> torch.Tensor:
-    """Rows (or entries) of ``heads`` heads of ``size``, each followed by zeros up to ``padded``."""
-    if size == padded:
-        return t
-    out = torch.zeros((heads, padded, *t.shape[1:]), dtype=t.dtype, device=t.device)
-    out[:, :size] = t.reshape(heads, size, *t.shape[1:])
-    return out.reshape(heads * padded, *t.shape[1:])
 
 
 def stack_rows(mats: list[torch.Tensor]) -> tuple[torch.Tensor, list[int]]:
@@ -51,7 +42,7 @@ def stack_rows(mats: list[torch.Tensor]) -> tuple[torch.Tensor, list[int]]:
 @register_mixer("gated_attention")
 class GatedAttention(PagedAttention):
     """params: ``hidden_size``, ``num_heads``, ``num_kv_heads``, ``head_dim``; optional ``v_head_dim``, ``scale``, ``window`` or
-    ``chunk`` (as ``paged_attention``), ``qkv_bias`` (tensors ``q.b``, ``k.b``, ``v.b``), ``joint_norm`` (``{"eps": e}``: tensors
+    ``chunk``, ``position`` (a rotation with any magnitude) and ``keep_window`` (as ``paged_attention``), ``qkv_bias`` (tensors ``q.b``, ``k.b``, ``v.b``), ``joint_norm`` (``{"eps": e}``: tensors
     ``q.norm``, ``k.norm``; ``None``: no norm), ``gate`` (``"head"``, ``"channel"`` or ``None``; tensor ``g``), ``shared_kv`` (keys and
     values are an earlier layer's: no tensors of its own for them) and ``keep_all`` (the cache keeps every key although
     this layer's queries do not see them all: a later layer that reads this cache does).  Other tensors: ``q``, ``k``, ``v``, ``o``.
@@ -61,12 +52,9 @@ class GatedAttention(PagedAttention):
 
     def __init__(self, params, prefix=""):
         p = dict(params)
-        self.d_true = int(p["head_dim"])
-        self.dv_true = int(p.get("v_head_dim") or self.d_true)
-        p["head_dim"], p["v_head_dim"] = _pad8(self.d_true), _pad8(self.dv_true)
-        p["scale"] = float(p.get("scale") or self.d_true**-0.5)
+        p["pad_heads"] = True
         super().__init__(p, prefix)
-        self.params = dict(params)  # the tensors have the sizes that were asked for
+        self.params = dict(params)
         self.qkv_bias = bool(p.get("qkv_bias", False))
         jn = p.get("joint_norm")
         self.norm_eps = float(jn["eps"]) if jn else None
@@ -76,8 +64,8 @@ class GatedAttention(PagedAttention):
         self.shared_kv = bool(p.get("shared_kv", False))
         self.keep_all = bool(p.get("keep_all", False))
         self.own_kv = 0 if self.shared_kv else self.nkv
-        if self.position_spec is not None or self.taps or self.qk_eps is not None or self.bias_shape or self.softcap or self.has_sink or self.value_mix:
-            raise ValueError("gated_attention has no rotation, convolution, per-head norm, bias on scores, cap, sink or mixed values")
+        if self.taps or self.qk_eps is not None or self.bias_shape or self.softcap or self.has_sink or self.value_mix:
+            raise ValueError("gated_attention has no convolution, per-head norm, bias on scores, cap, sink or mixed values")
         self.qkv_dim = self.q_dim + self.own_kv * (self.d + self.dv)
 
     @classmethod
@@ -127,10 +115,11 @@ class GatedAttention(PagedAttention):
         if self.norm_eps is not None:
             self.q_w = heads("q.norm", nh, self.d_true, d).contiguous()
             self.k_w = heads("k.norm", kv, self.d_true, d).contiguous() if kv else None
+        self._bind_position()
         self._bind_attention()
 
     # ------------------------------------------------------------------ between the two products
-    inner_width = property(lambda self: self.o_dim)
+    open_form = True
 
     def take_input(self) -> torch.Tensor:
         w, self.w_in = self.w_in, None
@@ -152,7 +141,8 @@ class GatedAttention(PagedAttention):
         ops.joint_norm_cache(
             y, parts, self.bias_vec, self.q_w, self.k_w, self.nh * self.d_true, max(1, self.own_kv * self.d_true), self.norm_eps or 0.0,
             ctx.slot_mappings[cache.group] if own else None, cache.k if own else None, cache.v if own else None,
-            self.nh, self.own_kv, self.d, self.dv, ctx.block_size, rt.err,
+            self.nh, self.own_kv, self.d, self.dv, ctx.block_size, rt.err, positions=ctx.positions, inv_freq=self.inv_freq,
+            interleaved=self.interleaved, magnitude=self.magnitude,
         )  # fmt: skip
         plain = self.out_gate is None and mult == 1.0 and out.is_contiguous()
         heads_out = out if plain else rt.buf("attn.out", n, self.o_dim)

@@ -117,6 +117,8 @@ class LatentAttention(Mixer):
         if self.position_spec is not None and self.position is None:
             self.position = build_part("position", self.position_spec)
             self.position.bind({}, rt)
+        if self.position is not None and self.position.magnitude != 1.0:
+            raise ValueError("latent_attention turns pairs without changing their size")
         table = self.position.table() if self.position is not None else None
         self.interleaved = bool(getattr(self.position, "pairs_interleaved", False))
         self.inv_freq = table

@@ -72,9 +72,9 @@ class StreamRMSNorm(Norm):
 
 @register_norm("layernorm")
 class LayerNorm(Norm):
-    """Layer norm with a weight and no bias, ``(x - mean) / sqrt(var + eps) * w`` with the variance of the
+    """Layer norm with a weight, ``(x - mean) / sqrt(var + eps) * w`` with the variance of the
     deviations, in 32-bit.  params: ``dim``, ``eps``; optional ``centred`` (default true; false: the RMS norm
-    through the same kernel).  What the sublayer before left pending may be an ``ops.GatedWrite``: a result that
+    through the same kernel) and ``bias`` (true: the tensor ``bias [dim]`` is added to the normed rows).  What the sublayer before left pending may be an ``ops.GatedWrite``: a result that
     is gated, normed in the same way with a weight of its own and only then added to the stream."""
 
     def __init__(self, params, prefix=""):
@@ -82,19 +82,24 @@ class LayerNorm(Norm):
         self.dim = int(params["dim"])
         self.eps = float(params["eps"])
         self.centred = bool(params.get("centred", True))
+        self.has_bias = bool(params.get("bias", False))
 
     @classmethod
     def weight_decls(cls, params):
-        return {"weight": WeightDecl((int(params["dim"]),), kind="vector", init="ones")}
+        out = {"weight": WeightDecl((int(params["dim"]),), kind="vector", init="ones")}
+        if params.get("bias"):
+            out["bias"] = WeightDecl((int(params["dim"]),), kind="vector", init="zeros")
+        return out
 
     def bind(self, weights, rt):
         super().bind(weights, rt)
         self.weight = weights["weight"]
+        self.bias = weights["bias"].contiguous() if self.has_bias else None
 
     def forward(self, ctx, resid: torch.Tensor, delta, rows: torch.Tensor | None = None, num_rows: int | None = None):
         n = num_rows if rows is not None else resid.shape[0]
         out = self.rt.buf("norm.out" if rows is None else "norm.rows", n, self.dim)
-        ops.norm_step(resid, delta, self.weight, out, self.eps, self.centred, rows)
+        ops.norm_step(resid, delta, self.weight, out, self.eps, self.centred, rows, next_b=self.bias)
         return out
 
     def settle(self, ctx, resid: torch.Tensor, delta, out: torch.Tensor | None = None) -> None:
@@ -103,7 +108,7 @@ class LayerNorm(Norm):
 
     def replace(self, ctx, resid: torch.Tensor, out: torch.Tensor | None = None) -> None:
         """The stream itself becomes its normed rows (float); ``out`` gets them in the storage type."""
-        ops.norm_step(resid, None, self.weight, out, self.eps, self.centred, store_normed=True)
+        ops.norm_step(resid, None, self.weight, out, self.eps, self.centred, store_normed=True, next_b=self.bias)
 
 
 @register_norm("tanh_norm")

@@ -14,11 +14,26 @@ import torch
 
 from .. import ops
 from .base import CacheNeed, Mixer, PartSpec, WeightDecl, build_part, register_mixer
+from .gated_attention import stack_rows
 from .projection import project
 
 
 def _spec(v) -> PartSpec:
     return v if isinstance(v, PartSpec) else PartSpec(v["kind"], v.get("params", {}))
+
+
+def stack_inputs(branches: list) -> tuple[torch.Tensor, list[tuple[int, int]]]:
+    """The input matrices of branches in the open form, one below the other, each from a multiple of 8 rows on, and where each lies."""
+    mats = [b.take_input() for b in branches]
+    stacked, offs = stack_rows(mats)
+    return stacked, [(at, at + m.shape[0]) for at, m in zip(offs, mats)]
+
+
+def input_product(x: torch.Tensor, w: torch.Tensor, y: torch.Tensor) -> None:
+    if ops.skinny_ok(x, w):
+        ops.gemm_skinny(x, w, y)
+    else:
+        ops.linear(x, w, y)
 
 
 class _SideBySide(Mixer):
@@ -68,7 +83,11 @@ class _SideBySide(Mixer):
 @register_mixer("parallel_mixers")
 class ParallelMixers(_SideBySide):
     """params: ``hidden_size``, ``eps``, ``branches``: a list of ``(name, PartSpec)``; branch
-    ``name`` has its tensors under ``<prefix><name>.`` and its norm weight is ``<prefix><name>.out``."""
+    ``name`` has its tensors under ``<prefix><name>.`` and its norm weight is ``<prefix><name>.out``.
+
+    When every branch has the open form (``open_form``: ``take_input``, ``mix``, ``take_output``, and ``read_input`` where a branch makes more
+    of the input than that product), their input matrices are one product.  Where a block lets its parts add into the
+    residual stream, the mean joins it in the kernel that makes it."""
 
     def __init__(self, params, prefix=""):
         super().__init__(params, prefix)
@@ -82,22 +101,48 @@ class ParallelMixers(_SideBySide):
     def bind(self, weights, rt):
         super().bind(weights, rt)
         self.out_w = [weights[f"{name}.out"] for name in self.names]
+        self.open = len(self.branches) > 1 and all(getattr(b, "open_form", False) for b in self.branches)
+        if self.open:
+            self.w_in, self.in_cols = stack_inputs(self.branches)
+            self.w_out = [b.take_output() for b in self.branches]
+
+    def _open_results(self, ctx, x, cache):
+        rt, n = self.rt, x.shape[0]
+        for b in self.branches:
+            if hasattr(b, "read_input"):
+                b.read_input(ctx, x)
+        y = rt.buf("parallel.in", n, self.w_in.shape[0])
+        input_product(x, self.w_in, y)
+        results = []
+        for i, (branch, cols, (lo, hi)) in enumerate(zip(self.branches, self._state_cols, self.in_cols)):
+            inner = rt.buf(f"parallel.inner{i}", n, branch.inner_width)
+            branch.mix(ctx, y[:, lo:hi], self.branch_view(cache, cols), inner)
+            results.append(project(rt, f"parallel.proj{i}", inner, self.w_out[i], ctx))
+        return results
+
+    def _branch_results(self, ctx, x, cache):
+        results = []
+        for branch, cols in zip(self.branches, self._state_cols):
+            y = branch.forward(ctx, x, self.branch_view(cache, cols))
+            t = y.t if isinstance(y, ops.Partials) else y
+            if any(t.data_ptr() == (o.t if isinstance(o, ops.Partials) else o).data_ptr() for o in results):
+                # two branches of one kind hand back the same persistent buffer: keep this one's result apart
+                kept = self.rt.buf(f"parallel.keep{len(results)}", t.numel() // t.shape[-1], t.shape[-1], t.dtype).view(t.shape)
+                kept.copy_(t)
+                y = ops.Partials(kept) if isinstance(y, ops.Partials) else kept
+            results.append(y)
+        return results
 
     def forward(self, ctx, x, cache):
-        keep, ctx.residual = ctx.residual, None  # a branch's result is normed before it is added anywhere
+        # a branch's result is normed before it is added anywhere
+        (keep, ctx.residual), (row, ctx.slices) = (ctx.residual, None), (getattr(ctx, "slices", None), None)
         try:
-            results = []
-            for branch, cols in zip(self.branches, self._state_cols):
-                y = branch.forward(ctx, x, self.branch_view(cache, cols))
-                t = y.t if isinstance(y, ops.Partials) else y
-                if any(t.data_ptr() == (o.t if isinstance(o, ops.Partials) else o).data_ptr() for o in results):
-                    # two branches of one kind hand back the same persistent buffer: keep this one's result apart
-                    kept = self.rt.buf(f"parallel.keep{len(results)}", t.numel() // t.shape[-1], t.shape[-1], t.dtype).view(t.shape)
-                    kept.copy_(t)
-                    y = ops.Partials(kept) if isinstance(y, ops.Partials) else kept
-                results.append(y)
+            results = self._open_results(ctx, x, cache) if self.open else self._branch_results(ctx, x, cache)
         finally:
-            ctx.residual = keep
+            ctx.residual, ctx.slices = keep, row
+        if keep is not None and keep.shape[0] >= x.shape[0] and keep.shape[1] == self.hidden:
+            ops.branch_norm_mean(results, self.out_w, self.eps, keep[: x.shape[0]], add=True)
+            return ops.ADDED
         out = self.rt.buf("parallel.out", x.shape[0], self.hidden)
         ops.branch_norm_mean(results, self.out_w, self.eps, out)
         return out
@@ -121,13 +166,8 @@ class SummedMixers(_SideBySide):
 
     def bind(self, weights, rt):
         super().bind(weights, rt)  # the branches are bound already: they hand over their matrices
-        mats = [b.take_input() for b in self.branches]
-        self.in_cols, self.out_cols, at = [], [], 0
-        for m in mats:
-            self.in_cols.append((at, at + m.shape[0]))  # a branch's matrix is a multiple of 8 rows long
-            at += m.shape[0]
-        self.w_in = torch.cat(mats, dim=0).contiguous()
-        outs, at = [], 0
+        self.w_in, self.in_cols = stack_inputs(self.branches)
+        self.out_cols, outs, at = [], [], 0
         for b in self.branches:
             w = b.take_output()
             pad = -w.shape[1] % 8  # every branch begins at a multiple of 8 columns
@@ -140,10 +180,7 @@ class SummedMixers(_SideBySide):
     def forward(self, ctx, x, cache):
         rt, n = self.rt, x.shape[0]
         y = rt.buf("summed.in", n, self.w_in.shape[0])
-        if ops.skinny_ok(x, self.w_in):
-            ops.gemm_skinny(x, self.w_in, y)
-        else:
-            ops.linear(x, self.w_in, y)
+        input_product(x, self.w_in, y)
         inner = rt.buf("summed.inner", n, self.w_o.shape[1])
         if self.padded:
             inner.zero_()  # columns between the branches meet zero weights, and must be numbers

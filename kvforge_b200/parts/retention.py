@@ -95,11 +95,14 @@ class Retention(Mixer):
         if self.position_spec is not None and self.position is None:
             self.position = build_part("position", self.position_spec)
             self.position.bind({}, rt)
+        if self.position is not None and self.position.magnitude != 1.0:
+            raise ValueError("retention turns pairs without changing their size")
         self.inv_freq = self.position.table() if self.position is not None else None
         self.interleaved = bool(getattr(self.position, "pairs_interleaved", False))
 
     # ------------------------------------------------------------------ between the two products
     inner_width = property(lambda self: self.nh * self.dv)
+    open_form = property(lambda self: self.norm == "joint")
 
     def take_input(self) -> torch.Tensor:
         w, self.w_in = self.w_in, None

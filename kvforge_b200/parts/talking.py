@@ -115,6 +115,8 @@ class TalkingAttention(Mixer):
         if self.position_spec is not None and self.position is None:
             self.position = build_part("position", self.position_spec)
             self.position.bind({}, rt)
+        if self.position is not None and self.position.magnitude != 1.0:
+            raise ValueError("talking_attention turns pairs without changing their size")
         table = self.position.table() if self.position is not None else None
         if table is not None and getattr(self.position, "pairs_interleaved", False):
             raise ValueError("attention whose heads talk turns split pairs")
