@@ -206,7 +206,6 @@ class LatuzenConfig:
     eps: float
     layers: list[LayerConfig]
     architectures: list[str] = field(default_factory=lambda: [ARCHITECTURE])
-    max_position_embeddings: int = 0  # the design has no longest context
     raw: dict[str, Any] = field(default_factory=dict, repr=False)
 
     @property
@@ -216,6 +215,10 @@ class LatuzenConfig:
     @property
     def num_layers(self) -> int:
         return len(self.layers)
+
+    @property
+    def max_position_embeddings(self) -> int:
+        return 1 << 30  # the design names no longest sequence
 
     def __post_init__(self) -> None:
         for i, lc in enumerate(self.layers):

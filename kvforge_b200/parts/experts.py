@@ -141,14 +141,15 @@ class RoutedExperts(FeedForward):
             bias=self.bias, chosen_softmax=self.score == "chosen_softmax", group_rank=self.group_rank, scale=self.weight_scale,
         )  # fmt: skip
         scratch = {
-            "order": rt.buf("experts.order", n * top, 1, torch.int32, cap=pairs_cap),
-            "tiles": rt.buf("experts.tiles", ops.moe_max_tiles(n * top, e), 3, torch.int32, cap=ops.moe_max_tiles(pairs_cap, e)),
+            # rows are pairs: layers whose tokens use other numbers of experts have buffers of their own
+            "order": rt.buf(f"experts.order.{top}", n * top, 1, torch.int32, cap=pairs_cap),
+            "tiles": rt.buf(f"experts.tiles.{top}.{e}", ops.moe_max_tiles(n * top, e), 3, torch.int32, cap=ops.moe_max_tiles(pairs_cap, e)),
             "meta": self._meta,
-            "act": rt.buf("experts.act", n * top, self.ff_pad, cap=pairs_cap),
-            "y": rt.buf("experts.y", n * top, self.hidden, torch.float32, cap=pairs_cap),
+            "act": rt.buf(f"experts.act.{top}", n * top, self.ff_pad, cap=pairs_cap),
+            "y": rt.buf(f"experts.y.{top}", n * top, self.hidden, torch.float32, cap=pairs_cap),
         }
         if x.dtype == torch.bfloat16 and n * top >= ops.GROUPED_TCGEN05_MIN_ROWS * e:
-            scratch["xs"] = rt.buf("experts.xs", n * top, self.hidden, cap=pairs_cap)
+            scratch["xs"] = rt.buf(f"experts.xs.{top}", n * top, self.hidden, cap=pairs_cap)
         resid = getattr(ctx, "residual", None)
         if resid is not None and resid.shape[0] >= n and resid.shape[1] == self.hidden:
             ops.moe_experts(x, self.w_up, self.w_down, ids, wts, scratch, resid[:n], rt.err, self.activation, self.gated, self.identity > 0)
