@@ -42,6 +42,7 @@ constexpr int NWARPS = 4;
 constexpr int UNIT = 16;  // keys per copy and per MMA row tile
 constexpr uint32_t SPIN_LIMIT = 1u << 20;
 constexpr float RESCALE_STEP = 8.f;
+constexpr float LOG2E = 1.4426950408889634f;
 
 struct DecParams {
   const bf16* q;
@@ -61,6 +62,7 @@ struct DecParams {
   int wave_target;  // > 0: the range size doubles until the ranges of the longest context are at most this many CTAs
   int total_rows;  // rows of the cache seen as [rows][D]: a copy from this row reads zeros
   float scale_log2;
+  const float* sinks;  // [nh] (natural-log units) or null: a number a head whose exponential joins the denominator, without a key or a value
 };
 
 __device__ __forceinline__ uint32_t sm32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
@@ -401,6 +403,11 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
         continue;
       }
       if (ns == 1) {  // the only range of its sequence: this is the result
+        if (p.sinks) {
+          const float sk = p.sinks[kvh * g + r] * LOG2E, mm = fmaxf(M, sk), f = M == -INFINITY ? 0.f : ex2(M - mm);
+          acc *= f;
+          L = L * f + ex2(sk - mm);
+        }
         p.out[(size_t)(q_begin + q_len - 1) * p.out_stride + (size_t)(kvh * g + r) * D + dcol] =
             __float2bfloat16_rn(L > 0.f ? acc / L : 0.f);
         continue;
@@ -430,6 +437,11 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
       float M = -INFINITY;
       for (int s2 = 0; s2 < ns; ++s2) M = fmaxf(M, ld_cluster(in_cta(mine + D * 4, (uint32_t)s2)));
       float acc = 0.f, L = 0.f;
+      if (p.sinks) {
+        const float sk = p.sinks[kvh * g + r] * LOG2E;
+        M = fmaxf(M, sk);
+        L = ex2(sk - M);
+      }
       for (int s2 = 0; s2 < ns; ++s2) {
         const uint32_t theirs = in_cta(mine, (uint32_t)s2);
         const float ms = ld_cluster(theirs + D * 4);
@@ -451,7 +463,8 @@ attn_decode_tma_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_c
   bf16* orow = p.out + (size_t)(q_begin + q_len - 1) * p.out_stride;
   for (int h = warp; h < g; h += NWARPS) {
     const int head = kvh * g + h;
-    merge_ranges_warp<D>(p.part_acc, p.part_ml, ((size_t)b * p.nh + head) * p.max_splits, ns, wgt, orow + (size_t)head * D, lane);
+    merge_ranges_warp<D>(p.part_acc, p.part_ml, ((size_t)b * p.nh + head) * p.max_splits, ns, wgt, orow + (size_t)head * D, lane,
+                         p.sinks ? p.sinks[head] : -INFINITY);
   }
 }
 
@@ -531,7 +544,7 @@ int run_dec(const void* q, void* out, const void* kcache, const void* vcache,
             const int* block_tables, const int* qsl, const int* ctx_lens, int B, int q_stride, int out_stride,
             int bt_stride, int nh, int nkv, int d, int block_size, long long num_blocks, float scale, int window,
             int split_size, int max_splits, int grid_splits, float* part_acc, float* part_ml, int* tickets, int* err,
-            int flags, int wave_target, cudaStream_t st) {
+            int flags, int wave_target, const float* sinks, cudaStream_t st) {
   if (B <= 0) return 0;
   const int cluster = flags & 1;
   if ((d != 64 && d != 128) || nkv <= 0 || nh <= 0 || nh % nkv != 0 || nh / nkv > 8) return (int)cudaErrorInvalidValue;
@@ -557,7 +570,8 @@ int run_dec(const void* q, void* out, const void* kcache, const void* vcache,
   p.split_size = split_size; p.max_splits = max_splits; p.wave_target = wave_target > 0 ? wave_target : 0;
   p.grid_splits = grid_splits > 0 && grid_splits < max_splits ? grid_splits : max_splits;
   p.total_rows = (int)rows;
-  p.scale_log2 = scale * 1.4426950408889634f;
+  p.scale_log2 = scale * LOG2E;
+  p.sinks = sinks;
   // more CTAs than fit at four stages: two stages, so that they run in fewer waves
   const long long ctas = (long long)p.grid_splits * B * nkv;
   static int sms = 0;
@@ -590,8 +604,8 @@ KVF_API int kvf_paged_attention_decode_tma_bf16(const void* q, void* out, const 
                                                 int block_size, long long num_blocks, float scale, int window,
                                                 int split_size, int max_splits, int grid_splits, float* part_acc,
                                                 float* part_ml, int* tickets, int* err, int flags, int wave_target,
-                                                cudaStream_t st) {
+                                                const float* sinks, cudaStream_t st) {
   return run_dec(q, out, kcache, vcache, block_tables, qsl, ctx_lens, B, q_stride, out_stride, bt_stride, nh,
                  nkv, d, block_size, num_blocks, scale, window, split_size, max_splits, grid_splits, part_acc, part_ml,
-                 tickets, err, flags, wave_target, st);
+                 tickets, err, flags, wave_target, sinks, st);
 }

@@ -83,6 +83,13 @@ struct TcAttnParams {
   int box_rows;    // 16, 32 or 64: the largest of them that divides the page
   int total_rows;  // rows of the cache seen as [rows][64]: a box from this row reads zeros
 };
+// The form with sinks has its own parameters: the plain form stands at its register budget, and a longer parameter block alone
+// makes it spill.
+struct TcAttnSinkParams : TcAttnParams {
+  const float* sinks;  // [nh] (natural-log units): a number a head whose exponential joins the denominator, without a key or a value
+};
+template <bool SINKS> struct ParamsOf { using type = TcAttnParams; };
+template <> struct ParamsOf<true> { using type = TcAttnSinkParams; };
 
 __device__ __forceinline__ uint32_t sm32(const void* p) { return (uint32_t)__cvta_generic_to_shared(p); }
 __device__ __forceinline__ void bar_init(uint32_t bar, uint32_t count) {
@@ -292,9 +299,9 @@ __device__ __forceinline__ float softmax_tile(uint32_t (&va)[32], uint32_t (&vb)
   return s0 + s1;
 }
 
-template <int D>
+template <int D, bool SINKS>
 __global__ void __launch_bounds__(THREADS, Shape<D>::CTAS_PER_SM)
-attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const TcAttnParams p) {
+attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, const typename ParamsOf<SINKS>::type p) {
   constexpr int HALVES = Shape<D>::HALVES, KV_STAGES = Shape<D>::KV_STAGES;
   constexpr uint32_t Q_BYTES = Shape<D>::Q_BYTES, KV_BYTES = Shape<D>::KV_BYTES;
   extern __shared__ __align__(1024) unsigned char smem_raw[];
@@ -565,6 +572,12 @@ attn_tcgen05_kernel(const __grid_constant__ CUtensorMap map_k, const __grid_cons
     const uint32_t my_s = tmem_s + lane_addr + (uint32_t)(grp * BN), my_o = tmem_o + lane_addr + (uint32_t)(grp * D);
     const uint32_t s_bar = s_full0 + 8 * grp, p_bar = p_full0 + 8 * grp, pv_bar = pv_done0 + 8 * grp;
     float m_ref = -INFINITY, l = 0.f;
+    if constexpr (SINKS) {
+      if (grp == 0 && valid) {  // the sink is where the first group starts: one in the sum at its own maximum
+        m_ref = p.sinks[kvh * g + hh] * 1.4426950408889634f;
+        l = 1.f;
+      }
+    }
     bool ok = true;
     int i = 0;  // index among this group's tiles
     for (int t = grp; t < n_tiles && ok; t += 2, ++i) {
@@ -687,11 +700,11 @@ int cache_map(CUtensorMap* map, const void* ptr, long long rows, int d, int box_
   return r == CUDA_SUCCESS ? 0 : (int)cudaErrorInvalidValue;
 }
 
-template <int D>
-int launch_tc_attn(const CUtensorMap& mk, const CUtensorMap& mv, const TcAttnParams& p, dim3 grid, cudaStream_t st) {
-  cudaError_t e = cudaFuncSetAttribute(attn_tcgen05_kernel<D>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Shape<D>::SMEM_BYTES);
+template <int D, bool SINKS>
+int launch_tc_attn(const CUtensorMap& mk, const CUtensorMap& mv, const typename ParamsOf<SINKS>::type& p, dim3 grid, cudaStream_t st) {
+  cudaError_t e = cudaFuncSetAttribute(attn_tcgen05_kernel<D, SINKS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)Shape<D>::SMEM_BYTES);
   if (e != cudaSuccess) return (int)e;
-  return launch(attn_tcgen05_kernel<D>, grid, dim3(THREADS), Shape<D>::SMEM_BYTES, st, mk, mv, p);
+  return launch(attn_tcgen05_kernel<D, SINKS>, grid, dim3(THREADS), Shape<D>::SMEM_BYTES, st, mk, mv, p);
 }
 
 }  // namespace
@@ -702,15 +715,17 @@ KVF_API int kvf_paged_attention_tcgen05_bf16(const void* q, void* out, const voi
                                              const int* block_tables, const int* qsl, const int* ctx_lens, int B,
                                              int max_q_len, int q_stride, int out_stride, int bt_stride, int nh,
                                              int nkv, int d, int block_size, long long num_blocks, float scale,
-                                             int window, const int* work, int n_work, int* err, cudaStream_t st) {
+                                             int window, const int* work, int n_work, int* err, const float* sinks,
+                                             cudaStream_t st) {
   if (B <= 0 || max_q_len <= 0) return 0;
   if ((d != 64 && d != 128) || nkv <= 0 || nh % nkv != 0 || nh / nkv > BM || block_size <= 0 || num_blocks <= 0) return (int)cudaErrorInvalidValue;
   if ((q_stride & 7) || (out_stride & 7) || ((((uintptr_t)q) | ((uintptr_t)out)) & 15)) return (int)cudaErrorInvalidValue;
   if ((unsigned)B > 65535u || (max_q_len + (BM / (nh / nkv)) - 1) / (BM / (nh / nkv)) > 65535) return (int)cudaErrorInvalidValue;
-  TcAttnParams p;
+  TcAttnSinkParams p;
   p.q = (const bf16*)q; p.out = (bf16*)out; p.kcache = (const bf16*)kcache; p.vcache = (const bf16*)vcache;
   p.block_tables = block_tables; p.qsl = qsl; p.ctx_lens = ctx_lens; p.err = err;
   p.work = work;
+  p.sinks = sinks;
   p.num_seqs = B;
   p.q_stride = q_stride; p.out_stride = out_stride; p.bt_stride = bt_stride;
   p.nh = nh; p.nkv = nkv; p.block_size = block_size; p.window = window;
@@ -732,5 +747,7 @@ KVF_API int kvf_paged_attention_tcgen05_bf16(const void* q, void* out, const voi
   const int g = nh / nkv, tq = BM / g;
   if (work && (n_work <= 0 || n_work > 65535)) return (int)cudaErrorInvalidValue;
   const dim3 grid(nkv, work ? n_work : B, work ? 1 : (max_q_len + tq - 1) / tq);
-  return d == 64 ? launch_tc_attn<64>(mk, mv, p, grid, st) : launch_tc_attn<128>(mk, mv, p, grid, st);
+  if (sinks) return d == 64 ? launch_tc_attn<64, true>(mk, mv, p, grid, st) : launch_tc_attn<128, true>(mk, mv, p, grid, st);
+  const TcAttnParams& plain = p;
+  return d == 64 ? launch_tc_attn<64, false>(mk, mv, plain, grid, st) : launch_tc_attn<128, false>(mk, mv, plain, grid, st);
 }

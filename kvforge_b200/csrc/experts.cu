@@ -49,12 +49,12 @@ template <> __device__ __forceinline__ void load8<bf16>(const bf16* src, float* 
   bf16x8_to_float(*reinterpret_cast<const uint4*>(src), dst);
 }
 
-// One CTA of eight warps per RT tokens (one token a CTA while a step has few, four when it has many).  The warps share out the experts: a logit is one warp's dot product (a lane
+// One CTA per RT tokens (one token and up to 32 warps a CTA while a step has few, four tokens and eight warps when it has many).  The warps share out the experts: a logit is one warp's dot product (a lane
 // adds its products in the order of the columns, then the lanes are summed in a fixed tree), so it does not depend on
 // the batch; a row of the router is read once for the CTA's tokens.  Then warp t chooses for token t.  Shared memory
 // per token: scores [E], choice scores [E], group scores [G], group flags [G].
 template <typename T, int RT>
-__global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ x, long long x_stride,
+__global__ void __launch_bounds__(RT == 1 ? 1024 : 256) moe_route_kernel(const T* __restrict__ x, long long x_stride,
                                                          const float* __restrict__ router, const float* __restrict__ correction,
                                                          int n_tokens, int W, int E, int top, int groups, int keep,
                                                          float norm_eps, int vec, int flags, int* __restrict__ ids, float* __restrict__ wts,
@@ -62,10 +62,10 @@ __global__ void __launch_bounds__(256) moe_route_kernel(const T* __restrict__ x,
   pdl_launch();
   pdl_wait();
   extern __shared__ float sm[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
   const int n0 = blockIdx.x * RT;
   const int per_token = 2 * E + 2 * groups;
-  for (int e = warp; e < E; e += 8) {
+  for (int e = warp; e < E; e += warps) {
     const float* wr = router + (size_t)e * W;
     float z[RT];
 #pragma unroll
@@ -625,7 +625,7 @@ int run_products<bf16>(const bf16* x, long long x_stride, const bf16* w_up, cons
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;                                                          \
     const int vec = (W % 8 == 0) && (x_stride % 8 == 0) && ((((uintptr_t)x) | ((uintptr_t)router)) % 16 == 0);        \
     if (rt == 1)                                                                                                      \
-      return launch(moe_route_kernel<T, 1>, dim3(n_tokens), dim3(256), smem, st, (const T*)x, x_stride, router,       \
+      return launch(moe_route_kernel<T, 1>, dim3(n_tokens), dim3(E > 16 ? 1024 : E > 8 ? 512 : 256), smem, st, (const T*)x, x_stride, router,       \
                     correction, n_tokens, W, E, top, groups, keep, norm_eps, vec, flags, ids, wts, logit_bias,        \
                     scale);                                                                                           \
     return launch(moe_route_kernel<T, 4>, dim3((n_tokens + 3) / 4), dim3(256), smem, st, (const T*)x, x_stride,       \

@@ -9,8 +9,8 @@ using namespace kvf;
 namespace {
 
 // ---------------------------------------------------------------- per-head norm, rotation, cache write
-// Rows of `qkv` hold nh query heads and nkv key heads of dk and nkv value heads of dv.  A warp owns
-// one (token, head).  Query and key heads: x <- x / sqrt(sum(x^2) / count + eps) * w (w of dk floats shared
+// Rows of `qkv` hold nh query heads and nkv key heads of dk and nkv value heads of dv.  A warp takes
+// a head at a time.  Query and key heads: x <- x / sqrt(sum(x^2) / count + eps) * w (w of dk floats shared
 // by all heads; skipped without w; count: the numbers of a head that are not padding, padded places hold zeros), then the
 // first `rot` dims turn by the angle pos * inv_freq[i] and are multiplied by `magnitude`, in
 // interleaved pairs (2i, 2i+1) or, with split_pairs, in pairs (i, i + rot/2) (skipped when rot == 0).
@@ -20,92 +20,100 @@ namespace {
 // step left for the same token: with v_keep the values as projected are also copied to v_keep[n][nkv*dv];
 // with v_first the value becomes (1 - lambda) v + lambda v_first[n] (lambda = *v_lambda, in float, rounded
 // once) before it is cached.
+// A CTA takes HEAD_WARPS heads of a token at a time (all of the token's when there are many tokens), and works out the token's
+// cosines and sines once.  A lane keeps its pairs in registers between the sum and the rotation.
+constexpr int HEAD_WARPS = 8;
+constexpr int HEAD_PAIRS = 4;  // pairs a lane holds: heads of up to 256
+
 template <typename T>
-__global__ void __launch_bounds__(128) head_norm_cache_kernel(T* __restrict__ qkv, long long row_stride,
+__global__ void __launch_bounds__(HEAD_WARPS * 32) head_norm_cache_kernel(T* __restrict__ qkv, long long row_stride,
                                                                const int* __restrict__ positions,
                                                                const float* __restrict__ q_w, const float* __restrict__ k_w,
                                                                float eps, const float* __restrict__ inv_freq, int rot,
                                                                const int* __restrict__ slots, T* __restrict__ kcache,
-                                                               T* __restrict__ vcache, int n_tokens, int nh, int nkv, int dk,
+                                                               T* __restrict__ vcache, int nh, int nkv, int dk,
                                                                int dv, int block_size, long long num_slots,
                                                                int* __restrict__ err, int split_pairs,
                                                                T* __restrict__ v_keep, const T* __restrict__ v_first,
                                                                const float* __restrict__ v_lambda, float count, float magnitude) {
   pdl_launch();
+  extern __shared__ float turn[];  // [rot / 2] cosines, [rot / 2] sines
   pdl_wait();
-  const int heads = nh + 2 * nkv;
-  const long long unit = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
-  if (unit >= (long long)n_tokens * heads) return;
-  const int n = (int)(unit / heads), h = (int)(unit - (long long)n * heads);
-  const int lane = threadIdx.x & 31;
-  T* row = qkv + (size_t)n * row_stride;
-  const bool is_q = h < nh, is_k = !is_q && h < nh + nkv;
-  long long slot = -1;
-  if (!is_q) {
-    slot = slots ? slots[n] : -1;
-    if (slot < 0 && !is_k && v_keep) {  // a row without a slot still leaves its values for the layers after
-      const int g = h - nh - nkv;
-      const T* src = row + (size_t)(nh + nkv) * dk + (size_t)g * dv;
-      for (int j = lane; j < dv; j += 32) v_keep[(size_t)n * nkv * dv + (size_t)g * dv + j] = src[j];
-    }
-    if (slot < 0) return;
-    if (slot >= num_slots) {
-      if (lane == 0 && err) atomicOr(err, 2);
-      return;
-    }
-  }
-  if (!is_q && !is_k) {  // a value head: copied as it is
-    const int g = h - nh - nkv;
-    const T* src = row + (size_t)(nh + nkv) * dk + (size_t)g * dv;
-    T* dst = vcache + (((size_t)(slot / block_size) * nkv + g) * block_size + (size_t)(slot % block_size)) * dv;
-    if (v_first) {
-      const float lam = v_lambda[0];
-      const T* first = v_first + (size_t)n * nkv * dv + (size_t)g * dv;
-      for (int j = lane; j < dv; j += 32) dst[j] = from_float<T>(fmaf(lam, to_float<T>(first[j]), (1.f - lam) * to_float<T>(src[j])));
-    } else {
-      for (int j = lane; j < dv; j += 32) dst[j] = src[j];
-    }
-    if (v_keep)
-      for (int j = lane; j < dv; j += 32) v_keep[(size_t)n * nkv * dv + (size_t)g * dv + j] = src[j];
-    return;
-  }
-  T* x = row + (size_t)h * dk;  // key heads follow the query heads with the same size
-  const float* w = is_q ? q_w : k_w;
-  if (is_q && !w && rot == 0) return;
-  float ss = 0.f;
-  if (w) {
-    for (int j = lane; j < dk; j += 32) {
-      const float v = to_float<T>(x[j]);
-      ss = fmaf(v, v, ss);
-    }
-    ss = warp_sum(ss);
-  }
-  const float r = w ? 1.f / sqrtf(ss / count + eps) : 1.f;
-  const float pos = (float)positions[n];
-  T* dst = x;
-  if (is_k) {
-    const int g = h - nh;
-    dst = kcache + (((size_t)(slot / block_size) * nkv + g) * block_size + (size_t)(slot % block_size)) * dk;
-  }
-  for (int i = lane; i < dk / 2; i += 32) {
-    // pair i: dims (2i, 2i+1), or (i, i + rot/2) among the dims that turn in split pairs
-    const bool turns = 2 * i < rot;
-    const int ia = (turns && split_pairs) ? i : 2 * i, ib = (turns && split_pairs) ? i + rot / 2 : 2 * i + 1;
-    float a = to_float<T>(x[ia]), b = to_float<T>(x[ib]);
-    if (w) {
-      a = a * r * w[ia];
-      b = b * r * w[ib];
-    }
-    if (turns) {
+  const int n = blockIdx.x, heads = nh + 2 * nkv, half = rot >> 1;
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  if (rot) {
+    const float pos = (float)positions[n];
+    for (int i = threadIdx.x; i < half; i += blockDim.x) {
       float sn, cs;
       sincosf(pos * inv_freq[i], &sn, &cs);
-      float ya, yb;
-      rotate_pair(a, b, cs * magnitude, sn * magnitude, ya, yb);
-      a = ya;
-      b = yb;
+      turn[i] = cs * magnitude;
+      turn[half + i] = sn * magnitude;
     }
-    dst[ia] = from_float<T>(a);
-    dst[ib] = from_float<T>(b);
+    __syncthreads();
+  }
+  T* row = qkv + (size_t)n * row_stride;
+  long long slot = slots ? slots[n] : -1;
+  if (slot >= num_slots) {
+    if (slots && threadIdx.x == 0 && err) atomicOr(err, 2);
+    slot = -2;  // beyond the pool: nothing of this token is kept
+  }
+  const size_t page = slot >= 0 ? (size_t)(slot / block_size) : 0, place = slot >= 0 ? (size_t)(slot % block_size) : 0;
+  for (int h = blockIdx.y * HEAD_WARPS + warp; h < heads; h += gridDim.y * HEAD_WARPS) {
+    const bool is_q = h < nh, is_k = !is_q && h < nh + nkv;
+    if (!is_q && !is_k) {  // a value head: copied, or mixed with an earlier layer's
+      const int g = h - nh - nkv;
+      const T* src = row + (size_t)(nh + nkv) * dk + (size_t)g * dv;
+      if (v_keep && slot >= -1)  // a row without a slot still leaves its values for the layers after
+        for (int j = lane; j < dv; j += 32) v_keep[(size_t)n * nkv * dv + (size_t)g * dv + j] = src[j];
+      if (slot < 0) continue;
+      T* dst = vcache + ((page * nkv + g) * block_size + place) * dv;
+      if (v_first) {
+        const float lam = v_lambda[0];
+        const T* first = v_first + (size_t)n * nkv * dv + (size_t)g * dv;
+        for (int j = lane; j < dv; j += 32) dst[j] = from_float<T>(fmaf(lam, to_float<T>(first[j]), (1.f - lam) * to_float<T>(src[j])));
+      } else {
+        for (int j = lane; j < dv; j += 32) dst[j] = src[j];
+      }
+      continue;
+    }
+    if (is_k && slot < 0) continue;
+    T* x = row + (size_t)h * dk;  // key heads follow the query heads with the same size
+    const float* w = is_q ? q_w : k_w;
+    if (is_q && !w && rot == 0) continue;
+    T* dst = is_q ? x : kcache + ((page * nkv + (h - nh)) * block_size + place) * dk;
+    float a[HEAD_PAIRS], b[HEAD_PAIRS], ss = 0.f;
+#pragma unroll
+    for (int k = 0; k < HEAD_PAIRS; ++k) {
+      // pair i: dims (2i, 2i+1), or (i, i + rot/2) among the dims that turn in split pairs
+      const int i = lane + 32 * k;
+      a[k] = b[k] = 0.f;
+      if (2 * i >= dk) continue;
+      const bool split = split_pairs && 2 * i < rot;
+      a[k] = to_float<T>(x[split ? i : 2 * i]);
+      b[k] = to_float<T>(x[split ? i + half : 2 * i + 1]);
+      ss = fmaf(a[k], a[k], fmaf(b[k], b[k], ss));
+    }
+    const float r = w ? 1.f / sqrtf(warp_sum(ss) / count + eps) : 1.f;
+#pragma unroll
+    for (int k = 0; k < HEAD_PAIRS; ++k) {
+      const int i = lane + 32 * k;
+      if (2 * i >= dk) continue;
+      const bool turns = 2 * i < rot, split = split_pairs && turns;
+      const int ia = split ? i : 2 * i, ib = split ? i + half : 2 * i + 1;
+      float u = a[k], v = b[k];
+      if (w) {
+        u = u * r * w[ia];
+        v = v * r * w[ib];
+      }
+      if (turns) {
+        float yu, yv;
+        rotate_pair(u, v, turn[i], turn[half + i], yu, yv);
+        u = yu;
+        v = yv;
+      }
+      dst[ia] = from_float<T>(u);
+      dst[ib] = from_float<T>(v);
+    }
   }
 }
 
@@ -250,13 +258,14 @@ inline unsigned grid_for(long long total, int threads) {
                                         int split_pairs, void* v_keep, const void* v_first, const float* v_lambda,   \
                                         int count, float magnitude, cudaStream_t st) {                               \
     if (n_tokens <= 0) return 0;                                                                                     \
-    if (dk <= 0 || (dk & 1) || rot < 0 || rot > dk || (rot & 1)) return (int)cudaErrorInvalidValue;                  \
+    if (dk <= 0 || (dk & 1) || dk > 64 * HEAD_PAIRS || rot < 0 || rot > dk || (rot & 1))                             \
+      return (int)cudaErrorInvalidValue;                                                                             \
     if ((v_first && !v_lambda) || count <= 0 || count > dk) return (int)cudaErrorInvalidValue;                       \
-    const long long units = (long long)n_tokens * (nh + 2 * nkv);                                                    \
-    return launch(head_norm_cache_kernel<T>, dim3((unsigned)((units + 3) / 4)), dim3(128), 0, st, (T*)qkv,           \
-                  row_stride, positions, q_w, k_w, eps, inv_freq, rot, slots, (T*)kcache, (T*)vcache, n_tokens, nh,  \
-                  nkv, dk, dv, block_size, num_slots, err, split_pairs, (T*)v_keep, (const T*)v_first, v_lambda,     \
-                  (float)count, magnitude);                                                                          \
+    const int groups = (nh + 2 * nkv + HEAD_WARPS - 1) / HEAD_WARPS;                                                 \
+    return launch(head_norm_cache_kernel<T>, dim3(n_tokens, n_tokens <= 256 ? groups : 1), dim3(HEAD_WARPS * 32),    \
+                  (size_t)rot * sizeof(float), st, (T*)qkv, row_stride, positions, q_w, k_w, eps, inv_freq, rot,     \
+                  slots, (T*)kcache, (T*)vcache, nh, nkv, dk, dv, block_size, num_slots, err, split_pairs,           \
+                  (T*)v_keep, (const T*)v_first, v_lambda, (float)count, magnitude);                                 \
   }                                                                                                                  \
   KVF_API int kvf_row_rmsnorm_##SUF(const void* x, long long x_stride, const float* w, float eps, long long n_rows,  \
                                     int r, void* out, long long out_stride, cudaStream_t st) {                       \

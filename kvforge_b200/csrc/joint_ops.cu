@@ -181,6 +181,25 @@ __global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParam
           f[e] = a;
           f[(e + 1) % V] = b;
         }
+      } else if (V == 4 && !p.interleaved && (half & 3) == 0 && (p.dk & 3) == 0) {  // four pairs' numbers of one side
+        const bool first = j0 < half;
+        const int d = first ? half : -half, i = first ? j0 : j0 - half;
+        float other[V], c4[V], s4[V];
+        Pack<float, V>::load(row + c + d, other);
+        Pack<float, V>::load(cs + i, c4);
+        Pack<float, V>::load(sn + i, s4);
+        if (p.qw) {
+          float w2[V];
+          Pack<float, V>::load(w + c_of_w + d, w2);
+#pragma unroll
+          for (int e = 0; e < V; ++e) other[e] = other[e] * r * w2[e];
+        }
+#pragma unroll
+        for (int e = 0; e < V; ++e) {
+          float a, b;
+          rotate_pair(first ? f[e] : other[e], first ? other[e] : f[e], c4[e], s4[e], a, b);
+          f[e] = first ? a : b;
+        }
       } else {
 #pragma unroll
         for (int e = 0; e < V; ++e) {

@@ -26,7 +26,7 @@ using namespace kvf;
 namespace {
 
 constexpr float READ_EPS = 1e-6f;  // joins the divisor of the read-out
-constexpr int GATE_CHUNK = 256;    // tokens a CTA of the gates kernel takes at a time
+constexpr int GATE_CHUNK = 1024;   // tokens a CTA of the gates kernel takes at a time, at most
 
 template <typename T, int V> struct Run;
 template <typename T> struct Run<T, 1> {
@@ -78,6 +78,7 @@ struct GateParams {
 // (log input gate, log forget gate) of token n and head h
 __device__ __forceinline__ void log_gates(const GateParams& p, long long n, int h, float& li, float& lf) {
   float zi = 0.f, zf = 0.f;
+#pragma unroll 8
   for (int s = 0; s < p.nsplit; ++s) {
     const float* row = p.z + (size_t)s * p.split_stride + n * p.ldz;
     zi += row[h];
@@ -101,13 +102,13 @@ __global__ void __launch_bounds__(GATE_CHUNK) memory_gates_kernel(const GatePara
   pdl_launch();
   pdl_wait();
   __shared__ __align__(16) float fs[GATE_CHUNK], is[GATE_CHUNK], ms[GATE_CHUNK + 1];
-  const int h = blockIdx.x, b = blockIdx.y, t = threadIdx.x;
+  const int h = blockIdx.x, b = blockIdx.y, t = threadIdx.x, chunk = blockDim.x;
   const int begin = p.qsl[b], len = p.qsl[b + 1] - begin, slot = p.slots[b];
   if (len <= 0 || slot < 0) return;
   float* mem = p.m + (size_t)slot * p.state_stride + h;
   if (t == 0) ms[0] = *mem;
-  for (int t0 = 0; t0 < len; t0 += GATE_CHUNK) {
-    const int n = min(GATE_CHUNK, len - t0);
+  for (int t0 = 0; t0 < len; t0 += chunk) {
+    const int n = min(chunk, len - t0);
     float li = 0.f, lf = 0.f;
     if (t < n) log_gates(p, begin + t0 + t, h, li, lf);
     fs[t] = lf;
@@ -144,13 +145,15 @@ struct PrepareParams {
   float* vn;      // [N][H * dvx]
 };
 
-// The token's numbers widened to float; `in`: the inflow of every head.
+// The numbers of heads h0 .. h1 - 1 of a token widened to float; `in`: their inflow.
 template <typename T, int V>
-__device__ __forceinline__ void widen(const PrepareParams& p, long long n, int H, const float* in) {
+__device__ __forceinline__ void widen(const PrepareParams& p, long long n, int H, int h0, int h1, const float* in) {
   const T* row = (const T*)p.x + n * p.ldx;
-  const int qk = H * p.dk, all = 2 * qk + H * p.dvx;
-  for (int c = threadIdx.x * V; c < all; c += blockDim.x * V) {
+  const int qk = H * p.dk, part = (h1 - h0) * p.dk, all = 2 * part + (h1 - h0) * p.dvx;
+  for (int u0 = threadIdx.x * V; u0 < all; u0 += blockDim.x * V) {
     float f[V];
+    // the place among all q, then all k, then all v columns
+    const int c = u0 < part ? h0 * p.dk + u0 : u0 < 2 * part ? qk + h0 * p.dk + (u0 - part) : 2 * qk + h0 * p.dvx + (u0 - 2 * part);
     if (c < qk) {
       Run<T, V>::load(row + p.q_off + c, f);
 #pragma unroll
@@ -161,7 +164,7 @@ __device__ __forceinline__ void widen(const PrepareParams& p, long long n, int H
       Run<float, V>::store(p.kn + n * qk + (c - qk), f);
     } else {
       const int u = c - 2 * qk, h = u / p.dvx, j = u - h * p.dvx;
-      const float g = in[h];
+      const float g = in[h - h0];
       if (j < p.dv) {
         Run<T, V>::load(row + p.v_off + h * p.dv + j, f);
 #pragma unroll
@@ -179,28 +182,30 @@ template <typename T, int V>
 __global__ void __launch_bounds__(256) memory_prepare_kernel(const PrepareParams p, int H, const float* __restrict__ inflow) {
   pdl_launch();
   pdl_wait();
-  widen<T, V>(p, blockIdx.x, H, inflow + (size_t)blockIdx.x * H);
+  widen<T, V>(p, blockIdx.x, H, 0, H, inflow + (size_t)blockIdx.x * H);
 }
 
-// Gates and widening of a step in which no sequence brings more than one token: a CTA per sequence.
+// Gates and widening of a step in which no sequence brings more than one token: a CTA per sequence and STEP_HEADS heads.
+constexpr int STEP_HEADS = 4;
 template <typename T, int V>
 __global__ void __launch_bounds__(256) memory_step_kernel(const PrepareParams p, const GateParams g) {
   pdl_launch();
-  extern __shared__ float in[];  // [H]
+  __shared__ float in[STEP_HEADS];
   pdl_wait();
   const int b = blockIdx.x, n = g.qsl[b], slot = g.slots[b];
   if (g.qsl[b + 1] - n != 1 || slot < 0) return;
-  for (int h = threadIdx.x; h < g.H; h += blockDim.x) {
+  const int h0 = blockIdx.y * STEP_HEADS, h1 = min(g.H, h0 + STEP_HEADS);
+  for (int h = h0 + threadIdx.x; h < h1; h += blockDim.x) {
     float* mem = g.m + (size_t)slot * g.state_stride + h;
     float li, lf;
     log_gates(g, n, h, li, lf);
     const float before = *mem, m = fmaxf(lf + before, li);
     leave_gates(g, n, h, li, lf, before, m);
-    in[h] = expf(li - m);
+    in[h - h0] = expf(li - m);
     *mem = m;
   }
   __syncthreads();
-  widen<T, V>(p, n, g.H, in);
+  widen<T, V>(p, n, g.H, h0, h1, in);
 }
 
 // A warp per (token, head).  out = y / sqrt(mean(y^2) + eps) * w * act(gate), y the read-out over its divisor; act: 0 none, 2 the
@@ -217,14 +222,14 @@ __global__ void __launch_bounds__(128) memory_read_kernel(const float* __restric
   const long long n = pair / H;
   const int h = (int)(pair - n * H);
   const float* row = o + n * ldo + (size_t)h * dvx;
-  const float size = fmaxf(fabsf(row[dv]), floor_[pair]) + READ_EPS;
+  const float one_over = 1.f / (fmaxf(fabsf(row[dv]), floor_[pair]) + READ_EPS);
   float ss = 0.f;
   for (int j = lane * V; j < dv; j += 32 * V) {
     float f[V];
     Run<float, V>::load(row + j, f);
 #pragma unroll
     for (int e = 0; e < V; ++e) {
-      const float y = f[e] / size;
+      const float y = f[e] * one_over;
       ss = fmaf(y, y, ss);
     }
   }
@@ -236,7 +241,7 @@ __global__ void __launch_bounds__(128) memory_read_kernel(const float* __restric
     Run<float, V>::load(row + j, f);
     Run<float, V>::load(w + (size_t)h * dv + j, wv);
 #pragma unroll
-    for (int e = 0; e < V; ++e) f[e] = f[e] / size * r * wv[e];
+    for (int e = 0; e < V; ++e) f[e] = f[e] * one_over * r * wv[e];
     if (g) {
       float z[V];
       Run<T, V>::load(g + j, z);
@@ -259,10 +264,10 @@ int memory_run(const GateParams& g0, const PrepareParams& p, float* state, float
                    aligned(p.qn, 16) && aligned(p.kn, 16) && aligned(p.vn, 16);
   int rc;
   if (max_q_len == 1) {
-    rc = launch(vec ? memory_step_kernel<T, 4> : memory_step_kernel<T, 1>, dim3(B), dim3(256), (size_t)H * sizeof(float), st, p, g);
+    rc = launch(vec ? memory_step_kernel<T, 4> : memory_step_kernel<T, 1>, dim3(B, (H + STEP_HEADS - 1) / STEP_HEADS), dim3(256), 0, st, p, g);
     if (rc) return rc;
   } else {
-    rc = launch(memory_gates_kernel, dim3(H, B), dim3(GATE_CHUNK), 0, st, g);
+    rc = launch(memory_gates_kernel, dim3(H, B), dim3(max_q_len > 0 && max_q_len <= 256 ? 256 : GATE_CHUNK), 0, st, g);
     if (rc) return rc;
     rc = launch(vec ? memory_prepare_kernel<T, 4> : memory_prepare_kernel<T, 1>, dim3((unsigned)N), dim3(256), 0, st, p, H, (const float*)g.inflow);
     if (rc) return rc;

@@ -293,6 +293,118 @@ __global__ void __launch_bounds__(256) branch_norm_mean_kernel(const BranchParam
   }
 }
 
+// Two branches whose rows start on 16-byte boundaries, at most 4 * TH * NIT numbers each: a thread owns four neighbouring numbers of up to
+// NIT stretches of a row and keeps them in registers; slices of split products are asked for several at a time and added in slice
+// order; both sums of squares go through one pair of barriers.
+template <typename T> struct Four;
+template <> struct Four<float> {
+  static __device__ __forceinline__ void load(const float* p, float* f) {
+    const float4 v = *reinterpret_cast<const float4*>(p);
+    f[0] = v.x; f[1] = v.y; f[2] = v.z; f[3] = v.w;
+  }
+  static __device__ __forceinline__ void store(float* p, const float* f) { *reinterpret_cast<float4*>(p) = make_float4(f[0], f[1], f[2], f[3]); }
+};
+template <> struct Four<bf16> {
+  static __device__ __forceinline__ void load(const bf16* p, float* f) {
+    const uint2 u = *reinterpret_cast<const uint2*>(p);
+    const float2 a = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.x));
+    const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&u.y));
+    f[0] = a.x; f[1] = a.y; f[2] = b.x; f[3] = b.y;
+  }
+  static __device__ __forceinline__ void store(bf16* p, const float* f) {
+    const __nv_bfloat162 a = __floats2bfloat162_rn(f[0], f[1]), b = __floats2bfloat162_rn(f[2], f[3]);
+    uint2 u;
+    u.x = *reinterpret_cast<const uint32_t*>(&a);
+    u.y = *reinterpret_cast<const uint32_t*>(&b);
+    *reinterpret_cast<uint2*>(p) = u;
+  }
+};
+
+template <typename T, int NIT, int TH>
+__global__ void __launch_bounds__(TH) branch_norm_mean_pair_kernel(const BranchParams p) {
+  pdl_launch();
+  pdl_wait();
+  __shared__ float red[64];
+  const size_t n = blockIdx.x;
+  const int W = p.W;
+  bool live[NIT];
+  float v[2][NIT][4], w[2][NIT][4], h[NIT][4];
+#pragma unroll
+  for (int it = 0; it < NIT; ++it) {
+    const int c = (it * TH + threadIdx.x) * 4;
+    live[it] = c < W;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) v[0][it][e] = v[1][it][e] = w[0][it][e] = w[1][it][e] = h[it][e] = 0.f;
+    if (!live[it]) continue;
+#pragma unroll
+    for (int b = 0; b < 2; ++b) {
+      Four<float>::load(p.w[b] + c, w[b][it]);
+      if (p.y[b]) Four<T>::load((const T*)p.y[b] + n * W + c, v[b][it]);
+    }
+    if (p.resid) Four<float>::load(p.resid + n * W + c, h[it]);
+  }
+#pragma unroll
+  for (int b = 0; b < 2; ++b) {
+    if (p.y[b]) continue;
+    constexpr int SL = NIT == 1 ? 8 : NIT == 2 ? 4 : 2;
+    const float* pr = p.partials[b] + n * W;
+    for (int s0 = 0; s0 < p.nsplit[b]; s0 += SL) {
+      float t[SL][NIT][4];
+#pragma unroll
+      for (int k = 0; k < SL; ++k)
+#pragma unroll
+        for (int it = 0; it < NIT; ++it) {
+          // no branch around a load: past the last slice it is read once more, past the row's end its start, and neither is used
+          const int s = min(s0 + k, p.nsplit[b] - 1), c = live[it] ? (it * TH + threadIdx.x) * 4 : 0;
+          Four<float>::load(pr + (size_t)s * p.split_stride[b] + c, t[k][it]);
+        }
+#pragma unroll
+      for (int k = 0; k < SL; ++k)
+#pragma unroll
+        for (int it = 0; it < NIT; ++it)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) v[b][it][e] += live[it] && s0 + k < p.nsplit[b] ? t[k][it][e] : 0.f;
+    }
+  }
+  float sq[2] = {0.f, 0.f};
+#pragma unroll
+  for (int b = 0; b < 2; ++b)
+#pragma unroll
+    for (int it = 0; it < NIT; ++it)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) sq[b] = fmaf(v[b][it][e], v[b][it][e], sq[b]);
+  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  sq[0] = warp_sum(sq[0]);
+  sq[1] = warp_sum(sq[1]);
+  if (lane == 0) {
+    red[warp] = sq[0];
+    red[32 + warp] = sq[1];
+  }
+  __syncthreads();
+  const float i0 = 0.5f / sqrtf(warp_sum(lane < TH / 32 ? red[lane] : 0.f) / (float)W + p.eps);
+  const float i1 = 0.5f / sqrtf(warp_sum(lane < TH / 32 ? red[32 + lane] : 0.f) / (float)W + p.eps);
+#pragma unroll
+  for (int it = 0; it < NIT; ++it) {
+    if (!live[it]) continue;
+    const int c = (it * TH + threadIdx.x) * 4;
+    float f[4];
+#pragma unroll
+    for (int e = 0; e < 4; ++e) f[e] = h[it][e] + (v[0][it][e] * i0 * w[0][it][e] + v[1][it][e] * i1 * w[1][it][e]);
+    if (p.resid)
+      Four<float>::store(p.resid + n * W + c, f);
+    else
+      Four<T>::store((T*)p.out + n * W + c, f);
+  }
+}
+
+template <typename T>
+bool branch_pair_ok(const BranchParams& p) {
+  auto al = [](const void* q, size_t b) { return q == nullptr || ((uintptr_t)q % b) == 0; };
+  bool ok = p.nb == 2 && p.W % 4 == 0 && p.W <= 4096 && al(p.out, 4 * sizeof(T)) && al(p.resid, 16);
+  for (int b = 0; b < p.nb; ++b) ok = ok && al(p.w[b], 16) && al(p.y[b], 4 * sizeof(T)) && (p.y[b] || (al(p.partials[b], 16) && p.split_stride[b] % 4 == 0));
+  return ok;
+}
+
 // ---------------------------------------------------------------- soft cap
 __global__ void softcap_kernel(float* __restrict__ x, size_t n, float cap) {
   pdl_launch();
@@ -412,6 +524,16 @@ int launch_hc(const HcParams& p, int n_rows, int S, cudaStream_t st) {
       if (!p.y[b] && !p.partials[b]) return (int)cudaErrorInvalidValue;                                                \
     }                                                                                                                  \
     p.nb = nb; p.W = W; p.eps = eps; p.out = out; p.resid = resid;                                                     \
+    if (branch_pair_ok<T>(p)) {                                                                                        \
+      const dim3 g((unsigned)N);                                                                                       \
+      /* few rows of slices: a thread for every four numbers, so that all slices of a row are asked for at once */     \
+      const bool few = !p.y[0] && !p.y[1] && N <= 148;                                                                 \
+      if (W <= 1024) return launch(branch_norm_mean_pair_kernel<T, 1, 256>, g, dim3(256), 0, st, p);                   \
+      if (W <= 2048) return few ? launch(branch_norm_mean_pair_kernel<T, 1, 512>, g, dim3(512), 0, st, p)              \
+                                : launch(branch_norm_mean_pair_kernel<T, 2, 256>, g, dim3(256), 0, st, p);             \
+      return few ? launch(branch_norm_mean_pair_kernel<T, 1, 1024>, g, dim3(1024), 0, st, p)                           \
+                 : launch(branch_norm_mean_pair_kernel<T, 4, 256>, g, dim3(256), 0, st, p);                            \
+    }                                                                                                                  \
     if (W <= 8192) {                                                                                                   \
       const dim3 g((unsigned)N);                                                                                       \
       /* small CTAs, so that many rows share an SM and their loads overlap */                                          \

@@ -29,9 +29,9 @@ _SIGNATURES = {
     "kvf_paged_attention_mma_biased_bf16": "pppppppiiiiiiiiifiipifpp",
     "kvf_latent_attention_bf16": "ppppppiiiiiiiiifiiiippp",
     "kvf_paged_attention_decode_biased_bf16": "pppppppiiiiiiiifiiiipppipifpp",
-    "kvf_paged_attention_tcgen05_bf16": "pppppppiiiiiiiiilfipipp",
+    "kvf_paged_attention_tcgen05_bf16": "pppppppiiiiiiiiilfipippp",
     "kvf_paged_attention_decode_fused_bf16": "pppppppiiiiiiiifiiiipppp",
-    "kvf_paged_attention_decode_tma_bf16": "pppppppiiiiiiiilfiiiippppiip",
+    "kvf_paged_attention_decode_tma_bf16": "pppppppiiiiiiiilfiiiippppiipp",
     "kvf_gemm_nt_f32": "pppiiiiiip",
     "kvf_gemm_skinny_bf16": "pppiiiiiiiilpp",
     "kvf_set_pdl": "i",
@@ -587,7 +587,7 @@ def paged_attention(
     distance), ``bias`` (added to the scaled scores, by distance and head), ``softcap`` (``c > 0``: a scaled
     score ``s`` becomes ``c * tanh(s / c)``) and ``sinks`` (float ``[nh]``: ``exp(sinks[h])`` joins the softmax's
     denominator of head ``h``; it has no key and no value) are taken by the FP32-pipe kernel and, for bfloat16
-    heads of 64 or 128 with values as wide, by the mma.sync kernels.
+    heads of 64 or 128 with values as wide, by the mma.sync kernels; ``sinks`` without the others also by the tcgen05 and TMA kernels.
 
     ``q``: rows of ``q_stride`` elements whose first ``nh*d`` are the query heads; ``out``:
     ``[N, nh*d]``.  With ``scratch`` (and every sequence holding one query) the decode form
@@ -607,7 +607,15 @@ def paged_attention(
     """
     s = _suffix(q.dtype)
     _rows2d(q, None, "q")
-    capped = float(softcap) > 0.0 or sinks is not None
+    # sinks alone, on a shape that the tcgen05 kernel (many queries) or the TMA kernel (decoding) takes: theirs
+    if sinks is not None and kernel in ("auto", "tcgen05", "tma"):
+        if scratch is None:
+            takes_sinks = tcgen05_attention_supported(q.dtype, nh, nkv, d, False) and max_q_len > 1 and (q_stride or q.stride(0)) % 8 == 0 and out.shape[-1] % 8 == 0
+        else:
+            takes_sinks = len(scratch) > 2 and tma_decode_supported(q.dtype, nh, nkv, d, kcache.shape[2], kcache.shape[0])
+    else:
+        takes_sinks = False
+    capped = float(softcap) > 0.0 or (sinks is not None and not takes_sinks)
     if chunk:
         if window or keep_first or chunk < 0:
             raise ValueError("paged_attention: chunk is a positive number of positions, without a window and kept first keys")
@@ -739,7 +747,7 @@ def paged_attention(
             _fn(name)(
                 _ptr(q), _ptr(out), _ptr(kcache), _ptr(vcache), _ptr(block_tables), _ptr(qsl), _ptr(ctx_lens),
                 num_seqs, max_q_len, q_stride, out.shape[-1], bt_stride, nh, nkv, d, block_size, int(kcache.shape[0]),
-                float(scale), int(window), _ptr(tiles), n_tiles, _ptr(err), _stream(),
+                float(scale), int(window), _ptr(tiles), n_tiles, _ptr(err), _ptr(sinks), _stream(),
             ),
             name,
         )  # fmt: skip
@@ -753,7 +761,7 @@ def paged_attention(
             _fn(name)(
                 _ptr(q), _ptr(out), _ptr(kcache), _ptr(vcache), _ptr(block_tables), _ptr(qsl), _ptr(ctx_lens),
                 num_seqs, q_stride, out.shape[-1], bt_stride, nh, nkv, d, block_size, int(kcache.shape[0]), float(scale),
-                int(window), split, max_splits, grid_splits, _ptr(pa), _ptr(pm), _ptr(tickets), _ptr(err), int(bool(cluster)) | (2 if single_only else 0), int(wave_target), _stream(),
+                int(window), split, max_splits, grid_splits, _ptr(pa), _ptr(pm), _ptr(tickets), _ptr(err), int(bool(cluster)) | (2 if single_only else 0), int(wave_target), _ptr(sinks), _stream(),
             ),
             name,
         )  # fmt: skip

@@ -246,9 +246,10 @@ class PagedAttention(Mixer):
         self._tickets = torch.zeros(max(1, rt.max_seqs) * self.nkv, dtype=torch.int32, device=rt.device)
         # the kernel of prompts and mixed batches takes its tiles of queries from a list made with the step
         self._query_tile = None
-        # kept first keys, a bias on the scores, capped scores and sinks are not the tcgen05 kernel's
-        self.plain_scores = self.bias is None and not self.keep_first and not self.softcap and self.sinks is None
-        if self.plain_scores and self.dv == self.d and ops.tcgen05_attention_supported(rt.dtype, self.nh, self.nkv, self.d, False):
+        # kept first keys, a bias on the scores and capped scores are not the tcgen05 kernel's (sinks alone are)
+        tiled = self.bias is None and not self.keep_first and not self.softcap
+        self.plain_scores = tiled and self.sinks is None
+        if tiled and self.dv == self.d and ops.tcgen05_attention_supported(rt.dtype, self.nh, self.nkv, self.d, False):
             self._query_tile = ops.tcgen05_query_tile(self.nh, self.nkv)
             rt.query_tile_sizes.add(self._query_tile)
 

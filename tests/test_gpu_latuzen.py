@@ -814,3 +814,49 @@ def test_a_parallel_layer_hands_on_the_slices_of_both_parts(dtype, n):
     if left is not ops.ADDED:
         got = got + as_float(left, n).cpu().double()
     assert rel_rows(got, want) < part_tol(dtype)
+
+
+@pytest.mark.parametrize("d", [64, 128])
+@pytest.mark.parametrize("nh,nkv,window,lens", [(8, 2, 0, [150, 3, 70]), (4, 4, 40, [90, 1, 33, 129]), (16, 2, 70, [700, 20])])
+def test_learned_sinks_on_the_tensor_core_kernels(d, nh, nkv, window, lens):
+    """Sinks of every size (far below every score to far above) as the tcgen05 kernel takes them for prompts and the TMA kernel for
+    decoding, its ranges merged through the scratch, through a cluster, or a single one."""
+    from kvforge_b200 import ops
+
+    g = torch.Generator().manual_seed(d + nh)
+    bs, scale, dev = 16, d**-0.5, "cuda"
+    i32 = lambda z: torch.tensor(z, dtype=torch.int32, device=dev)  # noqa: E731
+    sinks = torch.tensor([[-50.0, 0.0, 1.5, 3.0, 20.0][h % 5] for h in range(nh)])
+    n = sum(lens)
+    q, k, v = (1.5 * torch.randn(n, h, d, generator=g).bfloat16() for h in (nh, nkv, nkv))
+    per = -(-max(lens) // bs)
+    tables = torch.randperm(len(lens) * per, generator=g).reshape(len(lens), per)
+    kc, vc = (torch.zeros(len(lens) * per, nkv, bs, d, dtype=torch.bfloat16) for _ in range(2))
+    want, at = torch.zeros(n, nh, d, dtype=torch.float64), 0
+    for b, m in enumerate(lens):
+        rows = slice(at, at + m)
+        for p in range(m):
+            kc[tables[b, p // bs], :, p % bs], vc[tables[b, p // bs], :, p % bs] = k[at + p], v[at + p]
+        see = plain.window_mask(m, window or m)
+        for h in range(nh):
+            s = (q[rows, h].double() @ k[rows, h // (nh // nkv)].double().T * scale).masked_fill(~see, float("-inf"))
+            p = torch.softmax(torch.cat([s, torch.full((m, 1), float(sinks[h]), dtype=torch.float64)], dim=1), dim=1)[:, :m]
+            want[rows, h] = p @ v[rows, h // (nh // nkv)].double()
+        at += m
+    qsl = i32([0] + [sum(lens[: i + 1]) for i in range(len(lens))])
+    args = (kc.cuda(), vc.cuda(), tables.int().cuda())
+    err = torch.zeros(1, dtype=torch.int32, device=dev)
+    out = torch.zeros(n, nh * d, dtype=torch.bfloat16, device=dev)
+    ops.paged_attention(q.reshape(n, -1).cuda(), out, *args, qsl, i32(lens), len(lens), max(lens), nh, nkv, d, scale, window=window, err=err, sinks=sinks.cuda(), kernel="tcgen05")
+    assert int(err) == 0
+    assert rel_rows(out.float().cpu(), want.reshape(n, -1)) < 2e-2
+    last = [sum(lens[: i + 1]) - 1 for i in range(len(lens))]
+    for split, cluster in ((64, False), (64, True), (1024, False), (1024, True)):
+        b = len(lens)
+        sa, sm = ops.attention_scratch_shapes(b, nh, d, max(lens), split)
+        scratch = (torch.empty(sa, device=dev), torch.empty(sm, device=dev), torch.zeros(b * nkv, dtype=torch.int32, device=dev))
+        out = torch.zeros(b, nh * d, dtype=torch.bfloat16, device=dev)
+        ops.paged_attention(q[last].reshape(b, -1).cuda(), out, *args, i32(list(range(b + 1))), i32(lens), b, 1, nh, nkv, d, scale, window=window, err=err, sinks=sinks.cuda(),
+                            scratch=scratch, max_context=max(lens), split_size=split, cluster=cluster, kernel="tma")  # fmt: skip
+        assert int(err) == 0
+        assert rel_rows(out.float().cpu(), want[last].reshape(b, -1)) < 2e-2, (split, cluster)
