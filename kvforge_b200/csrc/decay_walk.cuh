@@ -65,10 +65,10 @@ __global__ void __launch_bounds__(256) decay_walk_kernel(const float* __restrict
   const int kh = h / heads_per_key, key_heads = H / heads_per_key;
 
   float* sbase = state + (size_t)slot * state_stride + (size_t)h * dk * dv + c0;
-  // whole tiles of whole rows go four numbers at a time
-  const bool tile4 = dkp == dk && ncol == CT && (CT & 3) == 0 && (dv & 3) == 0 && (((uintptr_t)sbase) & 15) == 0;
+  // whole rows go four numbers at a time (columns of the CTA beyond the tile's hold whatever lies there, and nothing reads them)
+  const bool tile4 = dkp == dk && (ncol & 3) == 0 && (CT & 3) == 0 && (dv & 3) == 0 && (((uintptr_t)sbase) & 15) == 0;
   if (tile4) {
-    const int c4 = CT >> 2;
+    const int c4 = ncol >> 2;
     for (int idx = tid; idx < dk * c4; idx += nthreads) {
       const int r = idx / c4, c = (idx - r * c4) << 2;
       const float4 t4 = *reinterpret_cast<const float4*>(sbase + (size_t)r * dv + c);
@@ -167,7 +167,7 @@ __global__ void __launch_bounds__(256) decay_walk_kernel(const float* __restrict
   for (int i = 0; i < R; ++i) St[(((i >> 2) * KS + s) * 4 + (i & 3)) * lds + col] = S[i];
   __syncthreads();
   if (tile4) {
-    const int c4 = CT >> 2;
+    const int c4 = ncol >> 2;
     for (int idx = tid; idx < dk * c4; idx += nthreads) {
       const int r = idx / c4, c = (idx - r * c4) << 2;
       const float* d = St + r * lds + c;

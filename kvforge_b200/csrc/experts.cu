@@ -49,64 +49,11 @@ template <> __device__ __forceinline__ void load8<bf16>(const bf16* src, float* 
   bf16x8_to_float(*reinterpret_cast<const uint4*>(src), dst);
 }
 
-// One CTA per RT tokens (one token and up to 32 warps a CTA while a step has few, four tokens and eight warps when it has many).  The warps share out the experts: a logit is one warp's dot product (a lane
-// adds its products in the order of the columns, then the lanes are summed in a fixed tree), so it does not depend on
-// the batch; a row of the router is read once for the CTA's tokens.  Then warp t chooses for token t.  Shared memory
-// per token: scores [E], choice scores [E], group scores [G], group flags [G].
-template <typename T, int RT>
-__global__ void __launch_bounds__(RT == 1 ? 1024 : 256) moe_route_kernel(const T* __restrict__ x, long long x_stride,
-                                                         const float* __restrict__ router, const float* __restrict__ correction,
-                                                         int n_tokens, int W, int E, int top, int groups, int keep,
-                                                         float norm_eps, int vec, int flags, int* __restrict__ ids, float* __restrict__ wts,
-                                                         const float* __restrict__ logit_bias, float scale) {
-  pdl_launch();
-  pdl_wait();
-  extern __shared__ float sm[];
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
-  const int n0 = blockIdx.x * RT;
-  const int per_token = 2 * E + 2 * groups;
-  for (int e = warp; e < E; e += warps) {
-    const float* wr = router + (size_t)e * W;
-    float z[RT];
-#pragma unroll
-    for (int t = 0; t < RT; ++t) z[t] = 0.f;
-    if (vec) {
-      for (int j = lane * 8; j < W; j += 256) {
-        float wv[8];
-        load8<float>(wr + j, wv);
-#pragma unroll
-        for (int t = 0; t < RT; ++t) {
-          if (n0 + t >= n_tokens) break;
-          float xv[8];
-          load8<T>(x + (size_t)(n0 + t) * x_stride + j, xv);
-#pragma unroll
-          for (int i = 0; i < 8; ++i) z[t] = fmaf(xv[i], wv[i], z[t]);
-        }
-      }
-    } else {
-      for (int j = lane; j < W; j += 32) {
-        const float wv = wr[j];
-#pragma unroll
-        for (int t = 0; t < RT; ++t)
-          if (n0 + t < n_tokens) z[t] = fmaf(to_float<T>(x[(size_t)(n0 + t) * x_stride + j]), wv, z[t]);
-      }
-    }
-#pragma unroll
-    for (int t = 0; t < RT; ++t) {
-      const float zt = warp_sum(z[t]) + (logit_bias ? logit_bias[e] : 0.f);
-      if (lane == 0) {
-        // flags bit 0: the scores are a softmax over all experts, made below from the logits kept here;
-        // bit 2: the logits themselves rank the experts, and the weights are a softmax over the chosen logits
-        const float s = (flags & 5) ? zt : 1.f / (1.f + expf(-zt));
-        sm[t * per_token + e] = s;
-        sm[t * per_token + E + e] = s + (correction ? correction[e] : 0.f);
-      }
-    }
-  }
-  __syncthreads();
-  if (warp >= RT || n0 + warp >= n_tokens) return;
-  const int n = n0 + warp;
-  float* sc = sm + warp * per_token;
+// What follows the logits, by one warp for token n: scores and choice scores in `sm` (scores [E], choice scores [E], group scores [G], group
+// flags [G]) become the chosen experts and their weights.
+__device__ __forceinline__ void choose_experts(float* sm, int n, int lane, const float* __restrict__ correction, int E, int top, int groups, int keep,
+                                               float norm_eps, int flags, int* __restrict__ ids, float* __restrict__ wts, float scale) {
+  float* sc = sm;
   float* ch = sc + E;
   float* gs = ch + E;
   float* ga = gs + groups;
@@ -198,6 +145,140 @@ __global__ void __launch_bounds__(RT == 1 ? 1024 : 256) moe_route_kernel(const T
   if ((flags & 2) && scale == 1.f) return;  // the weights are the chosen scores as they are
   const float inv = (flags & 2) ? scale : scale / (total + norm_eps);
   for (int k = lane; k < top; k += 32) my_w[k] *= inv;
+}
+
+// One CTA per RT tokens: one token and up to 32 warps a CTA while a step has few; four tokens and eight warps when it has many and the
+// kernel below does not take the sizes.  The warps share out the experts: a logit is one warp's dot product (a lane
+// adds its products in the order of the columns, then the lanes are summed in a fixed tree), so it does not depend on
+// the batch; a row of the router is read once for the CTA's tokens.  Then warp t chooses for token t.  Shared memory
+// per token: scores [E], choice scores [E], group scores [G], group flags [G].
+template <typename T, int RT>
+__global__ void __launch_bounds__(RT == 1 ? 1024 : 256) moe_route_kernel(const T* __restrict__ x, long long x_stride,
+                                                         const float* __restrict__ router, const float* __restrict__ correction,
+                                                         int n_tokens, int W, int E, int top, int groups, int keep,
+                                                         float norm_eps, int vec, int flags, int* __restrict__ ids, float* __restrict__ wts,
+                                                         const float* __restrict__ logit_bias, float scale) {
+  pdl_launch();
+  pdl_wait();
+  extern __shared__ float sm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int n0 = blockIdx.x * RT;
+  const int per_token = 2 * E + 2 * groups;
+  for (int e = warp; e < E; e += warps) {
+    const float* wr = router + (size_t)e * W;
+    float z[RT];
+#pragma unroll
+    for (int t = 0; t < RT; ++t) z[t] = 0.f;
+    if (vec) {
+      for (int j = lane * 8; j < W; j += 256) {
+        float wv[8];
+        load8<float>(wr + j, wv);
+#pragma unroll
+        for (int t = 0; t < RT; ++t) {
+          if (n0 + t >= n_tokens) break;
+          float xv[8];
+          load8<T>(x + (size_t)(n0 + t) * x_stride + j, xv);
+#pragma unroll
+          for (int i = 0; i < 8; ++i) z[t] = fmaf(xv[i], wv[i], z[t]);
+        }
+      }
+    } else {
+      for (int j = lane; j < W; j += 32) {
+        const float wv = wr[j];
+#pragma unroll
+        for (int t = 0; t < RT; ++t)
+          if (n0 + t < n_tokens) z[t] = fmaf(to_float<T>(x[(size_t)(n0 + t) * x_stride + j]), wv, z[t]);
+      }
+    }
+#pragma unroll
+    for (int t = 0; t < RT; ++t) {
+      const float zt = warp_sum(z[t]) + (logit_bias ? logit_bias[e] : 0.f);
+      if (lane == 0) {
+        // flags bit 0: the scores are a softmax over all experts, made below from the logits kept here;
+        // bit 2: the logits themselves rank the experts, and the weights are a softmax over the chosen logits
+        const float s = (flags & 5) ? zt : 1.f / (1.f + expf(-zt));
+        sm[t * per_token + e] = s;
+        sm[t * per_token + E + e] = s + (correction ? correction[e] : 0.f);
+      }
+    }
+  }
+  __syncthreads();
+  if (warp >= RT || n0 + warp >= n_tokens) return;
+  choose_experts(sm + warp * per_token, n0 + warp, lane, correction, E, top, groups, keep, norm_eps, flags, ids, wts, scale);
+}
+
+// The same for steps of many tokens: a CTA takes MANY tokens, whose rows it holds as floats in shared memory, and a warp makes the
+// logits of EPW experts of all of them at a time, so that a row of the router is read once for MANY tokens and a row of x once for EPW
+// experts.  A lane adds its products in the same order as above.
+constexpr int MANY = 8, EPW = 4, MANY_WARPS = 16;
+
+template <typename T>
+__global__ void __launch_bounds__(MANY_WARPS * 32) moe_route_many_kernel(const T* __restrict__ x, long long x_stride,
+                                                              const float* __restrict__ router, const float* __restrict__ correction,
+                                                              int n_tokens, int W, int E, int top, int groups, int keep, float norm_eps,
+                                                              int flags, int* __restrict__ ids, float* __restrict__ wts,
+                                                              const float* __restrict__ logit_bias, float scale) {
+  pdl_launch();
+  pdl_wait();
+  extern __shared__ __align__(16) float sm[];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, warps = blockDim.x >> 5;
+  const int n0 = blockIdx.x * MANY, rows = min(MANY, n_tokens - n0);
+  const int Wp = (W + 255) & ~255;  // rows padded with zeros
+  float* xs = sm;  // [MANY][Wp]; within 256 numbers the first halves of the lanes' eights, then the second halves
+  float* per_token = sm + (size_t)MANY * Wp;
+  const int stride = 2 * E + 2 * groups;
+  for (int idx = threadIdx.x; idx < MANY * (Wp >> 3); idx += blockDim.x) {
+    const int t = idx / (Wp >> 3), o = idx - t * (Wp >> 3), j = o * 8;
+    float f[8];
+#pragma unroll
+    for (int e = 0; e < 8; ++e) f[e] = 0.f;
+    if (t < rows && j < W) load8<T>(x + (size_t)(n0 + t) * x_stride + j, f);
+    float* dst = xs + (size_t)t * Wp + (o >> 5) * 256 + (o & 31) * 4;
+    *reinterpret_cast<float4*>(dst) = make_float4(f[0], f[1], f[2], f[3]);
+    *reinterpret_cast<float4*>(dst + 128) = make_float4(f[4], f[5], f[6], f[7]);
+  }
+  __syncthreads();
+  for (int e0 = warp * EPW; e0 < E; e0 += warps * EPW) {
+    float z[EPW][MANY];
+#pragma unroll
+    for (int e = 0; e < EPW; ++e)
+#pragma unroll
+      for (int t = 0; t < MANY; ++t) z[e][t] = 0.f;
+    for (int j = lane * 8; j < Wp; j += 256) {
+#pragma unroll
+      for (int half = 0; half < 2; ++half) {
+        float4 w[EPW];
+#pragma unroll
+        for (int e = 0; e < EPW; ++e) {
+          // (a row or a column past the last is the last one's, and its sums are not used; x is zero there)
+          const int je = j < W ? j + 4 * half : 0;
+          w[e] = *reinterpret_cast<const float4*>(router + (size_t)min(e0 + e, E - 1) * W + je);
+        }
+#pragma unroll
+        for (int t = 0; t < MANY; ++t) {
+          const float4 v = *reinterpret_cast<const float4*>(xs + (size_t)t * Wp + (j >> 8) * 256 + half * 128 + lane * 4);
+#pragma unroll
+          for (int e = 0; e < EPW; ++e) z[e][t] = fmaf(v.w, w[e].w, fmaf(v.z, w[e].z, fmaf(v.y, w[e].y, fmaf(v.x, w[e].x, z[e][t]))));
+        }
+      }
+    }
+#pragma unroll
+    for (int e = 0; e < EPW; ++e) {
+      if (e0 + e >= E) continue;
+#pragma unroll
+      for (int t = 0; t < MANY; ++t) {
+        const float zt = warp_sum(z[e][t]) + (logit_bias ? logit_bias[e0 + e] : 0.f);
+        if (lane == 0) {
+          const float s = (flags & 5) ? zt : 1.f / (1.f + expf(-zt));  // as above
+          per_token[t * stride + e0 + e] = s;
+          per_token[t * stride + E + e0 + e] = s + (correction ? correction[e0 + e] : 0.f);
+        }
+      }
+    }
+  }
+  __syncthreads();
+  for (int t = warp; t < rows; t += warps)
+    choose_experts(per_token + t * stride, n0 + t, lane, correction, E, top, groups, keep, norm_eps, flags, ids, wts, scale);
 }
 
 // One CTA.  ids [P] -> order [P] (pairs by expert, those of identity experts (ids from E on) left out), tiles: (expert, first
@@ -624,6 +705,20 @@ int run_products<bf16>(const bf16* x, long long x_stride, const bf16* w_up, cons
     const size_t smem = (size_t)rt * (2 * E + 2 * groups) * sizeof(float);                                            \
     if (smem > 48 * 1024) return (int)cudaErrorInvalidValue;                                                          \
     const int vec = (W % 8 == 0) && (x_stride % 8 == 0) && ((((uintptr_t)x) | ((uintptr_t)router)) % 16 == 0);        \
+    const int Wp = (W + 255) & ~255;                                                                                  \
+    const size_t many = ((size_t)MANY * Wp + (size_t)MANY * (2 * E + 2 * groups)) * sizeof(float);                    \
+    if (rt > 1 && vec && many <= 200 * 1024) {                                                                        \
+      int warps = (E + EPW - 1) / EPW;                                                                                \
+      warps = warps < MANY ? MANY : warps > MANY_WARPS ? MANY_WARPS : warps;                                          \
+      if (many > 48 * 1024) {                                                                                         \
+        cudaError_t e = cudaFuncSetAttribute(moe_route_many_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize,   \
+                                             (int)many);                                                              \
+        if (e != cudaSuccess) return (int)e;                                                                          \
+      }                                                                                                               \
+      return launch(moe_route_many_kernel<T>, dim3((n_tokens + MANY - 1) / MANY), dim3(warps * 32), many, st,         \
+                    (const T*)x, x_stride, router, correction, n_tokens, W, E, top, groups, keep, norm_eps, flags,    \
+                    ids, wts, logit_bias, scale);                                                                     \
+    }                                                                                                                 \
     if (rt == 1)                                                                                                      \
       return launch(moe_route_kernel<T, 1>, dim3(n_tokens), dim3(E > 16 ? 1024 : E > 8 ? 512 : 256), smem, st, (const T*)x, x_stride, router,       \
                     correction, n_tokens, W, E, top, groups, keep, norm_eps, vec, flags, ids, wts, logit_bias,        \

@@ -23,9 +23,20 @@ namespace {
 // A CTA takes HEAD_WARPS heads of a token at a time (all of the token's when there are many tokens), and works out the token's
 // cosines and sines once.  A lane keeps its pairs in registers between the sum and the rotation.
 constexpr int HEAD_WARPS = 8;
-constexpr int HEAD_PAIRS = 4;  // pairs a lane holds: heads of up to 256
+constexpr int HEAD_PAIRS = 4;  // pairs a lane holds at most: heads of up to 256
 
-template <typename T>
+template <typename T> struct Two;
+template <> struct Two<float> {
+  static __device__ __forceinline__ float2 load(const float* p) { return *reinterpret_cast<const float2*>(p); }
+  static __device__ __forceinline__ void store(float* p, float a, float b) { *reinterpret_cast<float2*>(p) = make_float2(a, b); }
+};
+template <> struct Two<bf16> {
+  static __device__ __forceinline__ float2 load(const bf16* p) { return __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(p)); }
+  static __device__ __forceinline__ void store(bf16* p, float a, float b) { *reinterpret_cast<__nv_bfloat162*>(p) = __floats2bfloat162_rn(a, b); }
+};
+
+// PAIRS: pairs a lane holds.  SPLIT: the pairs that turn are (i, i + rot/2).  Rows and pages begin where a pair of numbers may.
+template <typename T, int PAIRS, bool SPLIT>
 __global__ void __launch_bounds__(HEAD_WARPS * 32) head_norm_cache_kernel(T* __restrict__ qkv, long long row_stride,
                                                                const int* __restrict__ positions,
                                                                const float* __restrict__ q_w, const float* __restrict__ k_w,
@@ -33,9 +44,9 @@ __global__ void __launch_bounds__(HEAD_WARPS * 32) head_norm_cache_kernel(T* __r
                                                                const int* __restrict__ slots, T* __restrict__ kcache,
                                                                T* __restrict__ vcache, int nh, int nkv, int dk,
                                                                int dv, int block_size, long long num_slots,
-                                                               int* __restrict__ err, int split_pairs,
-                                                               T* __restrict__ v_keep, const T* __restrict__ v_first,
-                                                               const float* __restrict__ v_lambda, float count, float magnitude) {
+                                                               int* __restrict__ err, T* __restrict__ v_keep,
+                                                               const T* __restrict__ v_first, const float* __restrict__ v_lambda,
+                                                               float count, float magnitude) {
   pdl_launch();
   extern __shared__ float turn[];  // [rot / 2] cosines, [rot / 2] sines
   pdl_wait();
@@ -81,24 +92,29 @@ __global__ void __launch_bounds__(HEAD_WARPS * 32) head_norm_cache_kernel(T* __r
     const float* w = is_q ? q_w : k_w;
     if (is_q && !w && rot == 0) continue;
     T* dst = is_q ? x : kcache + ((page * nkv + (h - nh)) * block_size + place) * dk;
-    float a[HEAD_PAIRS], b[HEAD_PAIRS], ss = 0.f;
+    float a[PAIRS], b[PAIRS], ss = 0.f;
 #pragma unroll
-    for (int k = 0; k < HEAD_PAIRS; ++k) {
+    for (int k = 0; k < PAIRS; ++k) {
       // pair i: dims (2i, 2i+1), or (i, i + rot/2) among the dims that turn in split pairs
       const int i = lane + 32 * k;
       a[k] = b[k] = 0.f;
       if (2 * i >= dk) continue;
-      const bool split = split_pairs && 2 * i < rot;
-      a[k] = to_float<T>(x[split ? i : 2 * i]);
-      b[k] = to_float<T>(x[split ? i + half : 2 * i + 1]);
+      if (SPLIT && i < half) {
+        a[k] = to_float<T>(x[i]);
+        b[k] = to_float<T>(x[i + half]);
+      } else {
+        const float2 v = Two<T>::load(x + 2 * i);
+        a[k] = v.x;
+        b[k] = v.y;
+      }
       ss = fmaf(a[k], a[k], fmaf(b[k], b[k], ss));
     }
     const float r = w ? 1.f / sqrtf(warp_sum(ss) / count + eps) : 1.f;
 #pragma unroll
-    for (int k = 0; k < HEAD_PAIRS; ++k) {
+    for (int k = 0; k < PAIRS; ++k) {
       const int i = lane + 32 * k;
       if (2 * i >= dk) continue;
-      const bool turns = 2 * i < rot, split = split_pairs && turns;
+      const bool turns = i < half, split = SPLIT && turns;
       const int ia = split ? i : 2 * i, ib = split ? i + half : 2 * i + 1;
       float u = a[k], v = b[k];
       if (w) {
@@ -111,10 +127,21 @@ __global__ void __launch_bounds__(HEAD_WARPS * 32) head_norm_cache_kernel(T* __r
         u = yu;
         v = yv;
       }
-      dst[ia] = from_float<T>(u);
-      dst[ib] = from_float<T>(v);
+      if (split) {
+        dst[ia] = from_float<T>(u);
+        dst[ib] = from_float<T>(v);
+      } else {
+        Two<T>::store(dst + ia, u, v);
+      }
     }
   }
+}
+
+template <typename T>
+auto head_norm_kernel(int dk, bool split) {
+  if (dk <= 64) return split ? head_norm_cache_kernel<T, 1, true> : head_norm_cache_kernel<T, 1, false>;
+  if (dk <= 128) return split ? head_norm_cache_kernel<T, 2, true> : head_norm_cache_kernel<T, 2, false>;
+  return split ? head_norm_cache_kernel<T, HEAD_PAIRS, true> : head_norm_cache_kernel<T, HEAD_PAIRS, false>;
 }
 
 // ---------------------------------------------------------------- RMS norm of a column range
@@ -261,10 +288,12 @@ inline unsigned grid_for(long long total, int threads) {
     if (dk <= 0 || (dk & 1) || dk > 64 * HEAD_PAIRS || rot < 0 || rot > dk || (rot & 1))                             \
       return (int)cudaErrorInvalidValue;                                                                             \
     if ((v_first && !v_lambda) || count <= 0 || count > dk) return (int)cudaErrorInvalidValue;                       \
+    if ((row_stride & 1) || ((((uintptr_t)qkv) | ((uintptr_t)kcache)) & (2 * sizeof(T) - 1)))                       \
+      return (int)cudaErrorInvalidValue;                                                                             \
     const int groups = (nh + 2 * nkv + HEAD_WARPS - 1) / HEAD_WARPS;                                                 \
-    return launch(head_norm_cache_kernel<T>, dim3(n_tokens, n_tokens <= 256 ? groups : 1), dim3(HEAD_WARPS * 32),    \
+    return launch(head_norm_kernel<T>(dk, split_pairs != 0), dim3(n_tokens, n_tokens <= 256 ? groups : 1), dim3(HEAD_WARPS * 32),    \
                   (size_t)rot * sizeof(float), st, (T*)qkv, row_stride, positions, q_w, k_w, eps, inv_freq, rot,     \
-                  slots, (T*)kcache, (T*)vcache, nh, nkv, dk, dv, block_size, num_slots, err, split_pairs,           \
+                  slots, (T*)kcache, (T*)vcache, nh, nkv, dk, dv, block_size, num_slots, err,                        \
                   (T*)v_keep, (const T*)v_first, v_lambda, (float)count, magnitude);                                 \
   }                                                                                                                  \
   KVF_API int kvf_row_rmsnorm_##SUF(const void* x, long long x_stride, const float* w, float eps, long long n_rows,  \

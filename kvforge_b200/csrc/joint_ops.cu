@@ -103,15 +103,7 @@ __global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParam
   const int half = p.rot >> 1;
   float* cs = row + qk;
   float* sn = cs + half;
-  if (p.rot) {
-    const float pos = (float)p.positions[n];
-    for (int i = threadIdx.x; i < half; i += blockDim.x) {
-      float s, c;
-      sincosf(pos * p.inv_freq[i], &s, &c);
-      cs[i] = c * p.magnitude;
-      sn[i] = s * p.magnitude;
-    }
-  }
+  const float pos = p.rot ? (float)p.positions[n] : 0.f;
   float sq = 0.f, sk = 0.f;
   for (int c = threadIdx.x * V; c < qk; c += blockDim.x * V) {
     float f[V];
@@ -126,7 +118,19 @@ __global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParam
 #pragma unroll
     for (int e = 0; e < V; ++e) s = fmaf(f[e], f[e], s);
     if (c < q_dim) sq += s; else sk += s;
-    Pack<float, V>::store(row + c, f);
+    if (p.qw) {
+      float w[V];
+      Pack<float, V>::load(c < q_dim ? p.qw + c : p.kw + (c - q_dim), w);
+#pragma unroll
+      for (int e = 0; e < V; ++e) f[e] *= w[e];
+    }
+    Pack<float, V>::store(row + c, f);  // lacks the norm's one factor for all of q or of k
+  }
+  for (int i = threadIdx.x; i < half; i += blockDim.x) {
+    float s, c;
+    sincosf(pos * p.inv_freq[i], &s, &c);
+    cs[i] = c * p.magnitude;
+    sn[i] = s * p.magnitude;
   }
   float rq = 1.f, rk = 1.f;
   if (p.qw) {
@@ -160,18 +164,11 @@ __global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParam
     float f[V];
     Pack<float, V>::load(row + c, f);
     const bool is_q = c < q_dim;
-    if (p.qw) {
-      float w[V];
-      Pack<float, V>::load(is_q ? p.qw + c : p.kw + (c - q_dim), w);
-      const float r = is_q ? rq : rk;
+    const float r = is_q ? rq : rk;
 #pragma unroll
-      for (int e = 0; e < V; ++e) f[e] = f[e] * r * w[e];
-    }
+    for (int e = 0; e < V; ++e) f[e] *= r;
     const int j0 = c % p.dk;  // V numbers of one head from its j0 on
     if (j0 < p.rot) {
-      const float* w = is_q ? p.qw : p.kw;
-      const int c_of_w = is_q ? c : c - q_dim;
-      const float r = is_q ? rq : rk;
       if (V == 4 && p.interleaved && j0 + 4 <= p.rot) {  // whole pairs
 #pragma unroll
         for (int e = 0; e < V; e += 2) {
@@ -188,15 +185,10 @@ __global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParam
         Pack<float, V>::load(row + c + d, other);
         Pack<float, V>::load(cs + i, c4);
         Pack<float, V>::load(sn + i, s4);
-        if (p.qw) {
-          float w2[V];
-          Pack<float, V>::load(w + c_of_w + d, w2);
-#pragma unroll
-          for (int e = 0; e < V; ++e) other[e] = other[e] * r * w2[e];
-        }
 #pragma unroll
         for (int e = 0; e < V; ++e) {
           float a, b;
+          other[e] *= r;
           rotate_pair(first ? f[e] : other[e], first ? other[e] : f[e], c4[e], s4[e], a, b);
           f[e] = first ? a : b;
         }
@@ -208,9 +200,7 @@ __global__ void __launch_bounds__(1024) joint_norm_cache_kernel(const JointParam
           const bool first = p.interleaved ? !(j & 1) : j < half;
           const int d = p.interleaved ? (first ? 1 : -1) : (first ? half : -half);  // where the pair's other number is
           const int i = p.interleaved ? j >> 1 : (first ? j : j - half);
-          float other = row[c + e + d];
-          if (p.qw) other = other * r * w[c_of_w + e + d];
-          const float own = p.qw ? row[c + e] * r * w[c_of_w + e] : row[c + e];
+          const float other = row[c + e + d] * r, own = row[c + e] * r;
           float a, b;
           if (first)
             rotate_pair(own, other, cs[i], sn[i], a, b);

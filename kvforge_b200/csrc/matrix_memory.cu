@@ -26,7 +26,7 @@ using namespace kvf;
 namespace {
 
 constexpr float READ_EPS = 1e-6f;  // joins the divisor of the read-out
-constexpr int GATE_CHUNK = 1024;   // tokens a CTA of the gates kernel takes at a time, at most
+constexpr int GATE_CHUNK = 512;    // tokens a CTA of the gates kernel takes at a time, at most
 
 template <typename T, int V> struct Run;
 template <typename T> struct Run<T, 1> {
@@ -97,41 +97,52 @@ __device__ __forceinline__ void leave_gates(const GateParams& p, long long n, in
 }
 
 // A CTA per (head, sequence).  The maximum is carried by one thread, token by token, so it is the same bits however the
-// sequence is cut into steps.
-__global__ void __launch_bounds__(GATE_CHUNK) memory_gates_kernel(const GateParams p) {
+// sequence is cut into steps; while it goes through one stretch of tokens the other warps work out the next stretch's log gates and
+// write the stretch before's results.
+__global__ void __launch_bounds__(GATE_CHUNK + 32) memory_gates_kernel(const GateParams p) {
   pdl_launch();
   pdl_wait();
-  __shared__ __align__(16) float fs[GATE_CHUNK], is[GATE_CHUNK], ms[GATE_CHUNK + 1];
-  const int h = blockIdx.x, b = blockIdx.y, t = threadIdx.x, chunk = blockDim.x;
+  __shared__ __align__(16) float fs[3][GATE_CHUNK], is[3][GATE_CHUNK], ms[3][GATE_CHUNK + 4];  // ms[.][3]: the maximum before the stretch
+  const int h = blockIdx.x, b = blockIdx.y, chunk = blockDim.x - 32, t = threadIdx.x;
   const int begin = p.qsl[b], len = p.qsl[b + 1] - begin, slot = p.slots[b];
   if (len <= 0 || slot < 0) return;
   float* mem = p.m + (size_t)slot * p.state_stride + h;
-  if (t == 0) ms[0] = *mem;
-  for (int t0 = 0; t0 < len; t0 += chunk) {
-    const int n = min(chunk, len - t0);
-    float li = 0.f, lf = 0.f;
-    if (t < n) log_gates(p, begin + t0 + t, h, li, lf);
-    fs[t] = lf;
-    is[t] = li;
-    __syncthreads();
-    if (t == 0) {
-      float m = ms[0];
-      int j = 0;
-      for (; j + 4 <= n; j += 4) {
-        const float4 f4 = *reinterpret_cast<const float4*>(fs + j), i4 = *reinterpret_cast<const float4*>(is + j);
-        ms[j + 1] = m = fmaxf(f4.x + m, i4.x);
-        ms[j + 2] = m = fmaxf(f4.y + m, i4.y);
-        ms[j + 3] = m = fmaxf(f4.z + m, i4.z);
-        ms[j + 4] = m = fmaxf(f4.w + m, i4.w);
+  const int chunks = (len + chunk - 1) / chunk;
+  float m = t == chunk ? *mem : 0.f;
+  for (int it = 0; it < chunks + 2; ++it) {
+    if (t < chunk) {
+      if (it < chunks && it * chunk + t < len) {
+        float li, lf;
+        log_gates(p, begin + it * chunk + t, h, li, lf);
+        fs[it % 3][t] = lf;
+        is[it % 3][t] = li;
       }
-      for (; j < n; ++j) ms[j + 1] = m = fmaxf(fs[j] + m, is[j]);
+      const int done = it - 2;
+      if (done >= 0 && done * chunk + t < len) {
+        const float* mm = ms[done % 3] + 3;
+        leave_gates(p, begin + done * chunk + t, h, is[done % 3][t], fs[done % 3][t], mm[t], mm[t + 1]);
+      }
+    } else if (t == chunk && it >= 1 && it <= chunks) {
+      const int c = it - 1, n = min(chunk, len - c * chunk);
+      const float *f = fs[c % 3], *i = is[c % 3];
+      float* mm = ms[c % 3] + 3;
+      mm[0] = m;
+      int j = 0;
+#pragma unroll 2
+      for (; j + 4 <= n; j += 4) {
+        const float4 f4 = *reinterpret_cast<const float4*>(f + j), i4 = *reinterpret_cast<const float4*>(i + j);
+        float4 o;
+        o.x = fmaxf(f4.x + m, i4.x);
+        o.y = fmaxf(f4.y + o.x, i4.y);
+        o.z = fmaxf(f4.z + o.y, i4.z);
+        o.w = m = fmaxf(f4.w + o.z, i4.w);
+        *reinterpret_cast<float4*>(mm + 1 + j) = o;
+      }
+      for (; j < n; ++j) mm[j + 1] = m = fmaxf(f[j] + m, i[j]);
     }
     __syncthreads();
-    if (t < n) leave_gates(p, begin + t0 + t, h, li, lf, ms[t], ms[t + 1]);
-    __syncthreads();
-    if (t == 0) ms[0] = ms[n];
   }
-  if (t == 0) *mem = ms[0];
+  if (t == chunk) *mem = m;
 }
 
 struct PrepareParams {
@@ -267,7 +278,7 @@ int memory_run(const GateParams& g0, const PrepareParams& p, float* state, float
     rc = launch(vec ? memory_step_kernel<T, 4> : memory_step_kernel<T, 1>, dim3(B, (H + STEP_HEADS - 1) / STEP_HEADS), dim3(256), 0, st, p, g);
     if (rc) return rc;
   } else {
-    rc = launch(memory_gates_kernel, dim3(H, B), dim3(max_q_len > 0 && max_q_len <= 256 ? 256 : GATE_CHUNK), 0, st, g);
+    rc = launch(memory_gates_kernel, dim3(H, B), dim3((max_q_len > 0 && max_q_len <= 128 ? 128 : GATE_CHUNK) + 32), 0, st, g);
     if (rc) return rc;
     rc = launch(vec ? memory_prepare_kernel<T, 4> : memory_prepare_kernel<T, 1>, dim3((unsigned)N), dim3(256), 0, st, p, H, (const float*)g.inflow);
     if (rc) return rc;
