@@ -10,8 +10,8 @@
 //             g' = min(g, limit), u' = clamp(u, -limit, limit), g' / (1 + exp(-alpha g')) * (u' + shift)
 //   combine : resid[token] += sum_k weight_k * y[token, k]   (float, k in order)
 //
-// The router may have more outputs than there are experts: a choice beyond the last expert is an identity expert, whose result is
-// the token's own input; its pair enters no product, and combine takes x[token] for it.
+// The router may have more outputs than there are experts: a choice beyond the last expert hands the
+// token's own input on; its pair enters no product, and combine takes x[token] for it.
 //
 // A pair's row of a product depends on that row and on its expert's weights alone (its products are
 // added in the order of k: by one thread on the FP32 pipes, by the tensor cores' own order in bfloat16),

@@ -161,6 +161,61 @@ __device__ __forceinline__ void reg_stats(const float (&x)[NIT][4], const bool (
   rstd = 1.f / sqrtf(block_sum(q, red) / (float)W + eps);
 }
 
+// The same with nothing pending, nothing replaced and a norm: the row is read once and its normed rows go out, the statistics through one
+// barrier each.
+template <typename T, int NIT, int TH>
+__global__ void __launch_bounds__(TH) norm_rows_kernel(const NormStepParams p) {
+  pdl_launch();
+  pdl_wait();
+  __shared__ float red[64];
+  const int W = p.W, r = blockIdx.x, lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
+  const float* h = p.resid + (size_t)(p.rows ? p.rows[r] : r) * W;
+  float x[NIT][4], w[NIT][4], b[NIT][4];
+  float s = 0.f;
+#pragma unroll
+  for (int it = 0; it < NIT; ++it) {
+    const int i = (it * TH + threadIdx.x) * 4;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[it][e] = w[it][e] = b[it][e] = 0.f;
+    if (i >= W) continue;
+    Vec4<float>::load(h + i, x[it]);
+    Vec4<float>::load(p.next_w + i, w[it]);
+    if (p.next_b) Vec4<float>::load(p.next_b + i, b[it]);
+  }
+  float mean = 0.f;
+  if (p.centred) {
+#pragma unroll
+    for (int it = 0; it < NIT; ++it) s += (x[it][0] + x[it][1]) + (x[it][2] + x[it][3]);
+    s = warp_sum(s);
+    if (lane == 0) red[warp] = s;
+    __syncthreads();
+    mean = warp_sum(lane < TH / 32 ? red[lane] : 0.f) / (float)W;
+  }
+  float q = 0.f;
+#pragma unroll
+  for (int it = 0; it < NIT; ++it) {
+    if ((it * TH + threadIdx.x) * 4 >= W) continue;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) {
+      const float d = x[it][e] - mean;
+      q = fmaf(d, d, q);
+    }
+  }
+  q = warp_sum(q);
+  if (lane == 0) red[32 + warp] = q;
+  __syncthreads();
+  const float rstd = 1.f / sqrtf(warp_sum(lane < TH / 32 ? red[32 + lane] : 0.f) / (float)W + p.eps);
+  T* o = (T*)p.out + (size_t)r * p.out_stride;
+#pragma unroll
+  for (int it = 0; it < NIT; ++it) {
+    const int i = (it * TH + threadIdx.x) * 4;
+    if (i >= W) continue;
+#pragma unroll
+    for (int e = 0; e < 4; ++e) x[it][e] = fmaf((x[it][e] - mean) * rstd, w[it][e], b[it][e]);
+    Vec4<T>::store(o + i, x[it]);
+  }
+}
+
 template <typename T, int NIT, int TH>
 __global__ void __launch_bounds__(TH) norm_step_vec_kernel(const NormStepParams p) {
   pdl_launch();
@@ -414,6 +469,11 @@ KVF_API int kvf_gated_set_pdl(int enabled) {
     p.nsplit = nsplit; p.z = z; p.z_stride = z_stride; p.z_bias = z_bias; p.y_bias = y_bias; p.post_w = post_w; p.next_w = next_w; p.next_b = next_b; \
     p.out = out; p.out_stride = out_stride; p.W = W; p.centred = centred; p.store_normed = store_normed; p.eps = eps; \
     if (norm_step_vec_ok<T>(p)) {                                                                                     \
+      if (!y && !y_parts && !store_normed && next_w && out) {                                                         \
+        if (W <= 1024) return launch(norm_rows_kernel<T, 2, 128>, dim3(n_rows), dim3(128), 0, st, p);                 \
+        if (W <= 2048) return launch(norm_rows_kernel<T, 4, 128>, dim3(n_rows), dim3(128), 0, st, p);                 \
+        return launch(norm_rows_kernel<T, 4, 256>, dim3(n_rows), dim3(256), 0, st, p);                                \
+      }                                                                                                               \
       /* few rows of slices in bfloat16: a thread for every four numbers, so that all slices of a row are asked for at once */ \
       const bool few = sizeof(T) == 2 && y_parts && n_rows <= 148;                                                    \
       if (W <= 1024) return launch(norm_step_vec_kernel<T, 1, 256>, dim3(n_rows), dim3(256), 0, st, p);               \

@@ -128,15 +128,23 @@ __global__ void __launch_bounds__(GATE_CHUNK + 32) memory_gates_kernel(const Gat
       float* mm = ms[c % 3] + 3;
       mm[0] = m;
       int j = 0;
-#pragma unroll 2
-      for (; j + 4 <= n; j += 4) {
-        const float4 f4 = *reinterpret_cast<const float4*>(f + j), i4 = *reinterpret_cast<const float4*>(i + j);
-        float4 o;
-        o.x = fmaxf(f4.x + m, i4.x);
-        o.y = fmaxf(f4.y + o.x, i4.y);
-        o.z = fmaxf(f4.z + o.y, i4.z);
-        o.w = m = fmaxf(f4.w + o.z, i4.w);
-        *reinterpret_cast<float4*>(mm + 1 + j) = o;
+      // Rounding is monotone: max(a, b) + f, rounded, is the larger of a + f and b + f, rounded.  So what eight tokens make of the inputs among
+      // them is worked out beside the chain, which is eight additions and one maximum for eight tokens, with the same bits.
+      for (; j + 8 <= n; j += 8) {
+        float fj[8], c[8], a[8];
+        *reinterpret_cast<float4*>(fj) = *reinterpret_cast<const float4*>(f + j);
+        *reinterpret_cast<float4*>(fj + 4) = *reinterpret_cast<const float4*>(f + j + 4);
+        *reinterpret_cast<float4*>(c) = *reinterpret_cast<const float4*>(i + j);
+        *reinterpret_cast<float4*>(c + 4) = *reinterpret_cast<const float4*>(i + j + 4);
+#pragma unroll
+        for (int e = 1; e < 8; ++e) c[e] = fmaxf(fj[e] + c[e - 1], c[e]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) a[e] = fj[e] + (e ? a[e - 1] : m);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) a[e] = fmaxf(a[e], c[e]);
+        m = a[7];
+        *reinterpret_cast<float4*>(mm + 1 + j) = *reinterpret_cast<const float4*>(a);
+        *reinterpret_cast<float4*>(mm + 5 + j) = *reinterpret_cast<const float4*>(a + 4);
       }
       for (; j < n; ++j) mm[j + 1] = m = fmaxf(f[j] + m, i[j]);
     }
@@ -219,48 +227,65 @@ __global__ void __launch_bounds__(256) memory_step_kernel(const PrepareParams p,
   widen<T, V>(p, n, g.H, h0, h1, in);
 }
 
-// A warp per (token, head).  out = y / sqrt(mean(y^2) + eps) * w * act(gate), y the read-out over its divisor; act: 0 none, 2 the
-// logistic function.
-template <typename T, int V>
+// A warp per (token, head).  out = y / sqrt(mean(y^2) + eps) * w * sigmoid(gate) (without a gate: * 1), y the read-out over its divisor.
+// NIT: how many times 32 * V numbers a lane keeps in registers (a head has at most NIT * 32 * V).
+__device__ __forceinline__ float logistic(float z, bool exact) { return exact ? 1.f / (1.f + expf(-z)) : __fdividef(1.f, 1.f + __expf(-z)); }
+
+template <typename T, int V, int NIT>
 __global__ void __launch_bounds__(128) memory_read_kernel(const float* __restrict__ o, long long ldo, const float* __restrict__ floor_,
                                                            const T* __restrict__ gate, long long ldg, const float* __restrict__ w, float eps,
                                                            long long pairs, int H, int dv, int dvx, T* __restrict__ out, long long ldout) {
   pdl_launch();
   pdl_wait();
+  constexpr bool EXACT = sizeof(T) == 4;  // float storage: the library's exponential; bfloat16: the fast one, rounded right after
   const long long pair = (long long)blockIdx.x * 4 + (threadIdx.x >> 5);
   if (pair >= pairs) return;
   const int lane = threadIdx.x & 31;
   const long long n = pair / H;
   const int h = (int)(pair - n * H);
   const float* row = o + n * ldo + (size_t)h * dvx;
+  const T* g = gate ? gate + n * ldg + (size_t)h * dv : nullptr;
+  float f[NIT][V], z[NIT][V], wv[NIT][V];  // everything is asked for before the first number is used
+#pragma unroll
+  for (int it = 0; it < NIT; ++it) {
+    const int j = (it * 32 + lane) * V;
+#pragma unroll
+    for (int e = 0; e < V; ++e) f[it][e] = z[it][e] = wv[it][e] = 0.f;
+    if (j >= dv) continue;
+    Run<float, V>::load(row + j, f[it]);
+    Run<float, V>::load(w + (size_t)h * dv + j, wv[it]);
+    if (g) Run<T, V>::load(g + j, z[it]);
+  }
   const float one_over = 1.f / (fmaxf(fabsf(row[dv]), floor_[pair]) + READ_EPS);
   float ss = 0.f;
-  for (int j = lane * V; j < dv; j += 32 * V) {
-    float f[V];
-    Run<float, V>::load(row + j, f);
+#pragma unroll
+  for (int it = 0; it < NIT; ++it)
 #pragma unroll
     for (int e = 0; e < V; ++e) {
-      const float y = f[e] * one_over;
-      ss = fmaf(y, y, ss);
+      f[it][e] *= one_over;
+      ss = fmaf(f[it][e], f[it][e], ss);
     }
-  }
   const float r = 1.f / sqrtf(warp_sum(ss) / (float)dv + eps);
-  const T* g = gate ? gate + n * ldg + (size_t)h * dv : nullptr;
   T* dst = out + n * ldout + (size_t)h * dv;
-  for (int j = lane * V; j < dv; j += 32 * V) {
-    float f[V], wv[V];
-    Run<float, V>::load(row + j, f);
-    Run<float, V>::load(w + (size_t)h * dv + j, wv);
 #pragma unroll
-    for (int e = 0; e < V; ++e) f[e] = f[e] * one_over * r * wv[e];
-    if (g) {
-      float z[V];
-      Run<T, V>::load(g + j, z);
+  for (int it = 0; it < NIT; ++it) {
+    const int j = (it * 32 + lane) * V;
+    if (j >= dv) continue;
 #pragma unroll
-      for (int e = 0; e < V; ++e) f[e] *= 1.f / (1.f + expf(-z[e]));
+    for (int e = 0; e < V; ++e) {
+      f[it][e] = f[it][e] * r * wv[it][e];
+      if (g) f[it][e] *= logistic(z[it][e], EXACT);
     }
-    Run<T, V>::store(dst + j, f);
+    Run<T, V>::store(dst + j, f[it]);
   }
+}
+
+constexpr int READ_MAX = 1024;  // numbers of a head's value
+
+template <typename T>
+auto memory_read(bool vec, int dv) {
+  if (vec) return dv <= 128 ? memory_read_kernel<T, 4, 1> : dv <= 256 ? memory_read_kernel<T, 4, 2> : memory_read_kernel<T, 4, READ_MAX / 128>;
+  return dv <= 64 ? memory_read_kernel<T, 1, 2> : memory_read_kernel<T, 1, READ_MAX / 32>;
 }
 
 inline bool aligned(const void* p, size_t n) { return p == nullptr || ((uintptr_t)p % n) == 0; }
@@ -324,10 +349,10 @@ KVF_API int kvf_memory_columns(int dv) { return (dv + 4) & ~3; }
                                     long long ldout, cudaStream_t st) {                                                 \
     const long long pairs = N * H;                                                                                      \
     if (pairs <= 0) return 0;                                                                                           \
-    if (dv <= 0 || !w || !floor_) return (int)cudaErrorInvalidValue;                                                    \
+    if (dv <= 0 || dv > READ_MAX || !w || !floor_) return (int)cudaErrorInvalidValue;                                   \
     const bool vec = dv % 4 == 0 && ldo % 4 == 0 && ldg % 4 == 0 && ldout % 4 == 0 && aligned(o, 16) && aligned(w, 16) && \
                      aligned(gate, 4 * sizeof(T)) && aligned(out, 4 * sizeof(T));                                       \
-    return launch(vec ? memory_read_kernel<T, 4> : memory_read_kernel<T, 1>, dim3((unsigned)((pairs + 3) / 4)),         \
+    return launch(memory_read<T>(vec, dv), dim3((unsigned)((pairs + 3) / 4)),                                           \
                   dim3(128), 0, st, o, ldo, floor_, (const T*)gate, ldg, w, eps, pairs, H, dv, kvf_memory_columns(dv),  \
                   (T*)out, ldout);                                                                                      \
   }

@@ -2396,6 +2396,7 @@ def add_position_rows(resid: torch.Tensor, table: torch.Tensor, positions: torch
 
 MEMORY_LIB = "memory"
 MEMORY_MAX_KEY_DIM = RETENTION_MAX_KEY_DIM  # the same walk
+MEMORY_MAX_VALUE_DIM = 1024  # numbers of a head that a warp of the read-out holds in registers
 
 
 def memory_columns(dv: int) -> int:
@@ -2421,8 +2422,8 @@ def matrix_memory(
     s = _suffix(x.dtype)
     _rows2d(x, None, "x")
     n, h, dvx = x.shape[0], int(num_heads), memory_columns(dv)
-    if not 0 < dk <= MEMORY_MAX_KEY_DIM or dv <= 0:
-        raise ValueError(f"matrix_memory: key heads of 1 to {MEMORY_MAX_KEY_DIM} numbers")
+    if not 0 < dk <= MEMORY_MAX_KEY_DIM or not 0 < dv <= MEMORY_MAX_VALUE_DIM:
+        raise ValueError(f"matrix_memory: key heads of 1 to {MEMORY_MAX_KEY_DIM} numbers, value heads of 1 to {MEMORY_MAX_VALUE_DIM}")
     if max(q_off, k_off) + h * dk > x.shape[1] or v_off + h * dv > x.shape[1]:
         raise ValueError("matrix_memory: the columns do not fit the rows")
     if isinstance(logits, Partials):

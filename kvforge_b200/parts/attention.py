@@ -94,8 +94,8 @@ class PagedAttention(Mixer):
     scores by ``distance_buckets`` of the distance between query and key), ``keep_first`` (with a
     window: the first keys of a sequence that every later query sees, at their true positions),
     ``softcap`` (``c``: a scaled score ``s`` becomes ``c * tanh(s / c)``), ``sink`` (true: the tensor ``sink [num_heads]``;
-    ``exp(sink_h)`` joins the softmax's denominator of head ``h`` without a key or a value; ``"zero"``: a sink whose score is 0 in every
-    head, so one joins the denominator, and no tensor), ``keep_window`` (the cache keeps at least so many keys because a later
+    ``exp(sink_h)`` joins the softmax's denominator of head ``h`` without a key or a value; ``"zero"``: every head's sink stands at score
+    zero, so its exponential is one, and there is no tensor), ``keep_window`` (the cache keeps at least so many keys because a later
     layer that reads it sees them), ``pad_heads`` (heads whose size is no multiple of 8 are padded with zeros when the tensors are bound:
     that changes neither a norm's sum nor a score nor, through zero columns of the output projection, the result) and ``value_mix``
     (``"source"``: the values as projected are also kept for the later layers of the step; ``"mix"``: the values become

@@ -11,8 +11,8 @@ A router may add a bias to its logits (``z = W_router x + b``), and its weights 
 logits alone (the logits then rank the experts).  A gated expert is ``W_down[e] join(W_gate[e] x, W_up[e] x)`` with
 ``join(g, u) = g' sigmoid(alpha g') (u' + shift)``, ``g' = min(g, limit)``, ``u' = clamp(u, -limit, limit)``.
 
-The router may have more outputs than there are experts: the last ones are identity experts, which have no tensors and whose
-result is the input itself.
+The router may have more outputs than there are experts: a token that picks one of the last outputs gets its own input handed on,
+weighted like an expert's result (an identity expert).
 """
 
 from __future__ import annotations

@@ -1,8 +1,8 @@
 """Grouped-query attention whose query rows (and key rows) are normed as one vector and whose result may be gated.
 
-Per layer ``q = W_q x + b_q``, ``k = W_k x + b_k``, ``v = W_v x + b_v`` (the biases are optional); q and k are RMS-normed over
-all their numbers at once, before they are split into heads, with weights as wide as the projections; then the first
-dims of every head may turn with the position.  Attention sees every earlier key, a sliding window of them, or the keys of the query's own chunk.  The
+Per layer ``q = W_q x + b_q``, ``k = W_k x + b_k``, ``v = W_v x + b_v`` (the biases are optional); q and k are RMS-normed as
+one vector each (all heads together), with weights as wide as the projections; then the first dims of every head may turn
+with the position.  Attention sees every earlier key, a sliding window of them, or the keys of the query's own chunk.  The
 result may be multiplied by ``sigmoid(W_g x)``, one number a head or one a channel, before the output projection.  A layer may
 use the keys and values of an earlier layer (as that layer's cache holds them) with queries of its own.
 

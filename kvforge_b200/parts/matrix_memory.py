@@ -9,8 +9,8 @@ gates a head whose logarithms are ``i = c tanh((W_i x + b_i) / c)`` and ``f = lo
     S <- e^(f + m_before - m) S + e^(i - m) k v^T        n <- e^(f + m_before - m) n + e^(i - m) k
     o = S^T q / (max(|n . q|, e^(-m)) + 1e-6)
 
-Every head's ``o`` is divided by its root mean square, the heads side by side are multiplied by a weight and by
-``sigmoid(W_g x)``, then the output projection.  Everything from the gates' logits on is 32-bit.  A request's state is one row of
+The read-out is scaled to unit root mean square head by head; a weight as wide as all heads and ``sigmoid(W_g x)`` multiply it before
+the output projection.  Everything from the gates' logits on is 32-bit.  A request's state is one row of
 floats: per head ``S`` with ``n`` as one more column (``ops.memory_columns``), then the heads' ``m``; the mixer keeps no pages.
 """
 
@@ -40,8 +40,8 @@ class MatrixMemory(Mixer):
         p = params
         self.hidden, self.H, self.dk, self.dv = (int(p[k]) for k in ("hidden_size", "num_heads", "head_dim", "v_head_dim"))
         self.cap, self.eps = float(p["gate_cap"]), float(p["eps"])
-        if not 0 < self.dk <= ops.MEMORY_MAX_KEY_DIM or self.dv <= 0 or self.H <= 0:
-            raise ValueError(f"matrix_memory takes key heads of 1 to {ops.MEMORY_MAX_KEY_DIM} numbers")
+        if not 0 < self.dk <= ops.MEMORY_MAX_KEY_DIM or not 0 < self.dv <= ops.MEMORY_MAX_VALUE_DIM or self.H <= 0:
+            raise ValueError(f"matrix_memory takes key heads of 1 to {ops.MEMORY_MAX_KEY_DIM} numbers and value heads of 1 to {ops.MEMORY_MAX_VALUE_DIM}")
         if not self.cap > 0:
             raise ValueError("gate_cap must be positive")
         self.dvx = ops.memory_columns(self.dv)

@@ -12,7 +12,7 @@ llama3 scaling is not in kvforge; Llama 3.1/3.2 checkpoints need it.  For wavele
 YaRN scaling ("YaRN: Efficient Context Window Extension of Large Language Models", Peng et al.) blends by the index of a pair
 instead: the (fractional) pair whose wave turns ``t`` times within the original context ``P`` is ``rot ln(P / (2 pi t)) / (2 ln theta)``;
 from the one of ``fast`` turns (rounded down) to the one of ``slow`` turns (rounded up) the frequencies go linearly from ``f`` to
-``f/factor``.  Cosine and sine are multiplied by ``0.1 ln(factor) + 1``, the encoding's ``magnitude``.
+``f/factor``.  What turns also grows by the encoding's ``magnitude``, ``1 + ln(factor) / 10``.
 """
 
 from __future__ import annotations
